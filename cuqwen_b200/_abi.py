@@ -18,12 +18,19 @@ class Params(C.Structure):
         ("flags", C.c_uint32), ("norm_eps", C.c_float), ("rope_theta", C.c_float), ("repetition_penalty", C.c_float)]
 
 
+class OpenParams(C.Structure):
+    _fields_ = [("act", C.c_int32), ("max_seq_len", C.c_int32), ("device", C.c_int32), ("flags", C.c_uint32), ("repetition_penalty", C.c_float)]
+
+
 _vp, _i, _f, _sz, _l = C.c_void_p, C.c_int, C.c_float, C.c_size_t, C.c_long
 _pi = C.POINTER(C.c_int)
 
 # name -> (restype, argtypes); every symbol the header declares
 SIGNATURES = {
     "cuqwen_model_params": (_i, [_i, _i, C.POINTER(Params)]),
+    "cuqwen_open": (_i, [C.c_char_p, C.POINTER(OpenParams), C.POINTER(_vp)]),
+    "cuqwen_describe": (_i, [C.c_char_p, C.c_char_p, _sz]),
+    "cuqwen_extend": (_i, [_vp, _pi, _i, _i, _pi, _i, C.POINTER(_f)]),
     "cuqwen_create": (_i, [C.POINTER(Params), C.POINTER(_vp)]),
     "cuqwen_destroy": (None, [_vp]),
     "cuqwen_load": (_i, [_vp, C.c_char_p]),

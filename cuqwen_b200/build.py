@@ -94,6 +94,18 @@ def build_cuda(verbose: bool = False) -> Path:
     return LIB
 
 
+def ensure_cuda() -> Path:
+    """The CUDA library, built (and nothing else) when it is missing or older than its sources; one process at a time."""
+    import fcntl
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        deps = [p for pat in ("*.cu", "*.cuh", "*.h") for p in CSRC.glob(pat)] + [ROOT / "include" / "cuqwen_b200.h"]
+        if _newer(LIB, deps):
+            build_cuda()
+    return LIB
+
+
 def build_oracle() -> Path:
     if _newer(ORACLE_LIB, [ORACLE_SRC]):
         _run(["gcc", "-O2", "-fopenmp", "-ffp-contract=off", "-shared", "-fPIC", str(ORACLE_SRC), "-o", str(ORACLE_LIB), "-lm"])

@@ -18,11 +18,13 @@
 
 #include "../../include/cuqwen_b200.h"
 #include "attn.cuh"
+#include "engine.h"
 #include "errors.h"
 #include "gemv.cuh"
 #include "launch.h"
 #include "prefill.cuh"
 #include "prefill_gemm.cuh"
+#include "stack_host.h"
 #include "tp_plan.h"
 
 using namespace cq;
@@ -138,58 +140,28 @@ static int nccl_load() {
 // ---------------------------------------------------------------------------
 // engine
 // ---------------------------------------------------------------------------
-struct Mat { uint8_t* w = nullptr; __half* s = nullptr; int rows = 0, cols = 0; };
-struct Layer {
-    __half *in_norm = nullptr, *post_norm = nullptr, *bq = nullptr, *bk = nullptr, *bv = nullptr;
-    Mat q, k, v, o, gate, up, down;
-};
-
-struct cuqwen_engine {
-    cuqwen_params p{};
-    int sms = 0;
-    cudaStream_t stream = nullptr;
-    TpPlan plan{};
-    int tp = 1, rank = 0;
-    // local sizes
-    int n_heads_l = 0, n_kv_l = 0, q_dim_l = 0, kv_dim_l = 0, inter_l = 0, vocab_l = 0, nsplit = 0;
-    // weights
-    uint8_t* warena = nullptr; size_t warena_bytes = 0;
-    std::vector<Layer> layers;
-    __half *embed = nullptr, *norm = nullptr;
-    Mat lm; int lm_quant = 0; int lm_kind = 0;   // kind: 0 fp16 separate, 1 int8, 2 tied
-    bool loaded = false;
-    uint64_t weight_bytes = 0;                   // algorithmic bytes of all tensors a step reads (this rank)
-    // state
-    __half *x = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *att = nullptr, *gate = nullptr, *logits = nullptr;
-    __half *kc = nullptr, *vc = nullptr;                  // CUQWEN_FLAG_KV_INT8: int8 rows behind these pointers, scales below
-    float *kscale = nullptr, *vscale = nullptr; bool kv8 = false;
-    __half *spare_up = nullptr, *spare_out = nullptr;     // QwenState::up / mlp_out of the source-compatible layer (never read by the step)
-    float *part_o = nullptr, *part_ml = nullptr; unsigned* counters = nullptr;
-    StepCtl* ctl = nullptr; StepCtl* h_ctl = nullptr;
-    HostIo* hio = nullptr; HostIo* hio_dev = nullptr; int io_seq = 0; bool ctl_dirty = true;   // mailbox of cuqwen_step (launch.h); ctl_dirty: the device block must be rewritten first
-    int* d_hist = nullptr; unsigned* bitmap = nullptr; unsigned long long* best = nullptr; unsigned* ticket = nullptr;
-    int* out_ring = nullptr; int ring_cap = 65536; int* h_out = nullptr;   // h_out holds ring_cap + 1 ints
-    float* tp_partial = nullptr; unsigned long long* tp_keys = nullptr;
-    // peer exchange (tensor parallel without collective calls): one receive block per rank, mapped into every peer
-    unsigned char* tp_rx = nullptr; size_t tp_rx_bytes = 0; unsigned char* peer_rx[8] = {}; bool tp_peer = false;
-    __half* x2 = nullptr; bool tp_sum_separate = false;
-    unsigned char* gate_xd = nullptr; int* gate_corr = nullptr; float* gate_xscale = nullptr;    // SwiGLU output in staged form (see GemvArgs::xd_out)
-    unsigned char* att_xd = nullptr; int* att_corr = nullptr; float* att_xscale = nullptr;       // attention output in staged form (see AttnArgs::xd_out)
-    // batched prefill workspace (cuqwen_prefill), allocated at the first call for kPrefillChunk tokens
-    __half *pf_x = nullptr, *pf_xn = nullptr, *pf_q = nullptr, *pf_att = nullptr, *pf_g = nullptr; float* pf_qkv = nullptr; int* pf_tok = nullptr;
-    int steps_done = 0;                          // mirrors the device-side step counter (StepCtl::pad[1])
-    std::vector<cudaEvent_t>* prof = nullptr;    // cuqwen_step_profile: an event is recorded after every launch of the step
-    unsigned long long* step_trace = nullptr; size_t step_trace_bytes = 0;     // CUQWEN_FLAG_STEP_TRACE: eight timeline words per launch (tma.cuh)
-    // graph
-    cudaGraph_t graph = nullptr; cudaGraphExec_t gexec = nullptr; bool graph_ready = false;
-    int launches = 0;
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr; float last_ms = 0.f;
-    // nccl
-    ncclComm_t comm = nullptr;
-};
-
 static size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
 static size_t elem_bytes2(int quant, size_t rows, size_t cols) { return quant == 2 ? rows * cols / 2 : quant == 1 ? rows * cols : rows * cols * 2; }
+
+// What every engine has, whatever its design: stream, events, control block, mailbox, sampler state.
+static int open_device(cuqwen_engine* e) {
+    CK(cudaDeviceGetAttribute(&e->sms, cudaDevAttrMultiProcessorCount, e->p.device));
+    CK(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
+    CK(cudaEventCreate(&e->ev0)); CK(cudaEventCreate(&e->ev1));
+    return CUQWEN_OK;
+}
+static int alloc_step_state(cuqwen_engine* e) {
+    auto dalloc = [&](void** ptr, size_t bytes) -> cudaError_t { cudaError_t r = cudaMalloc(ptr, bytes); if (r == cudaSuccess) r = cudaMemset(*ptr, 0, bytes); return r; };
+    CK(dalloc((void**)&e->ctl, sizeof(StepCtl))); CK(cudaMallocHost((void**)&e->h_ctl, sizeof(StepCtl)));
+    CK(cudaHostAlloc((void**)&e->hio, sizeof(HostIo), cudaHostAllocMapped));
+    memset(e->hio, 0, sizeof(HostIo));
+    CK(cudaHostGetDevicePointer((void**)&e->hio_dev, e->hio, 0));
+    CK(dalloc((void**)&e->d_hist, (size_t)e->p.max_seq_len * 4));
+    CK(dalloc((void**)&e->bitmap, ((size_t)e->vocab_l + 31) / 32 * 4));
+    CK(dalloc((void**)&e->best, 8)); CK(dalloc((void**)&e->ticket, 4));
+    CK(dalloc((void**)&e->out_ring, (size_t)e->ring_cap * 4)); CK(cudaMallocHost((void**)&e->h_out, ((size_t)e->ring_cap + 1) * 4));
+    return CUQWEN_OK;
+}
 
 extern "C" int cuqwen_create(const cuqwen_params* pin, cuqwen_engine** out) {
     if (!pin || !out) return fail(CUQWEN_ERR_ARG, "null argument");
@@ -225,13 +197,11 @@ extern "C" int cuqwen_create(const cuqwen_params* pin, cuqwen_engine** out) {
     e->n_heads_l = plan.qh1 - plan.qh0; e->n_kv_l = plan.kvh1 - plan.kvh0;
     e->q_dim_l = e->n_heads_l * p.head_dim; e->kv_dim_l = e->n_kv_l * p.head_dim;
     e->inter_l = plan.i1 - plan.i0; e->vocab_l = plan.v1 - plan.v0;
-    CK(cudaDeviceGetAttribute(&e->sms, cudaDevAttrMultiProcessorCount, p.device));
+    if (int r = open_device(e)) return r;
     // one CTA per SM and not one more: the partial kernel takes a whole SM's shared memory, so a 149th CTA would wait for
     // a second wave (measured at 40/8 heads, 32K keys: 19 splits 40.7 us, 16 splits 26.9 us)
     e->nsplit = p.attn_splits > 0 ? p.attn_splits : (e->sms / e->n_kv_l > 0 ? e->sms / e->n_kv_l : 1);
     if (e->nsplit > kMaxSplit) e->nsplit = kMaxSplit;
-    CK(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
-    CK(cudaEventCreate(&e->ev0)); CK(cudaEventCreate(&e->ev1));
 
     auto dalloc = [&](void** ptr, size_t bytes) -> cudaError_t { cudaError_t r = cudaMalloc(ptr, bytes); if (r == cudaSuccess) r = cudaMemset(*ptr, 0, bytes); return r; };
     const size_t kvn = (size_t)p.n_layers * e->n_kv_l * p.max_seq_len * p.head_dim;
@@ -252,14 +222,7 @@ extern "C" int cuqwen_create(const cuqwen_params* pin, cuqwen_engine** out) {
     CK(dalloc((void**)&e->part_o, attn_scratch_floats_o(e->n_kv_l, e->nsplit, p.head_dim) * 4));
     CK(dalloc((void**)&e->part_ml, attn_scratch_floats_ml(e->n_kv_l, e->nsplit) * 4));
     CK(dalloc((void**)&e->counters, attn_scratch_counters(e->n_kv_l, e->nsplit) * 4));
-    CK(dalloc((void**)&e->ctl, sizeof(StepCtl))); CK(cudaMallocHost((void**)&e->h_ctl, sizeof(StepCtl)));
-    CK(cudaHostAlloc((void**)&e->hio, sizeof(HostIo), cudaHostAllocMapped));
-    memset(e->hio, 0, sizeof(HostIo));
-    CK(cudaHostGetDevicePointer((void**)&e->hio_dev, e->hio, 0));
-    CK(dalloc((void**)&e->d_hist, (size_t)p.max_seq_len * 4));
-    CK(dalloc((void**)&e->bitmap, ((size_t)e->vocab_l + 31) / 32 * 4));
-    CK(dalloc((void**)&e->best, 8)); CK(dalloc((void**)&e->ticket, 4));
-    CK(dalloc((void**)&e->out_ring, (size_t)e->ring_cap * 4)); CK(cudaMallocHost((void**)&e->h_out, ((size_t)e->ring_cap + 1) * 4));
+    if (int r = alloc_step_state(e)) return r;
     if (e->tp > 1) { CK(dalloc((void**)&e->tp_partial, (size_t)p.dim * 4)); CK(dalloc((void**)&e->tp_keys, (size_t)(e->tp + 1) * 8)); }
     *out = e;
     return CUQWEN_OK;
@@ -268,7 +231,7 @@ extern "C" int cuqwen_create(const cuqwen_params* pin, cuqwen_engine** out) {
 extern "C" void cuqwen_destroy(cuqwen_engine* e) {
     if (!e) return;
     cudaSetDevice(e->p.device);
-    cudaStreamSynchronize(e->stream);
+    if (e->stream) cudaStreamSynchronize(e->stream);
     if (e->gexec) cudaGraphExecDestroy(e->gexec);
     if (e->graph) cudaGraphDestroy(e->graph);
     for (int r = 0; r < 8; ++r) if (e->peer_rx[r] && e->peer_rx[r] != e->tp_rx) cudaIpcCloseMemHandle(e->peer_rx[r]);
@@ -281,9 +244,47 @@ extern "C" void cuqwen_destroy(cuqwen_engine* e) {
     if (e->h_ctl) cudaFreeHost(e->h_ctl);
     if (e->hio) cudaFreeHost(e->hio);
     if (e->h_out) cudaFreeHost(e->h_out);
-    cudaEventDestroy(e->ev0); cudaEventDestroy(e->ev1);
-    cudaStreamDestroy(e->stream);
+    stack_destroy(e);
+    if (e->ev0) cudaEventDestroy(e->ev0);
+    if (e->ev1) cudaEventDestroy(e->ev1);
+    if (e->stream) cudaStreamDestroy(e->stream);
     delete e;
+}
+
+// ---------------------------------------------------------------------------
+// model directories: the design is chosen by config.json (model_dir.h), everything after that by its layer list (stack.h)
+// ---------------------------------------------------------------------------
+extern "C" int cuqwen_describe(const char* dir, char* out, size_t cap) {
+    if (!dir || !out || !cap) return fail(CUQWEN_ERR_ARG, "null argument");
+    StackSpec spec;
+    if (int r = read_model_config(dir, &spec)) return r;
+    const std::string t = describe_spec(spec);
+    if (t.size() + 1 > cap) return fail(CUQWEN_ERR_ARG, "buffer too small: %zu bytes needed", t.size() + 1);
+    memcpy(out, t.c_str(), t.size() + 1);
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_open(const char* dir, const cuqwen_open_params* pin, cuqwen_engine** out) {
+    if (!dir || !out) return fail(CUQWEN_ERR_ARG, "null argument");
+    cuqwen_open_params o{};
+    if (pin) o = *pin;
+    if (o.act != CUQWEN_ACT_BF16 && o.act != CUQWEN_ACT_F32) return fail(CUQWEN_ERR_ARG, "activation type %d out of range", o.act);
+    if (o.flags & ~(uint32_t)(CUQWEN_FLAG_NO_PDL | CUQWEN_FLAG_NO_GRAPH)) return fail(CUQWEN_ERR_ARG, "flags 0x%x do not apply to a model directory", o.flags);
+    if (o.max_seq_len < 0) return fail(CUQWEN_ERR_ARG, "max_seq_len must be positive (or 0 for the default)");
+    StackSpec spec;
+    if (int r = read_model_config(dir, &spec)) return r;
+    CK(cudaSetDevice(o.device));
+    cuqwen_engine* e = new cuqwen_engine();
+    e->p.max_seq_len = o.max_seq_len > 0 ? o.max_seq_len : 32768;
+    e->p.device = o.device; e->p.flags = o.flags; e->p.tp_size = 1; e->p.quant = CUQWEN_FP16;
+    e->p.repetition_penalty = o.repetition_penalty > 0.f ? o.repetition_penalty : 1.1f;
+    int r = open_device(e);
+    if (!r) r = stack_create(e, spec, o.act, e->p.max_seq_len);
+    if (!r) r = alloc_step_state(e);
+    if (!r) r = stack_load(e, dir);
+    if (r) { const std::string msg = g_err; cuqwen_destroy(e); return fail(r, "%s", msg.c_str()); }
+    e->loaded = true;
+    *out = e;
+    return CUQWEN_OK;
 }
 
 // ---------------------------------------------------------------------------
@@ -373,6 +374,7 @@ static int walk_file(cuqwen_engine* e, Cursor cur, Arena& ar, int lm_fmt) {
 
 extern "C" int cuqwen_load(cuqwen_engine* e, const char* path) {
     if (!e || !path) return fail(CUQWEN_ERR_ARG, "null argument");
+    if (e->stack) return fail(CUQWEN_ERR_STATE, "cuqwen_open has loaded this engine's weights");
     if (e->loaded) return fail(CUQWEN_ERR_STATE, "weights already loaded");
     CK(cudaSetDevice(e->p.device));
     int fd = open(path, O_RDONLY);
@@ -564,6 +566,14 @@ static int record_step(cuqwen_engine* e, cudaStream_t s, bool pdl) {
 #define MARK() do { if (e->prof) { cudaEvent_t ev_; CK(cudaEventCreate(&ev_)); CK(cudaEventRecord(ev_, s)); e->prof->push_back(ev_); } } while (0)
 #define LK(call) do { int r_ = (call); if (r_) return fail(CUQWEN_ERR_CUDA, "%s: %s", #call, cudaGetErrorString((cudaError_t)r_)); ++n; MARK(); } while (0)
     MARK();
+    if (e->stack) {
+        if (int r = stack_record_step(e, cfg, [&]() -> int { ++n; MARK(); return CUQWEN_OK; })) return r;
+        float* lg = stack_logits(e->stack);
+        LK(launch_penalty(lg, e->d_hist, &e->ctl->hist_len, e->vocab_l, 0, pen, e->bitmap, cfg));
+        LK(launch_argmax(lg, e->vocab_l, 0, e->ctl, e->out_ring, e->ring_cap, e->d_hist, e->bitmap, e->best, e->ticket, nullptr, nullptr, cfg));
+        e->launches = n;
+        return CUQWEN_OK;
+    }
     LK(launch_embed_step(e->embed, e->ctl, e->x, p.dim, cfg_plain));
     {
         std::vector<HostPhase> hp;
@@ -684,9 +694,75 @@ static int prefill_gemm(cuqwen_engine* e, int mode, const __half* x, const Mat* 
     return CUQWEN_OK;
 }
 
+static int check_tokens(const cuqwen_engine* e, const int* tokens, int n_tokens, int pos0) {
+    if (n_tokens < 1 || pos0 < 0 || n_tokens > e->p.max_seq_len - pos0) return fail(CUQWEN_ERR_ARG, "positions [%d, %d) outside the cache", pos0, pos0 + n_tokens);
+    for (int i = 0; i < n_tokens; ++i) if (tokens[i] < 0 || tokens[i] >= e->p.vocab_size) return fail(CUQWEN_ERR_ARG, "token %d out of range", tokens[i]);
+    return CUQWEN_OK;
+}
+
+// A portion of a sequence through a layer-list design, chunk by chunk; logits of the wanted rows (ascending) to the host.
+static int stack_portion(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0, const int* want, int n_want, float* logits) {
+    const int C = stack_chunk();
+    CK(cudaSetDevice(e->p.device));
+    t_err = reinterpret_cast<unsigned*>(&e->ctl->pad[0]);
+    if (!e->pf_tok) CK(cudaMalloc((void**)&e->pf_tok, (size_t)C * 4));
+    CK(cudaMemsetAsync(&e->ctl->pad[0], 0, 4, e->stream));
+    CK(cudaEventRecord(e->ev0, e->stream));
+    int w0 = 0;
+    std::vector<int> rows;
+    for (int c0 = 0; c0 < n_tokens; c0 += C) {
+        const int T = n_tokens - c0 < C ? n_tokens - c0 : C;
+        int w1 = w0;
+        rows.clear();
+        while (w1 < n_want && want[w1] < c0 + T) rows.push_back(want[w1++] - c0);
+        CK(cudaMemcpyAsync(e->pf_tok, tokens + c0, (size_t)T * 4, cudaMemcpyHostToDevice, e->stream));
+        if (int r = stack_run_chunk(e, T, pos0 + c0, rows.data(), (int)rows.size(), logits ? logits + (size_t)w0 * e->p.vocab_size : nullptr)) return r;
+        w0 = w1;
+    }
+    CK(cudaEventRecord(e->ev1, e->stream));
+    CK(cudaMemcpyAsync(e->h_out, &e->ctl->pad[0], 4, cudaMemcpyDeviceToHost, e->stream));
+    CK(cudaStreamSynchronize(e->stream));
+    if (e->h_out[0]) return fail(CUQWEN_ERR_TIMEOUT, "a bounded device-side wait expired (code %d)", e->h_out[0]);
+    CK(cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1));
+    return CUQWEN_OK;
+}
+
+extern "C" int cuqwen_extend(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0, const int* want, int n_want, float* logits) {
+    if (!e || !tokens || n_want < 0 || (n_want > 0 && (!want || !logits))) return fail(CUQWEN_ERR_ARG, "null argument");
+    if (!e->loaded) return fail(CUQWEN_ERR_STATE, "cuqwen_extend before the weights are loaded");
+    if (e->tp > 1) return fail(CUQWEN_ERR_ARG, "cuqwen_extend runs on one GPU (tp_size 1)");
+    if (int r = check_tokens(e, tokens, n_tokens, pos0)) return r;
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < 0 || want[i] >= n_tokens || (i && want[i] <= want[i - 1])) return fail(CUQWEN_ERR_ARG, "wanted places must ascend within the portion");
+    const size_t V = (size_t)e->p.vocab_size;
+    if (e->stack && n_tokens > 1) return stack_portion(e, tokens, n_tokens, pos0, want, n_want, logits);
+    // one token, and the models of the table: the decode step gives the logits of a wanted token, the batched prefill takes
+    // the tokens between the wanted ones
+    for (int i = 0, w = 0; i < n_tokens;) {
+        const int stop = w < n_want ? want[w] : n_tokens;
+        if (i < stop && (n_tokens > 1 || !e->stack) && !e->kv8) { if (int r = cuqwen_prefill(e, tokens + i, stop - i, pos0 + i)) return r; i = stop; continue; }
+        if (int r = cuqwen_step(e, tokens[i], pos0 + i, nullptr, 0, nullptr)) return r;
+        if (w < n_want && i == want[w]) {
+            float* out = logits + (size_t)w * V;
+            if (e->stack) CK(cudaMemcpyAsync(out, stack_logits(e->stack), V * 4, cudaMemcpyDeviceToHost, e->stream));
+            else {
+                std::vector<__half> h(V);
+                CK(cudaMemcpyAsync(h.data(), e->logits, V * 2, cudaMemcpyDeviceToHost, e->stream));
+                CK(cudaStreamSynchronize(e->stream));
+                for (size_t k = 0; k < V; ++k) out[k] = __half2float(h[k]);
+            }
+            CK(cudaStreamSynchronize(e->stream));
+            ++w;
+        }
+        ++i;
+    }
+    return CUQWEN_OK;
+}
+
 extern "C" int cuqwen_prefill(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0) {
     if (!e || !tokens) return fail(CUQWEN_ERR_ARG, "null argument");
     if (!e->loaded) return fail(CUQWEN_ERR_STATE, "cuqwen_prefill before cuqwen_load");
+    if (e->stack) { if (int r = check_tokens(e, tokens, n_tokens, pos0)) return r; return stack_portion(e, tokens, n_tokens, pos0, nullptr, 0, nullptr); }
     if (e->tp > 1) return fail(CUQWEN_ERR_ARG, "cuqwen_prefill runs on one GPU (tp_size 1); feed the prompt through cuqwen_step on tensor-parallel engines");
     if (e->kv8) return fail(CUQWEN_ERR_ARG, "cuqwen_prefill writes the fp16 KV cache; not available with CUQWEN_FLAG_KV_INT8");
     const cuqwen_params& p = e->p;
@@ -809,6 +885,7 @@ extern "C" int cuqwen_step_profile(cuqwen_engine* e, int token, int pos, float* 
 
 extern "C" int cuqwen_kv_fill_normal(cuqwen_engine* e, int ctx_len, uint64_t seed) {
     if (!e || ctx_len < 0 || ctx_len > e->p.max_seq_len) return fail(CUQWEN_ERR_ARG, "ctx_len out of range");
+    if (e->stack) return fail(CUQWEN_ERR_ARG, "cuqwen_kv_fill_normal fills the key / value cache of the models of the table");
     CK(cudaSetDevice(e->p.device));
     const cuqwen_params& p = e->p;
     LaunchCfg cfg{e->stream, e->sms, false};
@@ -905,6 +982,7 @@ extern "C" int cuqwen_get_params(const cuqwen_engine* e, cuqwen_params* out) { i
 extern "C" int cuqwen_step_launches(const cuqwen_engine* e) { return e ? e->launches : 0; }
 extern "C" uint64_t cuqwen_step_bytes(const cuqwen_engine* e, int ctx) {
     if (!e) return 0;
+    if (e->stack) return stack_step_bytes(e->stack, ctx);
     const uint64_t row = e->kv8 ? (uint64_t)e->p.head_dim + 4 : (uint64_t)e->p.head_dim * 2;       // one cached K or V row of one head (8-bit: + its scale)
     return e->weight_bytes + (uint64_t)2 * e->p.n_layers * e->n_kv_l * row * (uint64_t)ctx;
 }
@@ -913,6 +991,22 @@ extern "C" int cuqwen_get_ptr(cuqwen_engine* e, int which, int layer, void** ptr
     if (!e || !ptr) return fail(CUQWEN_ERR_ARG, "null argument");
     const cuqwen_params& p = e->p;
     void* r = nullptr; size_t b = 0;
+    if (e->stack) {
+        switch (which) {
+            case CUQWEN_PTR_X: stack_residual(e->stack, &r, &b); break;                       // float32
+            case CUQWEN_PTR_LOGITS: r = stack_logits(e->stack); b = (size_t)p.vocab_size * 4; break;      // float32
+            case CUQWEN_PTR_KEY_CACHE: b = stack_cache_bytes(e->stack, &r); break;             // every layer's latent rows
+            case CUQWEN_PTR_HISTORY: r = e->d_hist; b = (size_t)p.max_seq_len * 4; break;
+            case CUQWEN_PTR_TOKEN: r = &e->ctl->token; b = 4; break;
+            case CUQWEN_PTR_POS: r = &e->ctl->pos; b = 4; break;
+            case CUQWEN_PTR_HISTORY_LEN: r = &e->ctl->hist_len; b = 4; break;
+            case CUQWEN_PTR_SAMPLED: r = &e->ctl->sampled; b = 4; break;
+            case CUQWEN_PTR_STREAM: r = (void*)e->stream; break;
+            default: return fail(CUQWEN_ERR_ARG, "pointer id %d does not exist in a model opened from a directory", which);
+        }
+        *ptr = r; if (bytes) *bytes = b;
+        return CUQWEN_OK;
+    }
     auto matb = [&](const Mat& m, int quant) { return elem_bytes2(quant, m.rows, m.cols); };
     auto scb = [&](const Mat& m) { return (size_t)m.rows * (m.cols / kGroup) * 2; };
     if (which >= CUQWEN_PTR_IN_NORM) {

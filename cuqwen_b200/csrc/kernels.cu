@@ -108,7 +108,12 @@ int launch_kv_store(const __half* k, const __half* v, __half* kc, __half* vc, co
 // The reference visits the first min(hist_len, 4096) history entries and rescales once per
 // occurrence, racing on duplicates.  Here the first thread to set the id's bit in `bitmap`
 // applies the penalty, so every distinct id is penalised exactly once.
-__global__ void penalty_kernel(__half* logits, const int* __restrict__ hist, const int* __restrict__ d_hist_len,
+__device__ __forceinline__ float logit_f(__half v) { return __half2float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+__device__ __forceinline__ void set_logit(__half* p, float v) { *p = __float2half(v); }
+__device__ __forceinline__ void set_logit(float* p, float v) { *p = v; }
+template <typename L>
+__global__ void penalty_kernel(L* logits, const int* __restrict__ hist, const int* __restrict__ d_hist_len,
                                int vocab, int vocab_base, float pen, unsigned* bitmap) {
     pdl_launch_dependents(); pdl_wait();
     const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -117,8 +122,8 @@ __global__ void penalty_kernel(__half* logits, const int* __restrict__ hist, con
     if (id < 0 || id >= vocab) return;
     const unsigned bit = 1u << (id & 31);
     if (atomicOr(bitmap + (id >> 5), bit) & bit) return;
-    const float l = __half2float(logits[id]);
-    logits[id] = __float2half(l < 0.f ? l * pen : l / pen);
+    const float l = logit_f(logits[id]);
+    set_logit(logits + id, l < 0.f ? l * pen : l / pen);
 }
 __global__ void clear_bitmap_kernel(const int* __restrict__ hist, const int* __restrict__ d_hist_len, int vocab, int vocab_base, unsigned* bitmap) {
     pdl_launch_dependents(); pdl_wait();
@@ -128,7 +133,10 @@ __global__ void clear_bitmap_kernel(const int* __restrict__ hist, const int* __r
     if (id >= 0 && id < vocab) bitmap[id >> 5] = 0u;
 }
 int launch_penalty(__half* logits, const int* hist, const int* d_hist_len, int vocab, int vocab_base, float penalty, unsigned* bitmap, const LaunchCfg& cfg) {
-    return launch_k(penalty_kernel, dim3(16), dim3(256), 0, cfg, logits, hist, d_hist_len, vocab, vocab_base, penalty, bitmap);
+    return launch_k(penalty_kernel<__half>, dim3(16), dim3(256), 0, cfg, logits, hist, d_hist_len, vocab, vocab_base, penalty, bitmap);
+}
+int launch_penalty(float* logits, const int* hist, const int* d_hist_len, int vocab, int vocab_base, float penalty, unsigned* bitmap, const LaunchCfg& cfg) {
+    return launch_k(penalty_kernel<float>, dim3(16), dim3(256), 0, cfg, logits, hist, d_hist_len, vocab, vocab_base, penalty, bitmap);
 }
 int launch_clear_bitmap(const int* hist, const int* d_hist_len, int vocab, int vocab_base, unsigned* bitmap, const LaunchCfg& cfg) {
     return launch_k(clear_bitmap_kernel, dim3(16), dim3(256), 0, cfg, hist, d_hist_len, vocab, vocab_base, bitmap);
@@ -169,7 +177,8 @@ __device__ __forceinline__ unsigned long long key_word(unsigned long long packed
     return (hi << 32) | (nidx << 14) | (unsigned long long)((step + 1u) & 0x3fffu);
 }
 
-__global__ void argmax_kernel(const __half* __restrict__ logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap,
+template <typename L>
+__global__ void argmax_kernel(const L* __restrict__ logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap,
                               const int* __restrict__ hist, unsigned* bitmap, unsigned long long* best, unsigned* ticket,
                               unsigned long long* key_out, int* token_out, const KeyPush kp) {
     __shared__ unsigned long long sbest[8];
@@ -184,7 +193,7 @@ __global__ void argmax_kernel(const __half* __restrict__ logits, int vocab, int 
     }
     unsigned long long b = 0ull;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < vocab; i += gridDim.x * blockDim.x) {
-        unsigned long long p = argmax_pack(__half2float(logits[i]), i + vocab_base);
+        unsigned long long p = argmax_pack(logit_f(logits[i]), i + vocab_base);
         b = p > b ? p : b;
     }
 #pragma unroll
@@ -211,7 +220,8 @@ __global__ void argmax_kernel(const __half* __restrict__ logits, int vocab, int 
         }
     }
 }
-int launch_argmax(const __half* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap, const int* hist, unsigned* bitmap,
+template <typename L>
+static int go_argmax(const L* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap, const int* hist, unsigned* bitmap,
                   unsigned long long* best, unsigned* ticket, unsigned long long* key_out, int* token_out, const LaunchCfg& cfg,
                   unsigned long long* const* push_slots, int n_push) {
     int blocks = cfg.sm_count > 16 ? cfg.sm_count : 16;   // >= 16 blocks x 256 threads cover the 4096 history slots
@@ -221,7 +231,17 @@ int launch_argmax(const __half* logits, int vocab, int vocab_base, StepCtl* ctl,
         kp.n = n_push;
         for (int d = 0; d < n_push; ++d) kp.slot[d] = push_slots[d];
     }
-    return launch_k(argmax_kernel, dim3(blocks), dim3(256), 0, cfg, logits, vocab, vocab_base, ctl, out_ring, ring_cap, hist, bitmap, best, ticket, key_out, token_out, kp);
+    return launch_k(argmax_kernel<L>, dim3(blocks), dim3(256), 0, cfg, logits, vocab, vocab_base, ctl, out_ring, ring_cap, hist, bitmap, best, ticket, key_out, token_out, kp);
+}
+int launch_argmax(const __half* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap, const int* hist, unsigned* bitmap,
+                  unsigned long long* best, unsigned* ticket, unsigned long long* key_out, int* token_out, const LaunchCfg& cfg,
+                  unsigned long long* const* push_slots, int n_push) {
+    return go_argmax(logits, vocab, vocab_base, ctl, out_ring, ring_cap, hist, bitmap, best, ticket, key_out, token_out, cfg, push_slots, n_push);
+}
+int launch_argmax(const float* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap, const int* hist, unsigned* bitmap,
+                  unsigned long long* best, unsigned* ticket, unsigned long long* key_out, int* token_out, const LaunchCfg& cfg,
+                  unsigned long long* const* push_slots, int n_push) {
+    return go_argmax(logits, vocab, vocab_base, ctl, out_ring, ring_cap, hist, bitmap, best, ticket, key_out, token_out, cfg, push_slots, n_push);
 }
 // Tensor parallel: waits (bounded) until the n key words of this step have arrived in this rank's slots, takes their
 // maximum and finishes the step like the single-GPU sampler does.  One warp; lane r watches rank r's word.

@@ -1,0 +1,129 @@
+// Latent attention, any sizes, both activation types: one CTA per (head, query), an online softmax over tiles of 128 keys;
+// and the two matrix steps that let a decoded token attend to the latents directly.  The 32-bit mode's only path.
+#include "stack_dev.cuh"
+
+namespace cq {
+
+constexpr int kLaThreads = 128;
+
+template <typename A>
+__global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(const LatentAttnArgs a) {
+    extern __shared__ float la_smem[];                  // query [dn + dr], accumulators [dv], probabilities [128]
+    __shared__ float red[40];
+    float *q = la_smem, *acc = q + a.dn + a.dr, *pr = acc + a.dv;
+    pdl_launch_dependents(); pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x;
+    const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
+    const A* qn = reinterpret_cast<const A*>(a.qn) + (size_t)t * a.ldqn + (size_t)h * a.qn_hs;
+    const A* qr = reinterpret_cast<const A*>(a.qr) + (size_t)t * a.ldqr + (size_t)h * a.qr_hs;
+    for (int i = tid; i < a.dn; i += kLaThreads) q[i] = act_f(qn[i]);
+    for (int i = tid; i < a.dr; i += kLaThreads) q[a.dn + i] = act_f(qr[i]);
+    for (int i = tid; i < a.dv; i += kLaThreads) acc[i] = 0.f;
+    const int lo = a.window > 0 && pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
+    float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f;       // the sink is a key without a value, unscaled
+    for (int k0 = lo; k0 <= pos; k0 += kLaThreads) {
+        __syncthreads();
+        const int k = k0 + tid;
+        float s = -INFINITY;
+        if (k <= pos) {
+            const A* kn = reinterpret_cast<const A*>(a.kn) + (size_t)(k - a.kbase) * a.ldkn + (size_t)h * a.kn_hs;
+            const A* kr = reinterpret_cast<const A*>(a.kr) + (size_t)k * a.ldkr;
+            float d = 0.f;
+            for (int i = 0; i < a.dn; ++i) d = fmaf(q[i], act_f(kn[i]), d);
+            for (int i = 0; i < a.dr; ++i) d = fmaf(q[a.dn + i], act_f(kr[i]), d);
+            s = d * a.scale;
+        }
+        float mx = s;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        if ((tid & 31) == 0) red[tid >> 5] = mx;
+        __syncthreads();
+        mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+        const float mn = fmaxf(m, mx);                   // finite: key k0 is visible
+        const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
+        m = mn;
+        const float p = k <= pos ? expf(s - mn) : 0.f;
+        pr[tid] = p;
+        l = l * alpha + cta_sum(p, red);                 // barriers inside: pr is complete
+        const int n = pos - k0 + 1 < kLaThreads ? pos - k0 + 1 : kLaThreads;
+        for (int c = tid; c < a.dv; c += kLaThreads) {
+            const A* v = reinterpret_cast<const A*>(a.v) + (size_t)(k0 - a.kbase) * a.ldv + (size_t)h * a.v_hs + c;
+            float o = acc[c] * alpha;
+            for (int j = 0; j < n; ++j) o = fmaf(pr[j], act_f(v[(size_t)j * a.ldv]), o);
+            acc[c] = o;
+        }
+    }
+    const float inv = 1.0f / l;
+    for (int c = tid; c < a.dv; c += kLaThreads) {
+        float o = acc[c] * inv;
+        if (a.gate) o *= sigmoid_f(a.gate[(size_t)t * a.ldg + (size_t)h * a.g_hs + c]);
+        const size_t i = (size_t)t * a.ldo + (size_t)h * a.o_hs + c;
+        if (a.out_f32) reinterpret_cast<float*>(a.out)[i] = o;
+        else reinterpret_cast<A*>(a.out)[i] = to_act<A>(o);
+    }
+}
+int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg) {
+    const size_t smem = (size_t)(a.dn + a.dr + a.dv + kLaThreads) * 4;
+    if (a.T < 1 || a.heads < 1 || smem > 40 * 1024) return (int)cudaErrorInvalidValue;
+    const dim3 grid(a.heads, a.T);
+    return act == ACT_F32 ? st_launch(latent_attn_kernel<float>, grid, dim3(kLaThreads), smem, cfg, a) : st_launch(latent_attn_kernel<bf16>, grid, dim3(kLaThreads), smem, cfg, a);
+}
+
+// CTA = one head, 256 latent columns: thread (c, part) walks a quarter of the head's rows of W_uk for eight columns.
+template <typename A>
+__global__ void __launch_bounds__(128) absorb_q_kernel(const AbsorbArgs a) {
+    __shared__ float part[3][256];
+    pdl_launch_dependents(); pdl_wait();
+    const int h = blockIdx.x, c0 = blockIdx.y * 256 + (threadIdx.x & 31) * 8, grp = threadIdx.x >> 5;
+    const A* q = reinterpret_cast<const A*>(a.q) + (size_t)h * a.q_hs;
+    const bf16* w = a.wk + (size_t)h * a.dimp * a.pitch + c0;
+    float s[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (c0 < a.ldo)                                      // ldo = the padded latent size, a multiple of eight within the pitch
+#pragma unroll 4
+        for (int d = grp; d < a.dim; d += 4) {
+            float v[8];
+            load8(w + (size_t)d * a.pitch, v);
+            const float qd = act_f(q[d]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s[i] = fmaf(qd, v[i], s[i]);
+        }
+    if (grp > 0)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) part[grp - 1][(threadIdx.x & 31) * 8 + i] = s[i];
+    __syncthreads();
+    if (grp == 0 && c0 < a.ldo) {
+        A* o = reinterpret_cast<A*>(a.out) + (size_t)h * a.ldo + c0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int j = threadIdx.x * 8 + i;
+            o[i] = to_act<A>(s[i] + part[0][j] + part[1][j] + part[2][j]);
+        }
+    }
+}
+int launch_absorb_q(int act, const AbsorbArgs& a, const LaunchCfg& cfg) {
+    const dim3 grid(a.heads, (a.ldo + 255) / 256);
+    return act == ACT_F32 ? st_launch(absorb_q_kernel<float>, grid, dim3(128), 0, cfg, a) : st_launch(absorb_q_kernel<bf16>, grid, dim3(128), 0, cfg, a);
+}
+
+// A warp per output value.
+template <typename A>
+__global__ void __launch_bounds__(256) uv_gate_kernel(const UvGateArgs a) {
+    pdl_launch_dependents(); pdl_wait();
+    const int h = blockIdx.x, v = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (v >= a.vdim) return;
+    const float* o = a.o + (size_t)h * a.ldo;
+    const bf16* w = a.wv + (size_t)(h * a.vdimp + v) * a.pitch;
+    float s = 0.f;
+    for (int r = lane; r < a.kv_rank; r += 32) s = fmaf(o[r], __bfloat162float(w[r]), s);
+    s = warp_sum(s);
+    if (lane == 0) {
+        if (a.gate) s *= sigmoid_f(a.gate[(size_t)h * a.g_hs + v]);
+        reinterpret_cast<A*>(a.out)[(size_t)h * a.o_hs + v] = to_act<A>(s);
+    }
+}
+int launch_uv_gate(int act, const UvGateArgs& a, const LaunchCfg& cfg) {
+    const dim3 grid(a.heads, (a.vdim + 7) / 8);
+    return act == ACT_F32 ? st_launch(uv_gate_kernel<float>, grid, dim3(256), 0, cfg, a) : st_launch(uv_gate_kernel<bf16>, grid, dim3(256), 0, cfg, a);
+}
+
+}  // namespace cq

@@ -66,6 +66,7 @@ int launch_kv_store(const __half* k, const __half* v, __half* kc, __half* vc, co
 // Repetition penalty, once per distinct id among the first min(hist_len, 4096) entries.
 // `bitmap` holds ceil(vocab/32) zeroed words; the sampler (or clear_bitmap) zeroes it again.
 int launch_penalty(__half* logits, const int* hist, const int* d_hist_len, int vocab, int vocab_base, float penalty, unsigned* bitmap, const LaunchCfg& cfg);
+int launch_penalty(float* logits, const int* hist, const int* d_hist_len, int vocab, int vocab_base, float penalty, unsigned* bitmap, const LaunchCfg& cfg);
 int launch_clear_bitmap(const int* hist, const int* d_hist_len, int vocab, int vocab_base, unsigned* bitmap, const LaunchCfg& cfg);
 // Greedy sampler.  best/ticket: one u64 and one u32 of zeroed scratch.  Writes ctl->sampled and, when
 // ctl->auto_advance is set, feeds the token back (token, pos+1, out_ring).  When key_out is non-null the packed
@@ -73,6 +74,10 @@ int launch_clear_bitmap(const int* hist, const int* d_hist_len, int vocab, int v
 // push_slots / n_push (tensor parallel without a collective call): the packed key, tagged with the step's number, is
 // stored into one 64-bit word per rank instead (kernels.cu: KeyPush); launch_merge_pushed_keys reads them.
 int launch_argmax(const __half* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap,
+                  const int* hist, unsigned* bitmap, unsigned long long* best, unsigned* ticket,
+                  unsigned long long* key_out, int* token_out, const LaunchCfg& cfg,
+                  unsigned long long* const* push_slots = nullptr, int n_push = 0);
+int launch_argmax(const float* logits, int vocab, int vocab_base, StepCtl* ctl, int* out_ring, int ring_cap,
                   const int* hist, unsigned* bitmap, unsigned long long* best, unsigned* ticket,
                   unsigned long long* key_out, int* token_out, const LaunchCfg& cfg,
                   unsigned long long* const* push_slots = nullptr, int n_push = 0);

@@ -1,0 +1,417 @@
+// Host side of the layer-list designs: weights from a model directory, the latent cache, and the launch sequences of a
+// decode step and of a prompt portion.  Kernels: stack.h.
+//
+// Layout.  Every per-head or per-part length is padded to a multiple of eight with zero weight rows / columns when the
+// weights are loaded, so that rows start on 16-byte boundaries and padded places hold zeros; weight rows are padded to a
+// multiple of 128 columns.  For the usual sizes nothing is added.
+//   q            [heads][dim | rot_dim]
+//   cache row    [latent kv_rank | rotated key part rot_dim], one array [max_seq_len][row] per layer with a projection of its own
+//   raw          [query latent q_rank | cache row | gate heads * vdim], float32 sums of the first launch of a layer
+#include "stack.h"
+
+#include <cmath>
+#include <cstring>
+#include <string>
+
+#include "stack_host.h"
+
+namespace cq {
+
+namespace {
+
+int pad8(int v) { return (v + 7) / 8 * 8; }
+constexpr int kChunk = 2048;                // tokens of a portion that go through the layers together
+constexpr int kLogitRows = 64;              // rows of logits computed at a time
+
+struct StMat { bf16* w = nullptr; int rows = 0, cols = 0, pitch = 0; };     // rows with padding, cols with padding of groups
+
+struct StLayer {
+    LatentAttnSpec a;
+    int ff = 0;
+    int dimp = 0, rotp = 0, vdimp = 0, kvrp = 0, qrp = 0, crow = 0, head_q = 0;
+    int cache = -1, rot = -1;
+    StMat dq, uq, dkv, uk, uv, g, o, up, down, side_gate, side_proj;
+    float *norm1 = nullptr, *norm2 = nullptr, *dq_norm = nullptr, *dkv_norm = nullptr, *sink = nullptr, *side_norm = nullptr;
+};
+
+struct Arena2 {
+    uint8_t* base = nullptr; size_t used = 0; bool dry = true;
+    void* get(size_t bytes) { const size_t o = used; used += (bytes + 255) / 256 * 256; return dry ? nullptr : base + o; }
+};
+
+}  // namespace
+
+struct Stack {
+    StackSpec spec;
+    int act = ACT_BF16, esz = 2, max_seq = 0, vocab_p = 0, wp = 0, sidep = 0;
+    std::vector<StLayer> layers;
+    StMat embed, side_embed, head;
+    float* final_norm = nullptr;
+    uint8_t* arena = nullptr;
+    uint64_t weight_bytes = 0;
+    // cache and rotation tables
+    uint8_t* cache = nullptr; size_t cache_bytes = 0; std::vector<size_t> cache_off;
+    std::vector<RotarySpec> rots; std::vector<float2*> rot_tables;
+    // workspace: a decode step's (one row), and a portion's (kChunk rows; allocated at first use)
+    struct Ws {
+        int rows = 0, kv_rows = 0;
+        float *x = nullptr, *raw = nullptr, *qf = nullptr, *y = nullptr, *o_lat = nullptr;
+        void *xn1 = nullptr, *xn2 = nullptr, *cq = nullptr, *q = nullptr, *q_abs = nullptr, *att = nullptr, *h = nullptr, *sg = nullptr, *k = nullptr, *v = nullptr;
+        uint8_t* arena = nullptr;
+    } dec, pf;
+    float* logits = nullptr;            // decode step
+    float* logits_rows = nullptr; void* xn_rows = nullptr; int* want_rows = nullptr;
+    int max_raw = 0, max_q = 0, max_att = 0, max_ff = 0, max_qr = 0, max_kn = 0, max_kvr = 0;
+};
+
+#define SK(call) do { cudaError_t e_ = (cudaError_t)(call); if (e_ != cudaSuccess) return report_error(e_ == cudaErrorInvalidValue ? CUQWEN_ERR_ARG : CUQWEN_ERR_CUDA, "%s: %s (%s:%d)", #call, cudaGetErrorString(e_), __FILE__, __LINE__); } while (0)
+
+const StackSpec& stack_spec(const Stack* s) { return s->spec; }
+int stack_act(const Stack* s) { return s->act; }
+float* stack_logits(const Stack* s) { return s->logits; }
+size_t stack_cache_bytes(const Stack* s, void** ptr) { *ptr = s->cache; return s->cache_bytes; }
+void stack_residual(const Stack* s, void** ptr, size_t* bytes) { *ptr = s->dec.x; *bytes = (size_t)s->spec.width * 4; }
+int stack_chunk() { return kChunk; }
+
+static int alloc_ws(Stack* s, Stack::Ws* w, int rows, bool decode) {
+    Arena2 dry, real;
+    for (int pass = 0; pass < 2; ++pass) {
+        Arena2& a = pass ? real : dry;
+        const size_t R = (size_t)rows, E = (size_t)s->esz;
+        w->x = (float*)a.get(R * s->wp * 4);
+        w->raw = (float*)a.get(R * s->max_raw * 4);
+        w->qf = (float*)a.get(R * s->max_q * 4);
+        w->y = (float*)a.get(R * s->wp * 4);
+        w->xn1 = a.get(R * s->wp * E); w->xn2 = a.get(R * s->wp * E);
+        w->cq = a.get(R * s->max_qr * E); w->q = a.get(R * s->max_q * E);
+        w->att = a.get(R * s->max_att * E); w->h = a.get(R * (s->max_ff ? s->max_ff : 8) * E);
+        w->sg = a.get(R * (s->sidep ? s->sidep : 8) * E);
+        if (decode) {
+            w->q_abs = a.get((size_t)s->max_kvr * E);
+            w->o_lat = (float*)a.get((size_t)s->max_kvr * 4);
+        } else {
+            // keys and values of everything a portion's queries can reach: the portion and the widest window before it
+            int reach = 0;
+            for (const StLayer& l : s->layers) { const int r = l.a.window > 0 && l.a.window < s->max_seq ? l.a.window - 1 : s->max_seq; reach = r > reach ? r : reach; }
+            w->kv_rows = rows + reach < s->max_seq ? rows + reach : s->max_seq;
+            w->k = a.get((size_t)w->kv_rows * s->max_kn * E); w->v = a.get((size_t)w->kv_rows * s->max_att * E);
+        }
+        if (!pass) {
+            SK(cudaMalloc((void**)&w->arena, dry.used + 256));
+            SK(cudaMemset(w->arena, 0, dry.used + 256));
+            real.base = w->arena; real.dry = false;
+        }
+    }
+    w->rows = rows;
+    return CUQWEN_OK;
+}
+
+int stack_create(cuqwen_engine* e, const StackSpec& spec, int act, int max_seq_len) {
+    Stack* s = e->stack = new Stack();
+    s->spec = spec; s->act = act; s->esz = act == ACT_F32 ? 4 : 2; s->max_seq = max_seq_len;
+    s->wp = pad8(spec.width); s->sidep = pad8(spec.side_dim); s->vocab_p = pad8(spec.vocab);
+    if (!spec.side_dim) s->sidep = 0;
+    size_t coff = 0;
+    for (const LayerSpec& L : spec.layers) {
+        StLayer l;
+        l.a = L.attn; l.ff = L.mlp.ff;
+        l.dimp = pad8(l.a.dim); l.rotp = pad8(l.a.rot_dim); l.vdimp = pad8(l.a.vdim); l.kvrp = pad8(l.a.kv_rank); l.qrp = pad8(l.a.q_rank);
+        l.crow = l.kvrp + l.rotp; l.head_q = l.dimp + l.rotp;
+        for (size_t i = 0; i < s->rots.size(); ++i) if (s->rots[i].dims == l.a.rot.dims && s->rots[i].base == l.a.rot.base) l.rot = (int)i;
+        if (l.rot < 0) { l.rot = (int)s->rots.size(); s->rots.push_back(l.a.rot); }
+        if (l.a.kv_from < 0) {
+            l.cache = (int)s->cache_off.size();
+            s->cache_off.push_back(coff);
+            coff += ((size_t)max_seq_len * l.crow * s->esz + 255) / 256 * 256;
+        } else l.cache = s->layers[l.a.kv_from].cache;
+        auto up = [](int& m, int v) { if (v > m) m = v; };
+        up(s->max_raw, l.qrp + (l.a.kv_from < 0 ? l.crow : 0) + l.a.heads * l.vdimp); up(s->max_q, l.a.heads * l.head_q); up(s->max_att, l.a.heads * l.vdimp);
+        up(s->max_ff, pad8(l.ff)); up(s->max_qr, l.qrp); up(s->max_kn, l.a.heads * l.dimp); up(s->max_kvr, l.a.heads * l.kvrp);
+        s->layers.push_back(l);
+    }
+    s->cache_bytes = coff;
+    SK(cudaMalloc((void**)&s->cache, coff + 256));
+    SK(cudaMemset(s->cache, 0, coff + 256));
+    for (const RotarySpec& r : s->rots) {
+        float2* t = nullptr;
+        SK(cudaMalloc((void**)&t, (size_t)max_seq_len * (r.dims / 2) * sizeof(float2)));
+        s->rot_tables.push_back(t);
+        SK(launch_rot_table(t, max_seq_len, r.dims, r.base, LaunchCfg{e->stream, e->sms, false}));
+    }
+    if (int r = alloc_ws(s, &s->dec, 1, true)) return r;
+    SK(cudaMalloc((void**)&s->logits, (size_t)s->vocab_p * 4)); SK(cudaMemset(s->logits, 0, (size_t)s->vocab_p * 4));
+    e->p.model_id = CUQWEN_MODEL_CUSTOM; e->p.vocab_size = spec.vocab; e->p.dim = spec.width; e->p.n_layers = (int)spec.layers.size();
+    e->p.n_heads = spec.layers[0].attn.heads; e->p.n_kv_heads = 1; e->p.head_dim = spec.layers[0].attn.dim + spec.layers[0].attn.rot_dim;
+    e->p.intermediate_size = spec.layers[0].mlp.ff; e->p.norm_eps = (float)spec.norm_eps; e->p.rope_theta = (float)spec.layers[0].attn.rot.base;
+    e->vocab_l = spec.vocab;
+    SK(cudaStreamSynchronize(e->stream));
+    return CUQWEN_OK;
+}
+
+void stack_destroy(cuqwen_engine* e) {
+    Stack* s = e->stack;
+    if (!s) return;
+    void* bufs[] = {s->arena, s->cache, s->dec.arena, s->pf.arena, s->logits, s->logits_rows, s->xn_rows, s->want_rows};
+    for (void* b : bufs) if (b) cudaFree(b);
+    for (float2* t : s->rot_tables) cudaFree(t);
+    delete s;
+    e->stack = nullptr;
+}
+
+// ---- weights --------------------------------------------------------------------------------------------------------
+// Lengths of consecutive groups of rows (or columns) and the places they take: group i of `len` elements starts at `at`.
+struct Groups {
+    std::vector<std::pair<int, int>> g;       // (length, start of its padded place)
+    int total = 0, padded = 0;
+    Groups& add(int len) { g.emplace_back(len, padded); total += len; padded += pad8(len); return *this; }
+    static Groups one(int len) { return Groups().add(len); }
+    static Groups heads(int n, int a, int b = 0) { Groups r; for (int i = 0; i < n; ++i) { r.add(a); if (b) r.add(b); } return r; }
+};
+
+static int put_matrix(const Safetensors& st, Stack* s, Arena2& ar, const std::string& name, const Groups& rows, const Groups& cols, StMat* m, bool counted = true) {
+    const Safetensors::Tensor* t = st.expect(name, rows.total, cols.total);
+    if (!t) return CUQWEN_ERR_DIMS;
+    m->rows = rows.padded; m->cols = cols.padded; m->pitch = (cols.padded + 127) / 128 * 128;
+    const size_t bytes = (size_t)m->rows * m->pitch * 2;
+    m->w = (bf16*)ar.get(bytes);
+    if (counted && ar.dry) s->weight_bytes += (uint64_t)rows.total * cols.total * 2;
+    if (ar.dry) return CUQWEN_OK;
+    if (rows.padded == rows.total && m->pitch == cols.total) { SK(cudaMemcpy(m->w, t->data, bytes, cudaMemcpyHostToDevice)); return CUQWEN_OK; }
+    std::vector<uint16_t> host((size_t)m->rows * m->pitch, 0);
+    size_t src_row = 0;
+    for (const auto& rg : rows.g)
+        for (int r = 0; r < rg.first; ++r, ++src_row) {
+            const uint8_t* src = t->data + src_row * cols.total * 2;
+            uint16_t* dst = host.data() + (size_t)(rg.second + r) * m->pitch;
+            for (const auto& cg : cols.g) { memcpy(dst + cg.second, src, (size_t)cg.first * 2); src += (size_t)cg.first * 2; }
+        }
+    SK(cudaMemcpy(m->w, host.data(), bytes, cudaMemcpyHostToDevice));
+    return CUQWEN_OK;
+}
+static int put_vector(const Safetensors& st, Stack* s, Arena2& ar, const std::string& name, int n, float** v) {
+    const Safetensors::Tensor* t = st.expect(name, n, 0);
+    if (!t) return CUQWEN_ERR_DIMS;
+    *v = (float*)ar.get((size_t)pad8(n) * 4);
+    if (ar.dry) { s->weight_bytes += (uint64_t)n * 2; return CUQWEN_OK; }
+    std::vector<float> host(pad8(n), 0.f);
+    for (int i = 0; i < n; ++i) { uint16_t h; memcpy(&h, t->data + 2 * (size_t)i, 2); const uint32_t u = (uint32_t)h << 16; memcpy(&host[i], &u, 4); }
+    SK(cudaMemcpy(*v, host.data(), host.size() * 4, cudaMemcpyHostToDevice));
+    return CUQWEN_OK;
+}
+
+static int walk_tensors(const Safetensors& st, Stack* s, Arena2& ar) {
+#define TRY(x) do { if (int r_ = (x)) return r_; } while (0)
+    const StackSpec& sp = s->spec;
+    const Groups W = Groups::one(sp.width);
+    TRY(put_matrix(st, s, ar, "embed", Groups::one(sp.vocab), W, &s->embed, false));
+    if (sp.side_dim) TRY(put_matrix(st, s, ar, "side.embed", Groups::one(sp.vocab), Groups::one(sp.side_dim * (int)sp.layers.size()), &s->side_embed, false));
+    for (size_t i = 0; i < s->layers.size(); ++i) {
+        StLayer& l = s->layers[i];
+        const LatentAttnSpec& a = l.a;
+        const std::string p = "l" + std::to_string(i) + ".", mix = p + "mix.";
+        TRY(put_vector(st, s, ar, p + "norm1", sp.width, &l.norm1));
+        TRY(put_matrix(st, s, ar, mix + "dq", Groups::one(a.q_rank), W, &l.dq));
+        TRY(put_vector(st, s, ar, mix + "dq.norm", a.q_rank, &l.dq_norm));
+        TRY(put_matrix(st, s, ar, mix + "uq", Groups::heads(a.heads, a.dim, a.rot_dim), Groups::one(a.q_rank), &l.uq));
+        if (a.kv_from < 0) {
+            TRY(put_matrix(st, s, ar, mix + "dkv", Groups::heads(1, a.kv_rank, a.rot_dim), W, &l.dkv));
+            TRY(put_vector(st, s, ar, mix + "dkv.norm", a.kv_rank, &l.dkv_norm));
+        }
+        TRY(put_matrix(st, s, ar, mix + "uk", Groups::heads(a.heads, a.dim), Groups::one(a.kv_rank), &l.uk));
+        TRY(put_matrix(st, s, ar, mix + "uv", Groups::heads(a.heads, a.vdim), Groups::one(a.kv_rank), &l.uv));
+        if (a.sink) TRY(put_vector(st, s, ar, mix + "sink", a.heads, &l.sink));
+        if (a.gate) TRY(put_matrix(st, s, ar, mix + "g", Groups::heads(a.heads, a.vdim), W, &l.g));
+        TRY(put_matrix(st, s, ar, mix + "o", W, Groups::heads(a.heads, a.vdim), &l.o));
+        if (l.ff) {
+            TRY(put_vector(st, s, ar, p + "norm2", sp.width, &l.norm2));
+            TRY(put_matrix(st, s, ar, p + "mlp.up", Groups::one(l.ff), W, &l.up));
+            TRY(put_matrix(st, s, ar, p + "mlp.down", W, Groups::one(l.ff), &l.down));
+        }
+        if (sp.side_dim) {
+            TRY(put_matrix(st, s, ar, p + "side.gate", Groups::one(sp.side_dim), W, &l.side_gate));
+            TRY(put_matrix(st, s, ar, p + "side.proj", W, Groups::one(sp.side_dim), &l.side_proj));
+            TRY(put_vector(st, s, ar, p + "side.norm", sp.width, &l.side_norm));
+        }
+    }
+    TRY(put_vector(st, s, ar, "final.norm", sp.width, &s->final_norm));
+    TRY(put_matrix(st, s, ar, "head", Groups::one(sp.vocab), W, &s->head));
+#undef TRY
+    return CUQWEN_OK;
+}
+
+int stack_load(cuqwen_engine* e, const char* dir) {
+    Stack* s = e->stack;
+    Safetensors st;
+    if (int r = st.open((std::string(dir) + "/model.safetensors").c_str())) return r;
+    Arena2 dry, real;
+    s->weight_bytes = (uint64_t)(s->spec.width + s->spec.side_dim * (int)s->layers.size()) * 2;      // a token's embedding rows
+    if (int r = walk_tensors(st, s, dry)) return r;
+    SK(cudaMalloc((void**)&s->arena, dry.used + 256));
+    real.base = s->arena; real.dry = false;
+    if (int r = walk_tensors(st, s, real)) return r;
+    SK(cudaDeviceSynchronize());
+    return CUQWEN_OK;
+}
+
+uint64_t stack_step_bytes(const Stack* s, int ctx) {
+    uint64_t b = s->weight_bytes;
+    for (const StLayer& l : s->layers) {
+        const int n = l.a.window > 0 && l.a.window < ctx ? l.a.window : ctx;
+        b += (uint64_t)n * (l.a.kv_rank + l.a.rot_dim) * s->esz;
+    }
+    return b;
+}
+
+// ---- launch sequences -------------------------------------------------------------------------------------------------
+namespace {
+
+// One pass over the layers for T rows.  decode: T = 1, token and position from the control block, attention over latents.
+struct Pass {
+    cuqwen_engine* e; Stack* s; Stack::Ws* w; LaunchCfg cfg;
+    int T; bool decode; const int* tokens; const int* pos_ptr; int pos0;
+    const std::function<int()>* after;
+
+    int done(int err, const char* what) {
+        if (err) return report_error(err == (int)cudaErrorInvalidValue ? CUQWEN_ERR_ARG : CUQWEN_ERR_CUDA, "%s: %s", what, cudaGetErrorString((cudaError_t)err));
+        return after ? (*after)() : CUQWEN_OK;
+    }
+#define GO(call) do { if (int r_ = done(call, #call)) return r_; } while (0)
+    LinArgs lin(const void* x, int ldx, const StMat& m, int epi, void* out, int ldo) {
+        LinArgs a{};
+        a.x = x; a.ldx = ldx; a.w = m.w; a.pitch = m.pitch; a.K = m.cols; a.T = T; a.R = m.rows; a.epi = epi; a.out = out; a.ldo = ldo;
+        return a;
+    }
+    int norms(const float* y, const float* y_w, const float* w1, const float* w2) {
+        NormRowsArgs n{};
+        n.x = w->x; n.ldx = s->wp; n.y = y; n.ldy = s->wp; n.y_w = y_w; n.width = s->spec.width; n.eps = (float)s->spec.norm_eps; n.ldo = s->wp;
+        if (w1) { n.w[n.n_out] = w1; n.out[n.n_out++] = w->xn1; }
+        if (w2) { n.w[n.n_out] = w2; n.out[n.n_out++] = w->xn2; }
+        GO(launch_st_norms(s->act, n, T, cfg));
+        return CUQWEN_OK;
+    }
+    uint8_t* cache_of(const StLayer& l) { return s->cache + s->cache_off[l.cache]; }
+
+    int attention(const StLayer& l, const float* gate, int ldraw) {
+        const LatentAttnSpec& a = l.a;
+        LatentAttnArgs t{};
+        t.qr = (uint8_t*)w->q + (size_t)l.dimp * s->esz; t.ldqr = a.heads * l.head_q; t.qr_hs = l.head_q; t.dr = a.rot_dim;
+        uint8_t* c = cache_of(l);
+        t.kr = c + (size_t)l.kvrp * s->esz; t.ldkr = l.crow;
+        t.sink = l.sink; t.T = T; t.heads = a.heads; t.window = a.window; t.scale = (float)a.scale; t.pos_ptr = pos_ptr; t.pos0 = pos0;
+        if (decode) {
+            AbsorbArgs b{};
+            b.q = w->q; b.q_hs = l.head_q; b.wk = l.uk.w; b.pitch = l.uk.pitch; b.heads = a.heads; b.dim = a.dim; b.dimp = l.dimp; b.kv_rank = a.kv_rank; b.out = w->q_abs; b.ldo = l.kvrp;
+            GO(launch_absorb_q(s->act, b, cfg));
+            t.qn = w->q_abs; t.ldqn = a.heads * l.kvrp; t.qn_hs = l.kvrp; t.dn = a.kv_rank;
+            t.kn = c; t.ldkn = l.crow; t.kn_hs = 0; t.v = c; t.ldv = l.crow; t.v_hs = 0; t.dv = a.kv_rank;
+            t.out = w->o_lat; t.out_f32 = 1; t.ldo = a.heads * l.kvrp; t.o_hs = l.kvrp;
+            GO(launch_latent_attn(s->act, t, cfg));
+            UvGateArgs u{};
+            u.o = w->o_lat; u.ldo = l.kvrp; u.wv = l.uv.w; u.pitch = l.uv.pitch; u.heads = a.heads; u.vdim = a.vdim; u.vdimp = l.vdimp; u.kv_rank = a.kv_rank;
+            u.gate = gate; u.g_hs = l.vdimp; u.out = w->att; u.o_hs = l.vdimp;
+            GO(launch_uv_gate(s->act, u, cfg));
+            return CUQWEN_OK;
+        }
+        // keys and values of every token the portion's queries reach
+        const int k0 = a.window > 0 && pos0 - a.window + 1 > 0 ? pos0 - a.window + 1 : 0, n = pos0 + T - k0;
+        LinArgs k = lin(c + (size_t)k0 * l.crow * s->esz, l.crow, l.uk, LIN_ACT, w->k, a.heads * l.dimp);
+        LinArgs v = lin(c + (size_t)k0 * l.crow * s->esz, l.crow, l.uv, LIN_ACT, w->v, a.heads * l.vdimp);
+        k.T = v.T = n;
+        GO(launch_st_linear(s->act, k, cfg));
+        GO(launch_st_linear(s->act, v, cfg));
+        t.qn = w->q; t.ldqn = a.heads * l.head_q; t.qn_hs = l.head_q; t.dn = a.dim;
+        t.kn = w->k; t.ldkn = a.heads * l.dimp; t.kn_hs = l.dimp; t.v = w->v; t.ldv = a.heads * l.vdimp; t.v_hs = l.vdimp; t.dv = a.vdim; t.kbase = k0;
+        t.gate = gate; t.ldg = ldraw; t.g_hs = l.vdimp; t.out = w->att; t.ldo = a.heads * l.vdimp; t.o_hs = l.vdimp;
+        GO(launch_latent_attn(s->act, t, cfg));
+        return CUQWEN_OK;
+    }
+
+    // All layers.  cache_only: nothing after the last layer's cache rows is needed.  Leaves the residual stream in w->x with
+    // the last layer's token input still to be added (w->y, side_norm of the last layer).
+    int layers(bool cache_only) {
+        const StackSpec& sp = s->spec;
+        const float* y = nullptr; const float* y_w = nullptr;
+        for (size_t i = 0; i < s->layers.size(); ++i) {
+            const StLayer& l = s->layers[i];
+            const LatentAttnSpec& a = l.a;
+            const bool own = a.kv_from < 0, stop = cache_only && i + 1 == s->layers.size();
+            if (stop && !own) return CUQWEN_OK;
+            if (int r = norms(y, y_w, l.norm1, l.ff && !stop ? l.norm2 : nullptr)) return r;
+            const int c_off = l.qrp, g_off = c_off + (own ? l.crow : 0), ldraw = g_off + a.heads * l.vdimp;
+            if (!stop) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.dq, LIN_F32, w->raw, ldraw), cfg));
+            if (own) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.dkv, LIN_F32, w->raw + c_off, ldraw), cfg));
+            if (a.gate && !stop) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.g, LIN_F32, w->raw + g_off, ldraw), cfg));
+            if (l.ff && !stop) GO(launch_st_linear(s->act, lin(w->xn2, s->wp, l.up, LIN_RELU2, w->h, l.up.rows), cfg));
+            LatentRowsArgs lr{};
+            lr.dq = w->raw; lr.ld = ldraw; lr.dq_w = l.dq_norm; lr.cq = w->cq; lr.ldcq = l.qrp; lr.q_rank = a.q_rank;
+            if (own) { lr.dkv = w->raw + c_off; lr.dkv_w = l.dkv_norm; lr.cache = cache_of(l); lr.ldc = l.crow; lr.kv_rank = a.kv_rank; lr.kr_off = l.kvrp; lr.rot_dim = a.rot_dim; lr.rot = s->rot_tables[l.rot]; }
+            lr.eps = (float)sp.norm_eps; lr.pos_ptr = pos_ptr; lr.pos0 = pos0;
+            GO(launch_st_latent_rows(s->act, lr, T, cfg));
+            if (stop) return CUQWEN_OK;
+            GO(launch_st_linear(s->act, lin(w->cq, l.qrp, l.uq, LIN_F32, w->qf, l.uq.rows), cfg));
+            RopeQArgs rq{w->qf, w->q, l.uq.rows, a.heads, l.head_q, l.dimp, a.rot_dim, s->rot_tables[l.rot], pos_ptr, pos0};
+            GO(launch_st_rope_q(s->act, rq, T, cfg));
+            if (int r = attention(l, a.gate ? w->raw + g_off : nullptr, ldraw)) return r;
+            LinArgs o = lin(w->att, a.heads * l.vdimp, l.o, LIN_ADD, w->x, s->wp);
+            if (l.ff) { o.x2 = w->h; o.ldx2 = l.up.rows; o.w2 = l.down.w; o.pitch2 = l.down.pitch; o.K2 = l.down.cols; }
+            GO(launch_st_linear(s->act, o, cfg));
+            if (sp.side_dim) {
+                // the token input reads the stream itself, narrowed like every activation
+                if (int r = narrow_x()) return r;
+                LinArgs g = lin(w->xn1, s->wp, l.side_gate, LIN_GELU_SIDE, w->sg, s->sidep);
+                g.side = s->side_embed.w + i * sp.side_dim; g.side_pitch = s->side_embed.pitch; g.side_dim = sp.side_dim; g.tokens = tokens;
+                GO(launch_st_linear(s->act, g, cfg));
+                GO(launch_st_linear(s->act, lin(w->sg, s->sidep, l.side_proj, LIN_F32, w->y, s->wp), cfg));
+                y = w->y; y_w = l.side_norm;
+            }
+        }
+        return CUQWEN_OK;
+    }
+    int narrow_x() { GO(launch_st_narrow(s->act, w->x, s->wp, w->xn1, s->wp, T, cfg)); return CUQWEN_OK; }
+    const float* last_y() const { return s->spec.side_dim ? w->y : nullptr; }
+    const float* last_y_w() const { return s->spec.side_dim ? s->layers.back().side_norm : nullptr; }
+};
+
+}  // namespace
+
+int stack_record_step(cuqwen_engine* e, const LaunchCfg& cfg, const std::function<int()>& after) {
+    Stack* s = e->stack;
+    Pass p{e, s, &s->dec, cfg, 1, true, &e->ctl->token, &e->ctl->pos, 0, &after};
+    LaunchCfg plain = cfg; plain.pdl = false;
+    if (int r = p.done(launch_st_embed_step(s->embed.w, s->embed.pitch, e->ctl, s->dec.x, s->spec.width, plain), "embedding")) return r;
+    if (int r = p.layers(false)) return r;
+    if (int r = p.norms(p.last_y(), p.last_y_w(), s->final_norm, nullptr)) return r;
+    return p.done(launch_st_linear(s->act, p.lin(s->dec.xn1, s->wp, s->head, LIN_F32, s->logits, s->vocab_p), cfg), "head");
+}
+
+int stack_run_chunk(cuqwen_engine* e, int T, int pos0, const int* want, int n_want, float* logits_host) {
+    Stack* s = e->stack;
+    if (T < 1 || T > kChunk) return report_error(CUQWEN_ERR_ARG, "a portion has 1 to %d tokens", kChunk);
+    if (!s->pf.arena) {
+        if (int r = alloc_ws(s, &s->pf, kChunk < s->max_seq ? kChunk : s->max_seq, false)) return r;
+        SK(cudaMalloc((void**)&s->logits_rows, (size_t)kLogitRows * s->vocab_p * 4));
+        SK(cudaMalloc((void**)&s->xn_rows, (size_t)kLogitRows * s->wp * s->esz));
+        SK(cudaMalloc((void**)&s->want_rows, (size_t)kChunk * 4));
+    }
+    const LaunchCfg cfg{e->stream, e->sms, false};
+    Pass p{e, s, &s->pf, cfg, T, false, e->pf_tok, nullptr, pos0, nullptr};
+    if (int r = p.done(launch_st_embed(s->embed.w, s->embed.pitch, e->pf_tok, s->pf.x, s->wp, s->spec.width, T, cfg), "embedding")) return r;
+    if (int r = p.layers(n_want == 0)) return r;
+    if (n_want == 0) return CUQWEN_OK;
+    if (p.last_y()) if (int r = p.norms(p.last_y(), p.last_y_w(), nullptr, nullptr)) return r;
+    SK(cudaMemcpyAsync(s->want_rows, want, (size_t)n_want * 4, cudaMemcpyHostToDevice, e->stream));
+    for (int i = 0; i < n_want; i += kLogitRows) {
+        const int n = n_want - i < kLogitRows ? n_want - i : kLogitRows;
+        NormRowsArgs a{};
+        a.x = s->pf.x; a.ldx = s->wp; a.w[0] = s->final_norm; a.out[0] = s->xn_rows; a.ldo = s->wp; a.n_out = 1; a.width = s->spec.width; a.eps = (float)s->spec.norm_eps; a.rows = s->want_rows + i;
+        if (int r = p.done(launch_st_norms(s->act, a, n, cfg), "final norm")) return r;
+        LinArgs h = p.lin(s->xn_rows, s->wp, s->head, LIN_F32, s->logits_rows, s->vocab_p);
+        h.T = n;
+        if (int r = p.done(launch_st_linear(s->act, h, cfg), "head")) return r;
+        SK(cudaMemcpy2DAsync(logits_host + (size_t)i * s->spec.vocab, (size_t)s->spec.vocab * 4, s->logits_rows, (size_t)s->vocab_p * 4, (size_t)s->spec.vocab * 4, n, cudaMemcpyDeviceToHost, e->stream));
+        SK(cudaStreamSynchronize(e->stream));
+    }
+    return CUQWEN_OK;
+}
+
+}  // namespace cq

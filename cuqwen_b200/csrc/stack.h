@@ -1,0 +1,100 @@
+// Designs described layer by layer (model_dir.h): argument blocks and launchers of their kernels, and the host object that
+// holds their weights, cache and workspace.  The engine's entry points (engine.cu) drive it: the same control block,
+// mailbox, CUDA graph, sampler and prefill calls as the models of the table.
+//
+// Activations are bfloat16 or float32 (Act); weights are bfloat16 as stored, norm weights and sinks are widened to float32.
+// The residual stream, norms, angles, scores, softmax and every accumulation are float32 in both.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+#include "common.cuh"
+#include "launch.h"
+
+namespace cq {
+
+typedef __nv_bfloat16 bf16;
+enum Act : int { ACT_BF16 = 0, ACT_F32 = 1 };
+
+// ---- row kernels (stack_rows.cu) ---------------------------------------------------------------------------------------
+// x[t] = embed[tokens[t]]
+int launch_st_embed(const bf16* table, int pitch, const int* tokens, float* x, int ldx, int width, int T, const LaunchCfg& cfg);
+// The first launch of a decode step: takes over the mailbox, then the same for ctl->token.
+int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, int width, const LaunchCfg& cfg);
+
+// Per row: x += y / rms(y) * y_w (y may be null), then n_out copies x / rms(x) * w[i] -> out[i].
+struct NormRowsArgs {
+    float* x; int ldx;
+    const float* y; int ldy; const float* y_w;
+    const float* w[2]; void* out[2]; int ldo; int n_out;
+    int width; float eps;
+    const int* rows;      // row t of the output comes from row rows[t] of x (null: t); y must be null then
+};
+int launch_st_norms(int act, const NormRowsArgs& a, int T, const LaunchCfg& cfg);
+
+// out[t] = x[t] in the activation type
+int launch_st_narrow(int act, const float* x, int ldx, void* out, int ldo, int T, const LaunchCfg& cfg);
+
+// Per row: the query latent and the cache row of a token from the raw projections.
+//   cq[t] = dq / rms(dq) * dq_w;  cache row pos = [ckv / rms(ckv) * dkv_w | rotated key part]
+struct LatentRowsArgs {
+    const float* dq; int ld; const float* dq_w; void* cq; int ldcq; int q_rank;
+    const float* dkv;                                   // null: the layer has no latent projection of its own
+    const float* dkv_w; void* cache; int ldc, kv_rank, kr_off, rot_dim;      // kr_off: where the rotated part starts, in dkv rows and in cache rows
+    const float2* rot;                                  // (cos, sin) [position][rot_dim / 2]
+    float eps;
+    const int* pos_ptr; int pos0;                       // position of row t: (pos_ptr ? *pos_ptr : pos0) + t
+};
+int launch_st_latent_rows(int act, const LatentRowsArgs& a, int T, const LaunchCfg& cfg);
+
+// q[t][h] = [unrotated dim | rotated rot_dim], heads head_pitch apart, rot part at rot_off: rotated and narrowed.
+struct RopeQArgs { const float* in; void* out; int ld, heads, head_pitch, rot_off, rot_dim; const float2* rot; const int* pos_ptr; int pos0; };
+int launch_st_rope_q(int act, const RopeQArgs& a, int T, const LaunchCfg& cfg);
+
+// ---- matrix products of both activation types on the CUDA cores (stack_linear.cu) -----------------------------------
+enum LinEpi : int {
+    LIN_F32 = 0,          // out (float) = acc
+    LIN_ACT = 1,          // out (activation type) = acc
+    LIN_RELU2 = 2,        // out (activation type) = max(acc, 0)^2
+    LIN_ADD = 3,          // out (float) += acc
+    LIN_GELU_SIDE = 4     // out (activation type) = gelu_tanh(acc) * side[tokens[t]][r]
+};
+struct LinArgs {
+    const void* x; int ldx; const bf16* w; int pitch, K;
+    const void* x2; int ldx2; const bf16* w2; int pitch2, K2;      // a second product summed into the same rows (w2 null: none)
+    int T, R, epi;
+    void* out; int ldo;
+    const bf16* side; int side_pitch, side_dim; const int* tokens; // LIN_GELU_SIDE
+};
+int launch_st_linear(int act, const LinArgs& a, const LaunchCfg& cfg);
+
+// ---- latent attention (latent_attn.cu) -------------------------------------------------------------------------------
+// Softmax attention over [unrotated | rotated] keys with a window, a sink and an output gate.  Keys and values either
+// per head (prefill: k = W_uk c, v = W_uv c of every key in reach) or the latents themselves (decode: queries carried
+// into the latent space by absorb_q, values left there for uv_gate).
+struct LatentAttnArgs {
+    const void *qn, *qr; int ldqn, qn_hs, dn, ldqr, qr_hs, dr;      // unrotated and rotated query parts: row stride, head stride, length
+    const void* kn; int ldkn, kn_hs;                                // unrotated keys; row 0 is key `kbase`
+    const void* kr; int ldkr;                                       // rotated keys, shared by the heads; row 0 is key 0
+    const void* v; int ldv, v_hs, dv;                               // values; row 0 is key `kbase`
+    int kbase;
+    const float* sink;                                              // [heads] or null
+    const float* gate; int ldg, g_hs;                               // out *= sigmoid(gate), or null
+    void* out; int ldo, o_hs;                                       // activation type, or float when out_f32
+    int out_f32;
+    int T, heads, window;                                           // window 0: all earlier keys
+    float scale;
+    const int* pos_ptr; int pos0;
+};
+int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg);
+// qn_abs[h] (float) = W_uk[h]^T qn[h]: the unrotated query against latents instead of keys.  wk: [heads * dimp][pitch].
+struct AbsorbArgs { const void* q; int q_hs; const bf16* wk; int pitch, heads, dim, dimp, kv_rank; void* out; int ldo; };
+int launch_absorb_q(int act, const AbsorbArgs& a, const LaunchCfg& cfg);
+// att[h][v] = sigmoid(g[h][v]) * sum_r W_uv[h][v][r] o[h][r].  o float [heads][ldo].
+struct UvGateArgs { const float* o; int ldo; const bf16* wv; int pitch, heads, vdim, vdimp, kv_rank; const float* gate; int g_hs; void* out; int o_hs; };
+int launch_uv_gate(int act, const UvGateArgs& a, const LaunchCfg& cfg);
+
+// (cos, sin) of pos * freq for every position; freq in double.
+int launch_rot_table(float2* table, int n_pos, int dims, double base, const LaunchCfg& cfg);
+
+}  // namespace cq

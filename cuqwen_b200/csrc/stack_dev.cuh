@@ -1,0 +1,58 @@
+// Device helpers of the layer-list designs' kernels: both activation types behind one interface, row reductions.
+#pragma once
+#include "stack.h"
+
+namespace cq {
+
+__device__ __forceinline__ float act_f(float v) { return v; }
+__device__ __forceinline__ float act_f(bf16 v) { return __bfloat162float(v); }
+template <typename A> __device__ __forceinline__ A to_act(float v);
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
+__device__ __forceinline__ uint32_t pack_bf(float lo, float hi) {
+    __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<uint32_t*>(&h);
+}
+// eight consecutive activations
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+    v[0] = bf_lo(u.x); v[1] = bf_hi(u.x); v[2] = bf_lo(u.y); v[3] = bf_hi(u.y); v[4] = bf_lo(u.z); v[5] = bf_hi(u.z); v[6] = bf_lo(u.w); v[7] = bf_hi(u.w);
+}
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), v); }
+
+// Sum over the CTA, returned to every thread.  `red`: 33 floats of shared memory; safe to call again at once.
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+    v = warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    if (threadIdx.x < 32) {
+        float s = threadIdx.x < (blockDim.x >> 5) ? red[threadIdx.x] : 0.f;
+        s = warp_sum(s);
+        if (threadIdx.x == 0) red[32] = s;
+    }
+    __syncthreads();
+    return red[32];
+}
+__device__ __forceinline__ float inv_rms(float sum_sq, int n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+template <typename... KArgs, typename... Args>
+static int st_launch(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, const LaunchCfg& cfg, Args... args) {
+    cudaLaunchConfig_t lc = {};
+    lc.gridDim = grid; lc.blockDim = block; lc.dynamicSmemBytes = smem; lc.stream = cfg.stream;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = 1;
+    lc.attrs = at; lc.numAttrs = cfg.pdl ? 1 : 0;
+    return (int)cudaLaunchKernelEx(&lc, kern, KArgs(args)...);
+}
+
+}  // namespace cq

@@ -17,6 +17,7 @@ from ._abi import Params, check
 
 FP16, INT8, INT4 = 0, 1, 2
 QUANT_ID = {"fp16": FP16, "int8": INT8, "int4": INT4}
+ACT_ID = {"bfloat16": 0, "float32": 1}
 MODEL_ID = {"0.5b": 0, "1.5b": 1, "3b": 2, "7b": 3, "14b": 4}
 FLAG_ACCURATE_ROPE, FLAG_NO_PDL, FLAG_NO_GRAPH, FLAG_STEP_TRACE, FLAG_TP_NCCL, FLAG_NO_HANDOVER, FLAG_KV_INT8, FLAG_TP_SUM_IN_GEMV, FLAG_PREFILL_ATTN_MMA = 1, 2, 4, 16, 32, 64, 128, 256, 512
 
@@ -108,6 +109,13 @@ def custom_params(vocab, dim, inter, layers, heads, kv, hd, quant, max_seq_len=3
     return p
 
 
+def describe(path) -> str:
+    """cuqwen_describe: a model directory's configuration as the library reads it."""
+    buf = C.create_string_buffer(1 << 20)
+    check(_abi.lib().cuqwen_describe(str(path).encode(), buf, len(buf)))
+    return buf.value.decode()
+
+
 class Engine:
     """malloc_qwen_state + load_weights + qwen_forward behind one object."""
 
@@ -117,6 +125,18 @@ class Engine:
         self.params = Params()
         check(_abi.lib().cuqwen_get_params(self._h, C.byref(self.params)))
         self.device = self.params.device
+
+    @classmethod
+    def open(cls, path, act: str = "bfloat16", max_seq_len: int = 0, device: int = 0, flags: int = 0, repetition_penalty: float = 0.0) -> "Engine":
+        """cuqwen_open: an engine for the design that DIR/config.json names, weights loaded from DIR/model.safetensors."""
+        o = _abi.OpenParams(ACT_ID[act], max_seq_len, device, flags, repetition_penalty)
+        self = cls.__new__(cls)
+        self._h = C.c_void_p()
+        check(_abi.lib().cuqwen_open(str(path).encode(), C.byref(o), C.byref(self._h)))
+        self.params = Params()
+        check(_abi.lib().cuqwen_get_params(self._h, C.byref(self.params)))
+        self.device = self.params.device
+        return self
 
     def close(self) -> None:
         if self._h:
@@ -160,6 +180,15 @@ class Engine:
         """cuqwen_prefill: the KV cache rows [pos0, pos0 + len(tokens)) of these prompt tokens, computed as batched tiles."""
         t = np.ascontiguousarray(tokens, dtype=np.int32)
         check(_abi.lib().cuqwen_prefill(self._h, t.ctypes.data_as(C.POINTER(C.c_int)), int(t.size), pos0))
+
+    def extend(self, tokens, pos0: int, want=()) -> np.ndarray:
+        """cuqwen_extend: a portion of a sequence; float32 logits [len(want), vocab] of the wanted places."""
+        t = np.ascontiguousarray(tokens, dtype=np.int32)
+        w = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((w.size, self.params.vocab_size), dtype=np.float32)
+        check(_abi.lib().cuqwen_extend(self._h, t.ctypes.data_as(C.POINTER(C.c_int)), int(t.size), pos0, w.ctypes.data_as(C.POINTER(C.c_int)), int(w.size),
+                                       out.ctypes.data_as(C.POINTER(C.c_float))))
+        return out
 
     @property
     def last_decode_ms(self) -> float:

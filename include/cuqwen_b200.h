@@ -67,6 +67,25 @@ typedef struct cuqwen_params {
     float norm_eps, rope_theta, repetition_penalty;   /* 0 = 1e-6, 1e6, 1.1 (include/config.h:124-126) */
 } cuqwen_params;
 
+/* ---- model directories (no counterpart in the reference, whose models are compiled in, CMakeLists.txt:18-82) ----
+ * DIR/config.json names a design of the library's registry and describes it layer by layer; DIR/model.safetensors holds
+ * its bfloat16 weights.  An engine opened from a directory takes the same calls as one made by cuqwen_create: cuqwen_step,
+ * cuqwen_step_loop, cuqwen_decode_n, cuqwen_prefill, cuqwen_extend, cuqwen_step_profile, cuqwen_destroy.  Its logits and
+ * residual stream (cuqwen_get_ptr) are float32.  One GPU. */
+enum { CUQWEN_ACT_BF16 = 0,      /* bfloat16 matrix products and activations, 32-bit accumulation, residual stream, norms, softmax */
+       CUQWEN_ACT_F32 = 1 };     /* everything in 32-bit (plain CUDA-core kernels: a check, not a serving mode) */
+typedef struct cuqwen_open_params {
+    int32_t act;                 /* CUQWEN_ACT_* */
+    int32_t max_seq_len;         /* cache rows per layer; 0 = 32768 */
+    int32_t device;
+    uint32_t flags;              /* CUQWEN_FLAG_NO_PDL, CUQWEN_FLAG_NO_GRAPH */
+    float repetition_penalty;    /* 0 = 1.1 */
+} cuqwen_open_params;
+/* Reads, creates and loads in one call.  Designs: Falivik. */
+int cuqwen_open(const char* dir, const cuqwen_open_params* p, cuqwen_engine** out);
+/* The configuration as the library understood it, one line of text per layer.  Host only. */
+int cuqwen_describe(const char* dir, char* out, size_t cap);
+
 /* Fill `p` from the model table.  Replaces the -Dmodel/-Dquant compile-time selection (CMakeLists.txt:18-82). */
 int cuqwen_model_params(int model_id, int quant, cuqwen_params* p);
 
@@ -98,6 +117,11 @@ int cuqwen_decode_n(cuqwen_engine* e, int first_token, int start_pos, int n, int
  * afterwards (prefill the tokens before it).  One GPU, fp16 KV cache, head_dim 64 or 128.  The device time is
  * readable through cuqwen_last_decode_ms. */
 int cuqwen_prefill(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0);
+/* A portion of a sequence with logits (no counterpart in the reference, which computes the logits of every token and keeps
+ * the last, src/main.cu:86-92): n_tokens tokens at positions pos0 .. from the cache that earlier calls left, and the
+ * float32 logits of the places want[0 .. n_want) (ascending, relative to the portion) into logits [n_want][vocab_size] in host
+ * memory.  A sequence may be cut anywhere.  One token takes the decode step's kernels, more take the prefill's. */
+int cuqwen_extend(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0, const int* want, int n_want, float* logits);
 /* Milliseconds the device spent in the last cuqwen_decode_n (CUDA events around the n graph launches). */
 float cuqwen_last_decode_ms(const cuqwen_engine* e);
 
