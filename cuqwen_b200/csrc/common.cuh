@@ -8,7 +8,7 @@ namespace cq {
 
 constexpr int kGroup = 128;  // weights per fp16 scale along the input dim (reference include/config.h:16)
 
-enum Quant : int { Q_F16 = 0, Q_I8 = 1, Q_I4 = 2 };
+enum Quant : int { Q_F16 = 0, Q_I8 = 1, Q_I4 = 2, Q_BF16 = 3 };      // Q_BF16: designs read from a model directory only
 
 // Tensor-parallel exchanges are numbered  step * kSeqPerStep + index + 1  (index < kSeqPerStep: two per layer and a few
 // per token), so that a receive word left over from an earlier exchange can never carry the number a reader expects.

@@ -69,39 +69,49 @@ int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg) {
     return act == ACT_F32 ? st_launch(latent_attn_kernel<float>, grid, dim3(kLaThreads), smem, cfg, a) : st_launch(latent_attn_kernel<bf16>, grid, dim3(kLaThreads), smem, cfg, a);
 }
 
-// CTA = one head, 256 latent columns: thread (c, part) walks a quarter of the head's rows of W_uk for eight columns.
+// One head's query against the latents: its unrotated part carried through W_uk, its rotated part rotated, side by side as
+// the cache rows are.  CTA = (head, 256 latent columns): a warp walks every fourth row of the head's W_uk, eight columns a
+// lane; the head's first CTA also rotates.
 template <typename A>
 __global__ void __launch_bounds__(128) absorb_q_kernel(const AbsorbArgs a) {
     __shared__ float part[3][256];
     pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.x, c0 = blockIdx.y * 256 + (threadIdx.x & 31) * 8, grp = threadIdx.x >> 5;
-    const A* q = reinterpret_cast<const A*>(a.q) + (size_t)h * a.q_hs;
+    const int h = blockIdx.x, lane = threadIdx.x & 31, c0 = blockIdx.y * 256 + lane * 8, grp = threadIdx.x >> 5;
+    const float* q = a.q + (size_t)h * a.q_hs;
+    A* out = reinterpret_cast<A*>(a.out) + (size_t)h * a.ldo;
+    if (blockIdx.y == 0) {
+        const int half = a.rot_dim / 2, pos = *a.pos_ptr;
+        for (int i = threadIdx.x; i < half; i += 128) {
+            const float2 cs = a.rot[(size_t)pos * half + i];
+            const float u = __ldcg(q + a.rot_off + i), v = __ldcg(q + a.rot_off + half + i);
+            out[a.kr_off + i] = to_act<A>(u * cs.x - v * cs.y);
+            out[a.kr_off + half + i] = to_act<A>(v * cs.x + u * cs.y);
+        }
+    }
     const bf16* w = a.wk + (size_t)h * a.dimp * a.pitch + c0;
     float s[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (c0 < a.ldo)                                      // ldo = the padded latent size, a multiple of eight within the pitch
-#pragma unroll 4
+    if (c0 < a.kr_off)                                   // kr_off = the padded latent length, a multiple of eight within the pitch
+#pragma unroll 8
         for (int d = grp; d < a.dim; d += 4) {
             float v[8];
             load8(w + (size_t)d * a.pitch, v);
-            const float qd = act_f(q[d]);
+            const float qd = __ldcg(q + d);
 #pragma unroll
             for (int i = 0; i < 8; ++i) s[i] = fmaf(qd, v[i], s[i]);
         }
     if (grp > 0)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) part[grp - 1][(threadIdx.x & 31) * 8 + i] = s[i];
+        for (int i = 0; i < 8; ++i) part[grp - 1][lane * 8 + i] = s[i];
     __syncthreads();
-    if (grp == 0 && c0 < a.ldo) {
-        A* o = reinterpret_cast<A*>(a.out) + (size_t)h * a.ldo + c0;
+    if (grp == 0 && c0 < a.kr_off)
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            const int j = threadIdx.x * 8 + i;
-            o[i] = to_act<A>(s[i] + part[0][j] + part[1][j] + part[2][j]);
+            const int j = lane * 8 + i;
+            out[c0 + i] = to_act<A>(s[i] + part[0][j] + part[1][j] + part[2][j]);
         }
-    }
 }
 int launch_absorb_q(int act, const AbsorbArgs& a, const LaunchCfg& cfg) {
-    const dim3 grid(a.heads, (a.ldo + 255) / 256);
+    const dim3 grid(a.heads, (a.kr_off + 255) / 256);
     return act == ACT_F32 ? st_launch(absorb_q_kernel<float>, grid, dim3(128), 0, cfg, a) : st_launch(absorb_q_kernel<bf16>, grid, dim3(128), 0, cfg, a);
 }
 

@@ -1,5 +1,6 @@
 // The batched-token GEMM kernel and its launcher (see prefill_gemm.cuh for the design).
 #include "prefill_gemm.cuh"
+#include "stack_dev.cuh"
 #include "tcgen05.cuh"
 
 #include <mutex>
@@ -65,12 +66,50 @@ __device__ __forceinline__ void convert_part(uint32_t raw, uint32_t brow, int sw
     }
 }
 
+// Epilogue of the bfloat16 modes: 32 columns of one token from column r of the matrix on (R of its rows exist).
+__device__ __forceinline__ void pf_store_bf16(const PfGemmArgs& a, const float (&v)[32], int token, int coff, int r, int R) {
+    if (a.mode == PF_ADD_F32) {
+        float* dst = a.out_f + (size_t)token * a.ldo + coff + r;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4)
+            if (r + i < R) {
+                float4 o = *reinterpret_cast<float4*>(dst + i);
+                o.x += v[i]; o.y += v[i + 1]; o.z += v[i + 2]; o.w += v[i + 3];
+                *reinterpret_cast<float4*>(dst + i) = o;
+            }
+        return;
+    }
+    __nv_bfloat16* dst = a.out_b + (size_t)token * a.ldo + coff + r;
+    const __nv_bfloat16* e = a.mode == PF_BF16_GELU_SIDE ? a.side + (size_t)a.tokens[token] * a.side_pitch + r : nullptr;
+#pragma unroll
+    for (int i = 0; i < 32; i += 8) {
+        if (r + i >= R) break;
+        uint4 o;
+        __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            float f[2] = {v[i + 2 * k], v[i + 2 * k + 1]};
+            if (a.mode == PF_BF16_RELU2) { f[0] = fmaxf(f[0], 0.f); f[1] = fmaxf(f[1], 0.f); f[0] *= f[0]; f[1] *= f[1]; }
+            else if (e) {
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    const int c = i + 2 * k + j;
+                    f[j] = r + c < a.side_dim ? gelu_tanh_f(f[j]) * __bfloat162float(e[c]) : 0.f;
+                }
+            }
+            ob[k] = __floats2bfloat162_rn(f[0], f[1]);
+        }
+        *reinterpret_cast<uint4*>(dst + i) = o;
+    }
+}
+
 template <int Q, int NT>
 __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __grid_constant__ PfGemmArgs a) {
     extern __shared__ unsigned char pf_smem_raw[];
     const uint32_t base = (smem_u32(pf_smem_raw) + 1023u) & ~1023u;
     constexpr int NA = pf_na(Q), NB = pf_nb(Q), kRawBytes = pf_raw_bytes(Q, NT), kPfBBytes = NT * 128;
-    constexpr uint32_t kPfIdesc = umma_idesc_f16(kPfM, NT, 0);
+    constexpr bool kRaw = Q == Q_I4 || Q == Q_I8;              // weights that are widened on the way
+    constexpr uint32_t kPfIdesc = Q == Q_BF16 ? umma_idesc_bf16(kPfM, NT, 0) : umma_idesc_f16(kPfM, NT, 0);
     constexpr int kASlot = kPfMH * kPfABytes;                  // X tiles of one slot
     const uint32_t ring_a = base, ring_raw = ring_a + NA * kASlot, ring_b = ring_raw + NA * kRawBytes;
     const uint32_t bars = ring_b + NB * kPfBBytes;
@@ -86,7 +125,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
         while (seg + 1 < a.nseg && tseg >= (a.seg_rows[seg] + NT - 1) / NT) { tseg -= (a.seg_rows[seg] + NT - 1) / NT; coff += a.seg_rows[seg]; ++seg; }
     const int row0 = tseg * rows_mat;                         // first row inside the matrix
     const int R = a.seg_rows[seg];
-    const int nkb = a.K / kPfKB;
+    const int nk1 = (a.K + kPfKB - 1) / kPfKB, nkb = Q == Q_BF16 ? nk1 + (a.K2 + kPfKB - 1) / kPfKB : nk1;      // columns past the end arrive as zeros
     constexpr int kRawKb = Q == Q_I4 ? 32 : 64;               // raw bytes of one row in one K block
     bool failed = false;
 
@@ -104,15 +143,21 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
 
     if (warp == 0) {
         if (lane == 0) {
-            const uint32_t wbytes = Q == Q_F16 ? (uint32_t)kPfBBytes : (uint32_t)(NT * kRawKb);
+            const uint32_t wbytes = !kRaw ? (uint32_t)kPfBBytes : (uint32_t)(NT * kRawKb);
             for (int kb = 0; kb < nkb && !failed; ++kb) {
                 const int sa = kb % NA, sb = kb % NB; const uint32_t pa = (uint32_t)(kb / NA) & 1u;
                 if (!mbar_wait(bar_afree + 8 * sa, pa ^ 1u)) { failed = true; break; }
                 mbar_expect_tx(bar_full + 8 * sa, (uint32_t)(mh * kPfABytes) + wbytes);
+                if (Q == Q_BF16 && kb >= nk1) {     // the second product
+                    const int k2 = (kb - nk1) * kPfKB;
+                    for (int h = 0; h < mh; ++h) tma_load_2d(ring_a + sa * kASlot + h * kPfABytes, &a.tx2, k2, (tm * mh + h) * kPfM, bar_full + 8 * sa);
+                    tma_load_2d(ring_b + sb * kPfBBytes, &a.tw2, k2, row0, bar_full + 8 * sa);
+                    continue;
+                }
                 for (int h = 0; h < mh; ++h)        // a half that lies past the last token arrives as zeros
                     tma_load_2d(ring_a + sa * kASlot + h * kPfABytes, &a.tx, kb * kPfKB, (tm * mh + h) * kPfM, bar_full + 8 * sa);
                 for (int m = 0; m < nmat; ++m) {
-                    if (Q == Q_F16) tma_load_2d(ring_b + sb * kPfBBytes + m * rows_mat * 128, &a.tw[seg + m], kb * kPfKB, row0, bar_full + 8 * sa);    // NB == NA: freed together
+                    if (!kRaw) tma_load_2d(ring_b + sb * kPfBBytes + m * rows_mat * 128, &a.tw[seg + m], kb * kPfKB, row0, bar_full + 8 * sa);    // NB == NA: freed together
                     else tma_load_2d(ring_raw + sa * kRawBytes + m * rows_mat * kRawKb, &a.tw[seg + m], kb * kRawKb, row0, bar_full + 8 * sa);
                 }
             }
@@ -122,7 +167,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
             for (int kb = 0; kb < nkb && !failed; ++kb) {
                 const int sa = kb % NA, sb = kb % NB; const uint32_t pa = (uint32_t)(kb / NA) & 1u, pb = (uint32_t)(kb / NB) & 1u;
                 if (!mbar_wait(bar_full + 8 * sa, pa)) { failed = true; break; }
-                if (Q != Q_F16 && !mbar_wait(bar_conv + 8 * sb, pb)) { failed = true; break; }
+                if (kRaw && !mbar_wait(bar_conv + 8 * sb, pb)) { failed = true; break; }
                 tc_fence_after();
                 const uint32_t at = ring_a + sa * kASlot, bt = ring_b + sb * kPfBBytes;
                 for (int h = 0; h < mh; ++h)
@@ -130,7 +175,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
                     for (int k4 = 0; k4 < kPfKB / 16; ++k4)
                         umma_f16(tmem + (uint32_t)(h * NT), umma_desc(at + h * kPfABytes + k4 * 32), umma_desc(bt + k4 * 32), kPfIdesc, (uint32_t)((kb | k4) != 0));
                 umma_commit(bar_afree + 8 * sa);           // both slots may be refilled once these MMAs have read them
-                if (Q != Q_F16) umma_commit(bar_bfree + 8 * sb);
+                if (kRaw) umma_commit(bar_bfree + 8 * sb);
             }
             umma_commit(bar_done);
         }
@@ -143,7 +188,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
         const int mat = swiglu ? c / rows_mat : 0, rin = swiglu ? c % rows_mat : c;
         const int grow = row0 + rin;
         const bool valid = grow < R;
-        if (Q != Q_F16) {
+        if (kRaw) {
             const int ngrp = a.K / kGroup;
             const __half* srow = a.s[seg + mat] + (size_t)(valid ? grow : 0) * ngrp;
             // the scales of the next two groups are already on their way while a group is widened (a load from L2 takes
@@ -157,7 +202,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
                 if (!mbar_wait(bar_full + 8 * sa, pa)) { failed = true; break; }
                 if (!mbar_wait(bar_bfree + 8 * sb, pb ^ 1u)) { failed = true; break; }     // the MMAs of two K blocks ago have read this B slot
                 {
-                    constexpr int QQ = Q == Q_F16 ? Q_I8 : Q;
+                    constexpr int QQ = kRaw ? Q : Q_I8;
                     const uint32_t rawrow = ring_raw + sa * kRawBytes + c * kRawKb, brow = ring_b + sb * kPfBBytes + c * 128;
                     if (kPerRow == 4) convert_part<QQ, 16>(rawrow + kpart * (kRawKb / 4), brow, c & 7, kpart * 2, __half2half2(sc_use));
                     else {
@@ -187,7 +232,8 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
                     tmem_ld32(tlane + (uint32_t)col, v);
                     const int r = row0 + col;
                     if (tv && r < R) {
-                    if (a.mode == PF_OUT_F32) {
+                    if (Q == Q_BF16 && a.mode != PF_OUT_F32) pf_store_bf16(a, v, token, coff, r, R);
+                    else if (a.mode == PF_OUT_F32) {
                         float* dst = a.out_f + (size_t)token * a.ldo + coff + r;
 #pragma unroll
                         for (int i = 0; i < 32; i += 4) if (r + i < R) *reinterpret_cast<float4*>(dst + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
@@ -263,11 +309,11 @@ static PfEncodeFn pf_encode() {
     }();
     return fn;
 }
-// Row-major 2-D map: `cols` elements a row (row pitch = cols * elem bytes), box box_cols x box_rows.
-static int pf_map(CUtensorMap* m, const void* p, CUtensorMapDataType dt, int elem, size_t rows, size_t cols, int box_cols, int box_rows, bool swizzle) {
+// Row-major 2-D map: `cols` elements a row (row pitch = cols elements, or `pitch`), box box_cols x box_rows.
+static int pf_map(CUtensorMap* m, const void* p, CUtensorMapDataType dt, int elem, size_t rows, size_t cols, int box_cols, int box_rows, bool swizzle, size_t pitch = 0) {
     PfEncodeFn fn = pf_encode();
     if (!fn) return (int)cudaErrorNotSupported;
-    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {cols * (size_t)elem};
+    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(pitch ? pitch : cols) * (size_t)elem};
     const cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows}, estr[2] = {1, 1};
     const CUresult r = fn(m, dt, 2, const_cast<void*>(p), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                           swizzle ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
@@ -331,6 +377,37 @@ int launch_prefill_gemm(int quant, PfGemmArgs& a, const void* x, const void* con
     if (quant == Q_I4) return pf_go<Q_I4, kPfN / 4>(a, grid, stream);
     if (quant == Q_I8) return pf_go<Q_I8, kPfN / 4>(a, grid, stream);
     return pf_go<Q_F16, kPfN / 4>(a, grid, stream);
+}
+
+int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16Mat* m, int nmat, const void* x2, int ldx2, const PfBf16Mat* m2, cudaStream_t stream) {
+    if (a.T <= 0 || a.K <= 0 || a.K % 8 || a.ldo % 8 || ldx % 8 || nmat < 1 || nmat > 3 || (a.mode != PF_OUT_F32 && a.mode < PF_BF16) || (x2 && (nmat != 1 || !m2 || m2->rows != m->rows || a.K2 % 8 || ldx2 % 8)))
+        return (int)cudaErrorInvalidValue;
+    if (!x2) a.K2 = 0;
+    int sms = 0, dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    a.mh = a.T > kPfM ? kPfMH : 1;
+    const int mtiles = (a.T + kPfM * a.mh - 1) / (kPfM * a.mh);
+    int wide = 0;
+    for (int i = 0; i < nmat; ++i) wide += (m[i].rows + kPfN - 1) / kPfN;
+    const int nt = (sms > 0 && wide * mtiles * 4 <= sms) ? kPfN / 4 : (sms > 0 && wide * mtiles * 2 <= sms) ? kPfN / 2 : kPfN;
+    const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    if (int r = pf_map(&a.tx, x, bf, 2, (size_t)a.T, (size_t)a.K, kPfKB, kPfM, true, (size_t)ldx)) return r;
+    int tiles = 0;
+    a.R = 0;
+    for (int i = 0; i < nmat; ++i) {
+        if (!m[i].w || m[i].rows <= 0 || m[i].rows % 8 || m[i].pitch % 8 || m[i].pitch < a.K) return (int)cudaErrorInvalidValue;
+        if (int r = pf_map(&a.tw[i], m[i].w, bf, 2, (size_t)m[i].rows, (size_t)a.K, kPfKB, nt, true, (size_t)m[i].pitch)) return r;
+        a.seg_rows[i] = m[i].rows;
+        tiles += (m[i].rows + nt - 1) / nt; a.R += m[i].rows;
+    }
+    a.nseg = nmat;
+    if (x2) {
+        if (int r = pf_map(&a.tx2, x2, bf, 2, (size_t)a.T, (size_t)a.K2, kPfKB, kPfM, true, (size_t)ldx2)) return r;
+        if (int r = pf_map(&a.tw2, m2->w, bf, 2, (size_t)m2->rows, (size_t)a.K2, kPfKB, nt, true, (size_t)m2->pitch)) return r;
+    }
+    const dim3 grid(mtiles, tiles);
+    return nt == kPfN ? pf_go<Q_BF16, kPfN>(a, grid, stream) : nt == kPfN / 2 ? pf_go<Q_BF16, kPfN / 2>(a, grid, stream) : pf_go<Q_BF16, kPfN / 4>(a, grid, stream);
 }
 
 }  // namespace cq

@@ -16,6 +16,8 @@
 // After the last K block warps 2-9 read the accumulators (tcgen05.ld, warp w owns TMEM lanes 32 * (w % 4) ..) and
 // apply the epilogue.  Every mbarrier wait is bounded (tma.cuh); a wait that runs out sets *err and the CTA drains.
 #pragma once
+#include <cuda_bf16.h>
+
 #include "tma.cuh"
 
 namespace cq {
@@ -33,7 +35,7 @@ constexpr int kPfABytes = kPfM * 128;          // one X tile of a stage
 // fp16 weights have no raw form: their B tile arrives by TMA, NB = NA.
 __host__ __device__ constexpr int pf_raw_bytes(int quant, int nt) { return quant == 2 ? nt * 32 : quant == 1 ? nt * 64 : 0; }
 __host__ __device__ constexpr int pf_na(int quant) { return quant == 2 ? 4 : 3; }
-__host__ __device__ constexpr int pf_nb(int quant) { return quant == 0 ? 3 : 2; }
+__host__ __device__ constexpr int pf_nb(int quant) { return quant == 0 || quant == 3 ? 3 : 2; }
 __host__ __device__ constexpr int pf_smem_bytes(int quant, int nt) {
     return pf_na(quant) * (kPfMH * kPfABytes + pf_raw_bytes(quant, nt)) + pf_nb(quant) * nt * 128 + 1024 /* alignment slack */ + 256 /* barriers, TMEM address */;
 }
@@ -42,7 +44,12 @@ enum PfMode : int {
     PF_OUT_F16 = 0,     // out_h[t][r] = half(acc + bias[r])
     PF_OUT_F32 = 1,     // out_f[t][r] = acc
     PF_RESID = 2,       // out_h[t][r] = half(float(out_h[t][r]) + acc)          (reference src/kernels.cu:670-671)
-    PF_SWIGLU = 3       // out_h[t][r] = half(silu(acc_gate) * acc_up), fast-math exp / divide (src/kernels.cu:565-567)
+    PF_SWIGLU = 3,      // out_h[t][r] = half(silu(acc_gate) * acc_up), fast-math exp / divide (src/kernels.cu:565-567)
+    // bfloat16 weights and activations (Q_BF16; PF_OUT_F32 as well)
+    PF_BF16 = 4,            // out_b[t][r] = acc
+    PF_BF16_RELU2 = 5,      // out_b[t][r] = max(acc, 0)^2
+    PF_ADD_F32 = 6,         // out_f[t][r] += acc
+    PF_BF16_GELU_SIDE = 7   // out_b[t][r] = gelu_tanh(acc) * side[tokens[t]][r], r < side_dim, else 0
 };
 
 struct PfGemmArgs {
@@ -61,10 +68,20 @@ struct PfGemmArgs {
     int mode;
     int mh;                    // token halves per CTA (1 or 2), set by the launcher
     unsigned* err;
+    // Q_BF16
+    __nv_bfloat16* out_b;
+    CUtensorMap tx2, tw2;      // a second product summed into the same rows (K2 = 0: none)
+    int K2;
+    const __nv_bfloat16* side; int side_pitch, side_dim; const int* tokens;
 };
 
 // Fills the tensor maps and launches.  PF_SWIGLU: w = {gate, up}, nmat = 2, rows[0] = rows of each.  Other modes: nmat
 // matrices of rows[i] rows each, outputs side by side; a.s[i] hold their scales.
 int launch_prefill_gemm(int quant, PfGemmArgs& a, const void* x, const void* const* w, const int* rows, int nmat, cudaStream_t stream);
+
+// bfloat16 form: x [T][ldx], matrices of rows[i] stored rows (multiples of 8) of pitch[i] columns, of which the first a.K
+// (any multiple of 8) count; x2 / w2: the second product (its rows = rows[0], columns a.K2).
+struct PfBf16Mat { const void* w; int rows, pitch; };
+int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16Mat* m, int nmat, const void* x2, int ldx2, const PfBf16Mat* m2, cudaStream_t stream);
 
 }  // namespace cq

@@ -9,6 +9,9 @@
 //   raw          [query latent q_rank | cache row | gate heads * vdim], float32 sums of the first launch of a layer
 #include "stack.h"
 
+#include "gemv_seg.cuh"
+#include "prefill_gemm.cuh"
+
 #include <cmath>
 #include <cstring>
 #include <string>
@@ -29,7 +32,7 @@ struct StLayer {
     LatentAttnSpec a;
     int ff = 0;
     int dimp = 0, rotp = 0, vdimp = 0, kvrp = 0, qrp = 0, crow = 0, head_q = 0;
-    int cache = -1, rot = -1;
+    int cache = -1, rot = -1, nsplit = 0;      // nsplit: key ranges of the bfloat16 decode attention (0: sizes it does not cover)
     StMat dq, uq, dkv, uk, uv, g, o, up, down, side_gate, side_proj;
     float *norm1 = nullptr, *norm2 = nullptr, *dq_norm = nullptr, *dkv_norm = nullptr, *sink = nullptr, *side_norm = nullptr;
 };
@@ -55,13 +58,14 @@ struct Stack {
     // workspace: a decode step's (one row), and a portion's (kChunk rows; allocated at first use)
     struct Ws {
         int rows = 0, kv_rows = 0;
-        float *x = nullptr, *raw = nullptr, *qf = nullptr, *y = nullptr, *o_lat = nullptr;
-        void *xn1 = nullptr, *xn2 = nullptr, *cq = nullptr, *q = nullptr, *q_abs = nullptr, *att = nullptr, *h = nullptr, *sg = nullptr, *k = nullptr, *v = nullptr;
+        float *x = nullptr, *x2 = nullptr, *raw = nullptr, *qf = nullptr, *y = nullptr, *o_lat = nullptr, *part_o = nullptr, *part_ml = nullptr;
+        void *xn1 = nullptr, *xn2 = nullptr, *cq = nullptr, *q = nullptr, *att = nullptr, *h = nullptr, *sg = nullptr, *kv = nullptr;
         uint8_t* arena = nullptr;
     } dec, pf;
+    float* dec_x = nullptr;             // where a decode step leaves the residual stream (every layer's part added)
     float* logits = nullptr;            // decode step
     float* logits_rows = nullptr; void* xn_rows = nullptr; int* want_rows = nullptr;
-    int max_raw = 0, max_q = 0, max_att = 0, max_ff = 0, max_qr = 0, max_kn = 0, max_kvr = 0;
+    int max_raw = 0, max_q = 0, max_att = 0, max_ff = 0, max_qr = 0, max_kv = 0, max_kvr = 0, max_heads = 0, max_split = 1;
 };
 
 #define SK(call) do { cudaError_t e_ = (cudaError_t)(call); if (e_ != cudaSuccess) return report_error(e_ == cudaErrorInvalidValue ? CUQWEN_ERR_ARG : CUQWEN_ERR_CUDA, "%s: %s (%s:%d)", #call, cudaGetErrorString(e_), __FILE__, __LINE__); } while (0)
@@ -70,7 +74,7 @@ const StackSpec& stack_spec(const Stack* s) { return s->spec; }
 int stack_act(const Stack* s) { return s->act; }
 float* stack_logits(const Stack* s) { return s->logits; }
 size_t stack_cache_bytes(const Stack* s, void** ptr) { *ptr = s->cache; return s->cache_bytes; }
-void stack_residual(const Stack* s, void** ptr, size_t* bytes) { *ptr = s->dec.x; *bytes = (size_t)s->spec.width * 4; }
+void stack_residual(const Stack* s, void** ptr, size_t* bytes) { *ptr = s->dec_x ? s->dec_x : s->dec.x; *bytes = (size_t)s->spec.width * 4; }
 int stack_chunk() { return kChunk; }
 
 static int alloc_ws(Stack* s, Stack::Ws* w, int rows, bool decode) {
@@ -87,14 +91,16 @@ static int alloc_ws(Stack* s, Stack::Ws* w, int rows, bool decode) {
         w->att = a.get(R * s->max_att * E); w->h = a.get(R * (s->max_ff ? s->max_ff : 8) * E);
         w->sg = a.get(R * (s->sidep ? s->sidep : 8) * E);
         if (decode) {
-            w->q_abs = a.get((size_t)s->max_kvr * E);
+            w->x2 = (float*)a.get(R * s->wp * 4);
             w->o_lat = (float*)a.get((size_t)s->max_kvr * 4);
+            w->part_o = (float*)a.get((size_t)s->max_split * s->max_kvr * 4);
+            w->part_ml = (float*)a.get((size_t)s->max_split * s->max_heads * 8);
         } else {
             // keys and values of everything a portion's queries can reach: the portion and the widest window before it
             int reach = 0;
             for (const StLayer& l : s->layers) { const int r = l.a.window > 0 && l.a.window < s->max_seq ? l.a.window - 1 : s->max_seq; reach = r > reach ? r : reach; }
             w->kv_rows = rows + reach < s->max_seq ? rows + reach : s->max_seq;
-            w->k = a.get((size_t)w->kv_rows * s->max_kn * E); w->v = a.get((size_t)w->kv_rows * s->max_att * E);
+            w->kv = a.get((size_t)w->kv_rows * s->max_kv * E);
         }
         if (!pass) {
             SK(cudaMalloc((void**)&w->arena, dry.used + 256));
@@ -126,7 +132,9 @@ int stack_create(cuqwen_engine* e, const StackSpec& spec, int act, int max_seq_l
         } else l.cache = s->layers[l.a.kv_from].cache;
         auto up = [](int& m, int v) { if (v > m) m = v; };
         up(s->max_raw, l.qrp + (l.a.kv_from < 0 ? l.crow : 0) + l.a.heads * l.vdimp); up(s->max_q, l.a.heads * l.head_q); up(s->max_att, l.a.heads * l.vdimp);
-        up(s->max_ff, pad8(l.ff)); up(s->max_qr, l.qrp); up(s->max_kn, l.a.heads * l.dimp); up(s->max_kvr, l.a.heads * l.kvrp);
+        up(s->max_ff, pad8(l.ff)); up(s->max_qr, l.qrp); up(s->max_kv, l.a.heads * (l.dimp + l.vdimp)); up(s->max_kvr, l.a.heads * l.kvrp); up(s->max_heads, l.a.heads);
+        up(s->max_q, l.a.heads * l.crow);
+        if (act == ACT_BF16) { l.nsplit = latent_decode_splits(l.a.heads, l.crow, l.kvrp, l.a.window, max_seq_len, e->sms); up(s->max_split, l.nsplit); }
         s->layers.push_back(l);
     }
     s->cache_bytes = coff;
@@ -291,18 +299,26 @@ struct Pass {
     }
     uint8_t* cache_of(const StLayer& l) { return s->cache + s->cache_off[l.cache]; }
 
+    // Attention of the queries in w->qf (float32, not yet rotated) -> w->att, gated.
     int attention(const StLayer& l, const float* gate, int ldraw) {
         const LatentAttnSpec& a = l.a;
-        LatentAttnArgs t{};
-        t.qr = (uint8_t*)w->q + (size_t)l.dimp * s->esz; t.ldqr = a.heads * l.head_q; t.qr_hs = l.head_q; t.dr = a.rot_dim;
         uint8_t* c = cache_of(l);
-        t.kr = c + (size_t)l.kvrp * s->esz; t.ldkr = l.crow;
+        const float2* rot = s->rot_tables[l.rot];
+        LatentAttnArgs t{};
+        t.kr = c + (size_t)l.kvrp * s->esz; t.ldkr = l.crow; t.dr = a.rot_dim;
         t.sink = l.sink; t.T = T; t.heads = a.heads; t.window = a.window; t.scale = (float)a.scale; t.pos_ptr = pos_ptr; t.pos0 = pos0;
         if (decode) {
-            AbsorbArgs b{};
-            b.q = w->q; b.q_hs = l.head_q; b.wk = l.uk.w; b.pitch = l.uk.pitch; b.heads = a.heads; b.dim = a.dim; b.dimp = l.dimp; b.kv_rank = a.kv_rank; b.out = w->q_abs; b.ldo = l.kvrp;
+            AbsorbArgs b{w->qf, l.head_q, l.dimp, a.rot_dim, rot, pos_ptr, l.uk.w, l.uk.pitch, a.heads, a.dim, l.dimp, w->q, l.crow, l.kvrp};
             GO(launch_absorb_q(s->act, b, cfg));
-            t.qn = w->q_abs; t.ldqn = a.heads * l.kvrp; t.qn_hs = l.kvrp; t.dn = a.kv_rank;
+            if (l.nsplit > 0) {
+                LatentDecodeArgs d{};
+                d.q = (const bf16*)w->q; d.crow = l.crow; d.cache = (const bf16*)c; d.kvrp = l.kvrp; d.sink = l.sink; d.heads = a.heads; d.window = a.window; d.scale = (float)a.scale;
+                d.pos_ptr = pos_ptr; d.nsplit = l.nsplit; d.part_o = w->part_o; d.part_ml = w->part_ml;
+                d.wv = l.uv.w; d.pitch = l.uv.pitch; d.vdim = a.vdim; d.vdimp = l.vdimp; d.kv_rank = a.kv_rank; d.gate = gate; d.g_hs = l.vdimp; d.out = (bf16*)w->att; d.o_hs = l.vdimp;
+                return launch_latent_decode(d, cfg, [this](int err, const char* what) { return done(err, what); });
+            }
+            t.qn = w->q; t.ldqn = a.heads * l.crow; t.qn_hs = l.crow; t.dn = a.kv_rank;
+            t.qr = (uint8_t*)w->q + (size_t)l.kvrp * s->esz; t.ldqr = a.heads * l.crow; t.qr_hs = l.crow;
             t.kn = c; t.ldkn = l.crow; t.kn_hs = 0; t.v = c; t.ldv = l.crow; t.v_hs = 0; t.dv = a.kv_rank;
             t.out = w->o_lat; t.out_f32 = 1; t.ldo = a.heads * l.kvrp; t.o_hs = l.kvrp;
             GO(launch_latent_attn(s->act, t, cfg));
@@ -312,22 +328,52 @@ struct Pass {
             GO(launch_uv_gate(s->act, u, cfg));
             return CUQWEN_OK;
         }
-        // keys and values of every token the portion's queries reach
+        RopeQArgs rq{w->qf, w->q, l.uq.rows, a.heads, l.head_q, l.dimp, a.rot_dim, rot, pos_ptr, pos0};
+        GO(launch_st_rope_q(s->act, rq, T, cfg));
+        // keys and values of every token the portion's queries reach, side by side in a row
         const int k0 = a.window > 0 && pos0 - a.window + 1 > 0 ? pos0 - a.window + 1 : 0, n = pos0 + T - k0;
-        LinArgs k = lin(c + (size_t)k0 * l.crow * s->esz, l.crow, l.uk, LIN_ACT, w->k, a.heads * l.dimp);
-        LinArgs v = lin(c + (size_t)k0 * l.crow * s->esz, l.crow, l.uv, LIN_ACT, w->v, a.heads * l.vdimp);
-        k.T = v.T = n;
-        GO(launch_st_linear(s->act, k, cfg));
-        GO(launch_st_linear(s->act, v, cfg));
+        const int kcols = a.heads * l.dimp, ldkv = kcols + a.heads * l.vdimp;
+        const StMat* kv[2] = {&l.uk, &l.uv};
+        if (int r = product(LIN_ACT, c + (size_t)k0 * l.crow * s->esz, l.crow, kv, 2, w->kv, ldkv, n)) return r;
+        t.qr = (uint8_t*)w->q + (size_t)l.dimp * s->esz; t.ldqr = a.heads * l.head_q; t.qr_hs = l.head_q;
         t.qn = w->q; t.ldqn = a.heads * l.head_q; t.qn_hs = l.head_q; t.dn = a.dim;
-        t.kn = w->k; t.ldkn = a.heads * l.dimp; t.kn_hs = l.dimp; t.v = w->v; t.ldv = a.heads * l.vdimp; t.v_hs = l.vdimp; t.dv = a.vdim; t.kbase = k0;
+        t.kn = w->kv; t.ldkn = ldkv; t.kn_hs = l.dimp; t.v = (uint8_t*)w->kv + (size_t)kcols * s->esz; t.ldv = ldkv; t.v_hs = l.vdimp; t.dv = a.vdim; t.kbase = k0;
         t.gate = gate; t.ldg = ldraw; t.g_hs = l.vdimp; t.out = w->att; t.ldo = a.heads * l.vdimp; t.o_hs = l.vdimp;
-        GO(launch_latent_attn(s->act, t, cfg));
+        if (s->act == ACT_BF16 && latent_prefill_fits(a.dim, a.rot_dim, a.vdim)) GO(launch_latent_prefill_attn(t, n, (size_t)s->max_seq, err_word(), cfg));
+        else GO(launch_latent_attn(s->act, t, cfg));
+        return CUQWEN_OK;
+    }
+    unsigned* err_word() { return reinterpret_cast<unsigned*>(&e->ctl->pad[0]); }
+
+    // out[t] = epilogue(W x[t]) for n rows of x; several matrices (one epilogue) write their rows side by side, m2 adds a second product
+    // (x2) to the one matrix.  The tensor-core GEMM in bfloat16, the CUDA-core kernels in float32.
+    int product(int epi, const void* x, int ldx, const StMat* const* m, int nm, void* out, int ldo, int n, const void* x2 = nullptr, int ldx2 = 0, const StMat* m2 = nullptr,
+                const LinArgs* side = nullptr) {
+        if (s->act == ACT_BF16 && n > 1) {
+            PfGemmArgs g; memset(&g, 0, sizeof g);
+            PfBf16Mat pm[3], pm2{};
+            for (int i = 0; i < nm; ++i) pm[i] = PfBf16Mat{m[i]->w, m[i]->rows, m[i]->pitch};
+            g.T = n; g.K = (m[0]->cols + 7) / 8 * 8; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = err_word();
+            g.mode = epi == LIN_F32 ? PF_OUT_F32 : epi == LIN_ACT ? PF_BF16 : epi == LIN_RELU2 ? PF_BF16_RELU2 : epi == LIN_ADD ? PF_ADD_F32 : PF_BF16_GELU_SIDE;
+            if (m2) { pm2 = PfBf16Mat{m2->w, m2->rows, m2->pitch}; g.K2 = m2->cols; }
+            if (side) { g.side = side->side; g.side_pitch = side->side_pitch; g.side_dim = side->side_dim; g.tokens = side->tokens; }
+            GO(launch_prefill_gemm_bf16(g, x, ldx, pm, nm, m2 ? x2 : nullptr, ldx2, m2 ? &pm2 : nullptr, cfg.stream));
+            return CUQWEN_OK;
+        }
+        size_t off = 0;
+        for (int i = 0; i < nm; ++i) {
+            LinArgs a = lin(x, ldx, *m[i], epi, (uint8_t*)out + off * (epi == LIN_F32 || epi == LIN_ADD ? 4 : s->esz), ldo);
+            a.T = n;
+            if (m2) { a.x2 = x2; a.ldx2 = ldx2; a.w2 = m2->w; a.pitch2 = m2->pitch; a.K2 = m2->cols; }
+            if (side) { a.side = side->side; a.side_pitch = side->side_pitch; a.side_dim = side->side_dim; a.tokens = side->tokens; }
+            GO(launch_st_linear(s->act, a, cfg));
+            off += m[i]->rows;
+        }
         return CUQWEN_OK;
     }
 
-    // All layers.  cache_only: nothing after the last layer's cache rows is needed.  Leaves the residual stream in w->x with
-    // the last layer's token input still to be added (w->y, side_norm of the last layer).
+    // All layers, one launch per operation.  cache_only: nothing after the last layer's cache rows is needed.  Leaves the
+    // residual stream in w->x with the last layer's token input still to be added (last_y).
     int layers(bool cache_only) {
         const StackSpec& sp = s->spec;
         const float* y = nullptr; const float* y_w = nullptr;
@@ -337,34 +383,115 @@ struct Pass {
             const bool own = a.kv_from < 0, stop = cache_only && i + 1 == s->layers.size();
             if (stop && !own) return CUQWEN_OK;
             if (int r = norms(y, y_w, l.norm1, l.ff && !stop ? l.norm2 : nullptr)) return r;
-            const int c_off = l.qrp, g_off = c_off + (own ? l.crow : 0), ldraw = g_off + a.heads * l.vdimp;
-            if (!stop) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.dq, LIN_F32, w->raw, ldraw), cfg));
-            if (own) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.dkv, LIN_F32, w->raw + c_off, ldraw), cfg));
-            if (a.gate && !stop) GO(launch_st_linear(s->act, lin(w->xn1, s->wp, l.g, LIN_F32, w->raw + g_off, ldraw), cfg));
-            if (l.ff && !stop) GO(launch_st_linear(s->act, lin(w->xn2, s->wp, l.up, LIN_RELU2, w->h, l.up.rows), cfg));
-            LatentRowsArgs lr{};
-            lr.dq = w->raw; lr.ld = ldraw; lr.dq_w = l.dq_norm; lr.cq = w->cq; lr.ldcq = l.qrp; lr.q_rank = a.q_rank;
-            if (own) { lr.dkv = w->raw + c_off; lr.dkv_w = l.dkv_norm; lr.cache = cache_of(l); lr.ldc = l.crow; lr.kv_rank = a.kv_rank; lr.kr_off = l.kvrp; lr.rot_dim = a.rot_dim; lr.rot = s->rot_tables[l.rot]; }
-            lr.eps = (float)sp.norm_eps; lr.pos_ptr = pos_ptr; lr.pos0 = pos0;
+            const int c_off = l.qrp, g_off = c_off + (own ? l.crow : 0), ldraw = g_off + (a.gate ? a.heads * l.vdimp : 0);
+            const StMat* first[3]; int nf = 0;
+            first[nf++] = &l.dq;
+            if (own) first[nf++] = &l.dkv;
+            if (a.gate && !stop) first[nf++] = &l.g;
+            if (int r = product(LIN_F32, w->xn1, s->wp, first, nf, w->raw, ldraw, T)) return r;
+            const StMat *up[1] = {&l.up}, *uq[1] = {&l.uq}, *o[1] = {&l.o}, *sg[1] = {&l.side_gate}, *sp1[1] = {&l.side_proj};
+            if (l.ff && !stop) if (int r = product(LIN_RELU2, w->xn2, s->wp, up, 1, w->h, l.up.rows, T)) return r;
+            LatentRowsArgs lr = latent_rows(l, ldraw);
             GO(launch_st_latent_rows(s->act, lr, T, cfg));
             if (stop) return CUQWEN_OK;
-            GO(launch_st_linear(s->act, lin(w->cq, l.qrp, l.uq, LIN_F32, w->qf, l.uq.rows), cfg));
-            RopeQArgs rq{w->qf, w->q, l.uq.rows, a.heads, l.head_q, l.dimp, a.rot_dim, s->rot_tables[l.rot], pos_ptr, pos0};
-            GO(launch_st_rope_q(s->act, rq, T, cfg));
+            if (int r = product(LIN_F32, w->cq, l.qrp, uq, 1, w->qf, l.uq.rows, T)) return r;
             if (int r = attention(l, a.gate ? w->raw + g_off : nullptr, ldraw)) return r;
-            LinArgs o = lin(w->att, a.heads * l.vdimp, l.o, LIN_ADD, w->x, s->wp);
-            if (l.ff) { o.x2 = w->h; o.ldx2 = l.up.rows; o.w2 = l.down.w; o.pitch2 = l.down.pitch; o.K2 = l.down.cols; }
-            GO(launch_st_linear(s->act, o, cfg));
+            if (int r = product(LIN_ADD, w->att, a.heads * l.vdimp, o, 1, w->x, s->wp, T, w->h, l.up.rows, l.ff ? &l.down : nullptr)) return r;
             if (sp.side_dim) {
                 // the token input reads the stream itself, narrowed like every activation
                 if (int r = narrow_x()) return r;
-                LinArgs g = lin(w->xn1, s->wp, l.side_gate, LIN_GELU_SIDE, w->sg, s->sidep);
-                g.side = s->side_embed.w + i * sp.side_dim; g.side_pitch = s->side_embed.pitch; g.side_dim = sp.side_dim; g.tokens = tokens;
-                GO(launch_st_linear(s->act, g, cfg));
-                GO(launch_st_linear(s->act, lin(w->sg, s->sidep, l.side_proj, LIN_F32, w->y, s->wp), cfg));
+                const LinArgs e1 = side_args(i);
+                if (int r = product(LIN_GELU_SIDE, w->xn1, s->wp, sg, 1, w->sg, s->sidep, T, nullptr, 0, nullptr, &e1)) return r;
+                if (int r = product(LIN_F32, w->sg, s->sidep, sp1, 1, w->y, s->wp, T)) return r;
                 y = w->y; y_w = l.side_norm;
             }
         }
+        return CUQWEN_OK;
+    }
+    LatentRowsArgs latent_rows(const StLayer& l, int ldraw) {
+        const LatentAttnSpec& a = l.a;
+        LatentRowsArgs lr{};
+        lr.dq = w->raw; lr.ld = ldraw; lr.dq_w = l.dq_norm; lr.cq = w->cq; lr.ldcq = l.qrp; lr.q_rank = a.q_rank;
+        if (a.kv_from < 0) { lr.dkv = w->raw + l.qrp; lr.dkv_w = l.dkv_norm; lr.cache = cache_of(l); lr.ldc = l.crow; lr.kv_rank = a.kv_rank; lr.kr_off = l.kvrp; lr.rot_dim = a.rot_dim; lr.rot = s->rot_tables[l.rot]; }
+        lr.eps = (float)s->spec.norm_eps; lr.pos_ptr = pos_ptr; lr.pos0 = pos0;
+        return lr;
+    }
+    LinArgs side_args(size_t layer) {
+        LinArgs g{};
+        g.side = s->side_embed.w + layer * s->spec.side_dim; g.side_pitch = s->side_embed.pitch; g.side_dim = s->spec.side_dim; g.tokens = tokens;
+        return g;
+    }
+
+    // A decode step's layers in bfloat16, fused: per layer eight launches - [dq | dkv | g | up] with the previous layer's token
+    // input and both norms in the prologue; uq with the latent's norm, and the cache row; the queries into latent space; the
+    // split attention and its fold with W_uv and the gate; [o + down]; the token input's two matrices (its norm is left to the
+    // next prologue).  The stream alternates between two buffers: a prologue reads one and CTA 0 writes the other.
+    SegGemvArgs seg(int stage, int K) {
+        SegGemvArgs g; memset(&g, 0, sizeof g);
+        g.stage = stage; g.K = K; g.eps = (float)s->spec.norm_eps; g.width = s->spec.width; g.nvar = 1; g.tokens = tokens; g.err = err_word();
+        return g;
+    }
+    static SegMat sm(const StMat& m) { return SegMat{m.w, m.rows, m.pitch}; }
+    int fused_layers() {
+        const StackSpec& sp = s->spec;
+        float *x = w->x, *other = w->x2;
+        const float* y_w = nullptr;
+        auto take_x = [&](SegGemvArgs& g) {              // the stream, with the token input that is still to be added
+            g.x = x;
+            if (y_w) { g.y = w->y; g.y_w = y_w; g.x_next = other; float* t = x; x = other; other = t; y_w = nullptr; }
+        };
+        for (size_t i = 0; i < s->layers.size(); ++i) {
+            const StLayer& l = s->layers[i];
+            const LatentAttnSpec& a = l.a;
+            const bool own = a.kv_from < 0;
+            const int c_off = l.qrp, g_off = c_off + (own ? l.crow : 0), ldraw = g_off + (a.gate ? a.heads * l.vdimp : 0);
+            {
+                SegGemvArgs g = seg(SEG_NORM, l.dq.pitch);
+                SegMat m[4]; int n = 0;
+                take_x(g);
+                auto add = [&](const StMat& mat, int var, int epi, void* out) { g.seg_var[n] = var; g.epi[n] = epi; g.out[n] = out; m[n++] = sm(mat); };
+                g.nw[0] = l.norm1;
+                add(l.dq, 0, LIN_F32, w->raw);
+                if (own) add(l.dkv, 0, LIN_F32, w->raw + c_off);
+                if (a.gate) add(l.g, 0, LIN_F32, w->raw + g_off);
+                if (l.ff) { g.nw[1] = l.norm2; g.nvar = 2; add(l.up, 1, LIN_RELU2, w->h); }
+                GO(launch_gemv_seg(g, m, n, cfg));
+            }
+            {
+                SegGemvArgs g = seg(SEG_NORM, l.uq.pitch);
+                g.x = w->raw; g.width = a.q_rank; g.nw[0] = l.dq_norm; g.epi[0] = LIN_F32; g.out[0] = w->qf;
+                if (own) { g.has_kv = 1; g.kv = latent_rows(l, ldraw); }
+                const SegMat m[1] = {sm(l.uq)};
+                GO(launch_gemv_seg(g, m, 1, cfg));
+            }
+            if (int r = attention(l, a.gate ? w->raw + g_off : nullptr, ldraw)) return r;
+            {
+                SegGemvArgs g = seg(SEG_PLAIN, l.o.pitch + (l.ff ? l.down.pitch : 0));
+                g.xb[0] = (const bf16*)w->att; g.klen[0] = a.heads * l.vdimp; g.kp[0] = l.o.pitch;
+                if (l.ff) { g.xb[1] = (const bf16*)w->h; g.klen[1] = l.up.rows; g.kp[1] = l.down.pitch; }
+                g.epi[0] = LIN_ADD; g.out[0] = x;
+                const SegMat m[2] = {sm(l.o), sm(l.down)};
+                GO(launch_gemv_seg(g, m, l.ff ? 2 : 1, cfg));
+            }
+            if (sp.side_dim) {
+                SegGemvArgs g = seg(SEG_NARROW, l.side_gate.pitch);
+                const LinArgs e1 = side_args(i);
+                g.x = x; g.side = e1.side; g.side_pitch = e1.side_pitch; g.side_dim = e1.side_dim; g.epi[0] = LIN_GELU_SIDE; g.out[0] = w->sg;
+                const SegMat m[1] = {sm(l.side_gate)};
+                GO(launch_gemv_seg(g, m, 1, cfg));
+                SegGemvArgs p = seg(SEG_PLAIN, l.side_proj.pitch);
+                p.xb[0] = (const bf16*)w->sg; p.klen[0] = s->sidep; p.kp[0] = l.side_proj.pitch; p.epi[0] = LIN_F32; p.out[0] = w->y;
+                const SegMat m2[1] = {sm(l.side_proj)};
+                GO(launch_gemv_seg(p, m2, 1, cfg));
+                y_w = l.side_norm;
+            }
+        }
+        SegGemvArgs g = seg(SEG_NORM, s->head.pitch);
+        take_x(g);
+        g.nw[0] = s->final_norm; g.epi[0] = LIN_F32; g.out[0] = s->logits;
+        const SegMat m[1] = {sm(s->head)};
+        GO(launch_gemv_seg(g, m, 1, cfg));
+        s->dec_x = x;
         return CUQWEN_OK;
     }
     int narrow_x() { GO(launch_st_narrow(s->act, w->x, s->wp, w->xn1, s->wp, T, cfg)); return CUQWEN_OK; }
@@ -379,6 +506,7 @@ int stack_record_step(cuqwen_engine* e, const LaunchCfg& cfg, const std::functio
     Pass p{e, s, &s->dec, cfg, 1, true, &e->ctl->token, &e->ctl->pos, 0, &after};
     LaunchCfg plain = cfg; plain.pdl = false;
     if (int r = p.done(launch_st_embed_step(s->embed.w, s->embed.pitch, e->ctl, s->dec.x, s->spec.width, plain), "embedding")) return r;
+    if (s->act == ACT_BF16) return p.fused_layers();
     if (int r = p.layers(false)) return r;
     if (int r = p.norms(p.last_y(), p.last_y_w(), s->final_norm, nullptr)) return r;
     return p.done(launch_st_linear(s->act, p.lin(s->dec.xn1, s->wp, s->head, LIN_F32, s->logits, s->vocab_p), cfg), "head");
@@ -405,9 +533,8 @@ int stack_run_chunk(cuqwen_engine* e, int T, int pos0, const int* want, int n_wa
         NormRowsArgs a{};
         a.x = s->pf.x; a.ldx = s->wp; a.w[0] = s->final_norm; a.out[0] = s->xn_rows; a.ldo = s->wp; a.n_out = 1; a.width = s->spec.width; a.eps = (float)s->spec.norm_eps; a.rows = s->want_rows + i;
         if (int r = p.done(launch_st_norms(s->act, a, n, cfg), "final norm")) return r;
-        LinArgs h = p.lin(s->xn_rows, s->wp, s->head, LIN_F32, s->logits_rows, s->vocab_p);
-        h.T = n;
-        if (int r = p.done(launch_st_linear(s->act, h, cfg), "head")) return r;
+        const StMat* head[1] = {&s->head};
+        if (int r = p.product(LIN_F32, s->xn_rows, s->wp, head, 1, s->logits_rows, s->vocab_p, n)) return r;
         SK(cudaMemcpy2DAsync(logits_host + (size_t)i * s->spec.vocab, (size_t)s->spec.vocab * 4, s->logits_rows, (size_t)s->vocab_p * 4, (size_t)s->spec.vocab * 4, n, cudaMemcpyDeviceToHost, e->stream));
         SK(cudaStreamSynchronize(e->stream));
     }

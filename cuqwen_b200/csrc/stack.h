@@ -8,6 +8,8 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include <functional>
+
 #include "common.cuh"
 #include "launch.h"
 
@@ -87,9 +89,29 @@ struct LatentAttnArgs {
     const int* pos_ptr; int pos0;
 };
 int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg);
-// qn_abs[h] (float) = W_uk[h]^T qn[h]: the unrotated query against latents instead of keys.  wk: [heads * dimp][pitch].
-struct AbsorbArgs { const void* q; int q_hs; const bf16* wk; int pitch, heads, dim, dimp, kv_rank; void* out; int ldo; };
+// The same for bfloat16 portions on the tensor cores (latent_prefill_attn.cu), where the sizes fit: keys and values hold n_keys
+// rows from kbase on, kr the cache's cache_rows.
+bool latent_prefill_fits(int dn, int dr, int dv);
+int launch_latent_prefill_attn(const LatentAttnArgs& a, int n_keys, size_t cache_rows, unsigned* err, const LaunchCfg& cfg);
+// One token's queries as the cache rows are laid out: out[h] = [W_uk[h]^T q[h] (kv_rank) | rotated q[h] (rot_dim, from
+// kr_off)], so that a score is one dot product with a cache row.  q float [heads][q_hs], its rotated part from rot_off.
+struct AbsorbArgs {
+    const float* q; int q_hs, rot_off, rot_dim; const float2* rot; const int* pos_ptr;
+    const bf16* wk; int pitch, heads, dim, dimp; void* out; int ldo, kr_off;
+};
 int launch_absorb_q(int act, const AbsorbArgs& a, const LaunchCfg& cfg);
+// bfloat16 decode attention over cache rows, split over the keys (latent_decode.cu): partials, then one kernel that merges
+// them, multiplies with W_uv and applies the gate.
+struct LatentDecodeArgs {
+    const bf16* q; int crow;                             // [heads][crow], crow = kv_rank (padded) + rot_dim (padded)
+    const bf16* cache; int kvrp;                         // rows [crow]; the values are their first kvrp places
+    const float* sink; int heads, window; float scale; const int* pos_ptr;
+    int nsplit; float* part_o; float* part_ml;           // [nsplit][heads][kvrp], [nsplit][heads][2]
+    const bf16* wv; int pitch, vdim, vdimp, kv_rank; const float* gate; int g_hs; bf16* out; int o_hs;
+};
+// Splits that launch_latent_decode wants for a cache of max_seq rows; 0 = sizes it does not cover.
+int latent_decode_splits(int heads, int crow, int kvrp, int window, int max_seq, int sm_count);
+int launch_latent_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done);
 // att[h][v] = sigmoid(g[h][v]) * sum_r W_uv[h][v][r] o[h][r].  o float [heads][ldo].
 struct UvGateArgs { const float* o; int ldo; const bf16* wv; int pitch, heads, vdim, vdimp, kv_rank; const float* gate; int g_hs; void* out; int o_hs; };
 int launch_uv_gate(int act, const UvGateArgs& a, const LaunchCfg& cfg);

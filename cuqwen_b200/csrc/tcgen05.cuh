@@ -70,5 +70,7 @@ __device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t smem_addr, uint32_t
 __host__ __device__ constexpr uint32_t umma_idesc_f16(int m, int n, int b_mn_major) {
     return (1u << 4) | ((uint32_t)b_mn_major << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
 }
+// The same for bfloat16 operands: formats at [7,10) (A) and [10,13) (B), 1 = bf16.
+__host__ __device__ constexpr uint32_t umma_idesc_bf16(int m, int n, int b_mn_major) { return umma_idesc_f16(m, n, b_mn_major) | (1u << 7) | (1u << 10); }
 
 }  // namespace cq
