@@ -505,6 +505,9 @@ def run_sweep(a):
     if a.sweep == "prefill":
         run_prefill_sweep(a, rng)
         return
+    if a.sweep == "stack":
+        run_stack_sweep(a)
+        return
     if a.impl == "ours":
         if a.sweep == "gemv":
             rows = MB.single_gemv(4864, 896, "int4", 2000)
@@ -625,6 +628,84 @@ def run_prefill_sweep(a, rng):
           "how": "qwen_forward once per prompt token (src/main.cu:86-92): 32 calls at each of four positions, mean x prompt length"})
 
 
+# Layers of the sizes that the table's models have, for designs read from a model directory (--sweep stack): Falivik layers
+# with about as many weights as a layer of the table model named beside them.
+STACK_SIZES = {
+    "1.5b": dict(width=1536, heads=12, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, window=1024, ff=13440, side=128,
+                 table=dict(vocab=32000, dim=1536, inter=8960, heads=12, kv=2, hd=128, tied=False)),
+    "7b": dict(width=3584, heads=28, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=4096, ff=25600, side=256,
+               table=dict(vocab=32000, dim=3584, inter=18944, heads=28, kv=4, hd=128, tied=False)),
+}
+
+
+def stack_model(size: str, layers: int) -> Path:
+    """Random-weight model directory of the given layers (every second pair of layers shares its latents), made once."""
+    from cuqwen_b200 import stackfmt as F
+    z = STACK_SIZES[size]
+    base = Path("/dev/shm") if os.access("/dev/shm", os.W_OK) else Path("/tmp")
+    d = base / f"cuqwen_bench_falivik_{size}_L{layers}_seed{SEED}"
+    if not (d / "done").exists():
+        ls = [F.latent_layer(z["heads"], z["dim"], z["rot_dim"], z["vdim"], z["q_rank"], z["kv_rank"], z["window"], z["ff"], kv_from=i - 1 if i % 4 == 3 else None) for i in range(layers)]
+        cfg = F.falivik_config(z["table"]["vocab"], z["width"], z["side"], ls)
+        F.write_model_dir(d, cfg, F.random_weights(cfg, SEED, block=1 << 20))
+        (d / "done").touch()
+    return d
+
+
+def run_stack_sweep(a):
+    """--sweep stack: decode and prefill of a Falivik model in bfloat16 (random weights) beside the table's model of about
+    equal layers in fp16, both cut to the same number of layers (default 8) and the same vocabulary.  --stack picks the
+    size, --only one of the two arms (profiler runs)."""
+    from cuqwen_b200 import binfmt, build
+    from cuqwen_b200 import engine as E
+    z, nl, ctx, n, Kst = STACK_SIZES[a.stack], a.layers or 8, a.ctx, a.prompt, a.steps
+    hbm, _ = peaks()
+    tp = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    tf = float(tp.get("bf16_tflops", 1590.0))
+    toks = np.random.default_rng(SEED).integers(0, z["table"]["vocab"], size=max(n, ctx)).astype(np.int32)
+    W, H, t = z["width"], z["heads"], z["table"]
+
+    def measure(name, eng, fill, gemm_flop, attn_flop, step_bytes):
+        fill()
+        eng.prefill(toks[:min(n, 512)], 0)
+        with ClockSampler(0) as cs:
+            pms = []
+            for _ in range(a.repeat):
+                eng.prefill(toks[:n], 0)
+                pms.append(eng.last_decode_ms)
+            fill()
+            eng.decode_n(1234, ctx, max(a.warmup, 3))
+            eng.decode_n(1234, ctx, Kst)
+        ms, p = eng.last_decode_ms / Kst, min(pms)
+        emit({"sweep": "stack", "model": name, "layers": nl, "decode": {"ctx": ctx, "tok_s": round(1e3 / ms, 1), "ms_per_step": round(ms, 4), "launches": eng.step_launches, "algorithmic_bytes": step_bytes,
+              "gbs": round(step_bytes / ms / 1e6, 1), "frac_of_measured_hbm": round(step_bytes / ms / 1e6 / hbm, 4)},
+              "prefill": {"tokens": n, "ms": round(p, 3), "tok_s": round(n / p * 1e3, 1), "tflops": round((gemm_flop + attn_flop) / p / 1e9, 1),
+                          "frac_of_measured_bf16": round((gemm_flop + attn_flop) / p / 1e9 / tf, 4)},
+              "l2": "no flush: a step streams more weights than L2 holds", "clocks": cs.result})
+        eng.close()
+
+    if a.only in ("", "stack"):
+        d = stack_model(a.stack, nl)
+        eng = E.Engine.open(d, max_seq_len=max(n, ctx + Kst + 64))
+        keys = sum(min(i + 1, z["window"]) for i in range(n))
+        own = sum(1 for i in range(nl) if i % 4 != 3)
+        # every layer; the last one of a prefill without logits stops after its cache row (or before, when it shares one)
+        per = W * (z["q_rank"] + 2 * H * z["vdim"] + 2 * z["ff"] + 2 * z["side"]) + z["q_rank"] * H * (z["dim"] + z["rot_dim"]) + z["kv_rank"] * H * (z["dim"] + z["vdim"])
+        measure(f"Falivik {a.stack} layers, bfloat16", eng, lambda: eng.prefill(toks[:ctx], 0), 2.0 * n * ((nl - 1) * per + own * W * (z["kv_rank"] + z["rot_dim"])),
+                2.0 * keys * H * (z["dim"] + z["rot_dim"] + z["vdim"]) * (nl - 1), eng.step_bytes(ctx + Kst // 2))
+    if a.only in ("", "table"):
+        cfg = dict(t, layers=nl)
+        p = model_path(f"stack_{a.stack}", "fp16", nl)
+        if not p.exists():
+            build.build_gen()
+            subprocess.run([str(build.GEN_BIN), "--out", str(p), "--dims", *[str(cfg[k]) for k in ("vocab", "dim", "inter", "layers", "heads", "kv", "hd")], "--quant", "fp16", "--seed", str(SEED), "--untied"], check=True)
+        eng = E.Engine(E.custom_params(cfg["vocab"], cfg["dim"], cfg["inter"], nl, cfg["heads"], cfg["kv"], cfg["hd"], "fp16", max_seq_len=max(n, ctx + Kst + 64)))
+        eng.load(str(p))
+        qd, kd = cfg["heads"] * cfg["hd"], cfg["kv"] * cfg["hd"]
+        gemm = 2.0 * n * (nl * cfg["dim"] * (qd + 2 * kd) + (nl - 1) * (qd * cfg["dim"] + 3 * cfg["dim"] * cfg["inter"]))
+        measure(f"Qwen2.5 {a.stack} layers, fp16", eng, lambda: eng.kv_fill_normal(ctx, SEED), gemm, 4.0 * qd * (n * (n + 1) / 2) * (nl - 1), eng.step_bytes(ctx + Kst // 2))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -640,7 +721,11 @@ def main():
     ap.add_argument("--kv", default="fp16", choices=["fp16", "int8"], help="KV cache format (int8: opt-in 8-bit cache, outside the parity contract)")
     ap.add_argument("--no-parity", action="store_true")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers (profiler captures only; the JSON line says so)")
-    ap.add_argument("--sweep", default="", choices=["", "gemv", "attention", "prefill"], help="kernel-level sweeps of the other benchmark configurations")
+    ap.add_argument("--sweep", default="", choices=["", "gemv", "attention", "prefill", "stack"],
+                    help="kernel-level sweeps of the other benchmark configurations; stack: a model directory's design beside the table's closest model")
+    ap.add_argument("--stack", default="7b", choices=sorted(STACK_SIZES), help="--sweep stack: layer size")
+    ap.add_argument("--only", default="", choices=["", "stack", "table"], help="--sweep stack: one arm only")
+    ap.add_argument("--repeat", type=int, default=3, help="--sweep stack: timed prefills (the best counts)")
     a = ap.parse_args()
     # Libraries (NCCL's version banner, for one) write to file descriptor 1.  Keep the real stdout aside for the one
     # JSON line and send everything else to stderr.

@@ -70,49 +70,68 @@ int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg) {
 }
 
 // One head's query against the latents: its unrotated part carried through W_uk, its rotated part rotated, side by side as
-// the cache rows are.  CTA = (head, 256 latent columns): a warp walks every fourth row of the head's W_uk, eight columns a
-// lane; the head's first CTA also rotates.
+// the cache rows are.  CTA = (head, 64 latent columns): eight lanes hold a row segment, thirty-two row groups walk the
+// head's rows of W_uk; the first four segments of a thread are on their way before the dependency wait (the weights do not
+// depend on the step).  The head's first CTA also rotates.
+constexpr int kAqThreads = 256, kAqCols = 64, kAqPre = 4;
 template <typename A>
-__global__ void __launch_bounds__(128) absorb_q_kernel(const AbsorbArgs a) {
-    __shared__ float part[3][256];
-    pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.x, lane = threadIdx.x & 31, c0 = blockIdx.y * 256 + lane * 8, grp = threadIdx.x >> 5;
+__global__ void __launch_bounds__(kAqThreads) absorb_q_kernel(const AbsorbArgs a) {
+    __shared__ float part[8][kAqCols];
+    pdl_launch_dependents();
+    const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, cl = (lane & 7) * 8, c0 = blockIdx.y * kAqCols + cl, grp = threadIdx.x >> 3;
+    const bf16* w = a.wk + (size_t)h * a.dimp * a.pitch + c0;
+    const bool live = c0 < a.kr_off;                     // kr_off = the padded latent length, a multiple of eight within the pitch
+    uint4 pre[kAqPre];
+#pragma unroll
+    for (int i = 0; i < kAqPre; ++i) pre[i] = live && grp + 32 * i < a.dim ? ldg_stream(w + (size_t)(grp + 32 * i) * a.pitch) : make_uint4(0u, 0u, 0u, 0u);
+    pdl_wait();
     const float* q = a.q + (size_t)h * a.q_hs;
     A* out = reinterpret_cast<A*>(a.out) + (size_t)h * a.ldo;
     if (blockIdx.y == 0) {
         const int half = a.rot_dim / 2, pos = *a.pos_ptr;
-        for (int i = threadIdx.x; i < half; i += 128) {
+        for (int i = threadIdx.x; i < half; i += kAqThreads) {
             const float2 cs = a.rot[(size_t)pos * half + i];
             const float u = __ldcg(q + a.rot_off + i), v = __ldcg(q + a.rot_off + half + i);
             out[a.kr_off + i] = to_act<A>(u * cs.x - v * cs.y);
             out[a.kr_off + half + i] = to_act<A>(v * cs.x + u * cs.y);
         }
     }
-    const bf16* w = a.wk + (size_t)h * a.dimp * a.pitch + c0;
     float s[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (c0 < a.kr_off)                                   // kr_off = the padded latent length, a multiple of eight within the pitch
-#pragma unroll 8
-        for (int d = grp; d < a.dim; d += 4) {
+    float qd[kAqPre];
+#pragma unroll
+    for (int i = 0; i < kAqPre; ++i) qd[i] = grp + 32 * i < a.dim ? __ldcg(q + grp + 32 * i) : 0.f;
+#pragma unroll
+    for (int i = 0; i < kAqPre; ++i) {
+        float v[8];
+        unpack8(pre[i], v);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) s[k] = fmaf(qd[i], v[k], s[k]);
+    }
+    if (live)
+        for (int d = grp + 32 * kAqPre; d < a.dim; d += 32) {
             float v[8];
             load8(w + (size_t)d * a.pitch, v);
-            const float qd = __ldcg(q + d);
+            const float f = __ldcg(q + d);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) s[i] = fmaf(qd, v[i], s[i]);
+            for (int k = 0; k < 8; ++k) s[k] = fmaf(f, v[k], s[k]);
         }
-    if (grp > 0)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) part[grp - 1][lane * 8 + i] = s[i];
+    for (int k = 0; k < 8; ++k) {
+        s[k] += __shfl_xor_sync(0xffffffffu, s[k], 8);
+        s[k] += __shfl_xor_sync(0xffffffffu, s[k], 16);
+        if (lane < 8) part[warp][cl + k] = s[k];
+    }
     __syncthreads();
-    if (grp == 0 && c0 < a.kr_off)
+    if (threadIdx.x < kAqCols && blockIdx.y * kAqCols + threadIdx.x < a.kr_off) {
+        float v = 0.f;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int j = lane * 8 + i;
-            out[c0 + i] = to_act<A>(s[i] + part[0][j] + part[1][j] + part[2][j]);
-        }
+        for (int k = 0; k < 8; ++k) v += part[k][threadIdx.x];
+        out[blockIdx.y * kAqCols + threadIdx.x] = to_act<A>(v);
+    }
 }
 int launch_absorb_q(int act, const AbsorbArgs& a, const LaunchCfg& cfg) {
-    const dim3 grid(a.heads, (a.kr_off + 255) / 256);
-    return act == ACT_F32 ? st_launch(absorb_q_kernel<float>, grid, dim3(128), 0, cfg, a) : st_launch(absorb_q_kernel<bf16>, grid, dim3(128), 0, cfg, a);
+    const dim3 grid(a.heads, (a.kr_off + kAqCols - 1) / kAqCols);
+    return act == ACT_F32 ? st_launch(absorb_q_kernel<float>, grid, dim3(kAqThreads), 0, cfg, a) : st_launch(absorb_q_kernel<bf16>, grid, dim3(kAqThreads), 0, cfg, a);
 }
 
 // A warp per output value.

@@ -5,8 +5,9 @@
 // (cp.async, two buffers; rows of earlier steps are requested before the dependency wait), scores on mma.sync m16n8k16 with
 // the sixteen heads as the M rows - warp w takes keys 8 w .. 8 w + 7 of the tile - an online softmax in float32 over the
 // tile, then P V with the columns of the latent dealt over the warps.  Un-normalised partials and (max, sum) per head go out.
-// latent_fold_kernel: grid (heads, slices of 32 value rows): merges the ranges and the sink, multiplies the head's latent
-// output with W_uv, applies the gate.
+// latent_fold_kernel: grid (heads, slices of 32 value rows): merges the ranges and the sink - up to eight slices of a head
+// form a cluster whose CTAs merge a share of the columns each and exchange them through distributed shared memory -
+// multiplies the head's latent output with W_uv, applies the gate.
 #include "stack_dev.cuh"
 #include "tma.cuh"
 
@@ -192,8 +193,11 @@ __global__ void __launch_bounds__(256) latent_fold_kernel(const LatentDecodeArgs
     extern __shared__ float lf_smem[];          // [kvrp] the head's latent output
     __shared__ float wgt[kLdMaxSplit];
     __shared__ float red[16];
+    __shared__ __align__(16) float mrg[8][128];
     const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_launch_dependents();
+    const int ncl = gridDim.y == a.ncl ? a.ncl : 1, rank = ncl > 1 ? (int)blockIdx.y : 0;
+    if (ncl > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // waited for before the first store to another CTA: by then all have started
     // the weights do not depend on the step: on their way before the wait (four rows a warp, two 16-byte units a lane)
     uint4 w[4][2];
     const int v0 = blockIdx.y * kLfRows + warp * 4;
@@ -203,6 +207,18 @@ __global__ void __launch_bounds__(256) latent_fold_kernel(const LatentDecodeArgs
         for (int j = 0; j < 2; ++j)
             w[i][j] = v0 + i < a.vdim && lane + 32 * j < a.kvrp / 8 ? ldg_stream(a.wv + (size_t)(h * a.vdimp + v0 + i) * a.pitch + (lane + 32 * j) * 8) : make_uint4(0u, 0u, 0u, 0u);
     pdl_wait();
+    // This CTA's columns of the merged output, 128 at a time: a lane four columns, a warp every eighth key range; every CTA of
+    // the cluster receives them.  The partials are requested together with the ranges' (max, sum); those of an empty range are
+    // whatever an earlier step left (finite) and get the weight zero.
+    const int cw = ((a.kvrp + ncl - 1) / ncl + 127) / 128 * 128;
+    const float* po = a.part_o + (size_t)h * a.kvrp;
+    const size_t ps = (size_t)a.heads * a.kvrp;
+    float4 pre[8];
+    {
+        const int c = rank * cw + lane * 4;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) pre[k] = c < a.kvrp && warp + 8 * k < a.nsplit ? __ldcg(reinterpret_cast<const float4*>(po + (warp + 8 * k) * ps + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     float m = -INFINITY, l = 0.f;
     if (tid < a.nsplit) {
         const float2 v = __ldcg(reinterpret_cast<const float2*>(a.part_ml) + (size_t)tid * a.heads + h);
@@ -226,14 +242,37 @@ __global__ void __launch_bounds__(256) latent_fold_kernel(const LatentDecodeArgs
 #pragma unroll
     for (int i = 0; i < 8; ++i) den += red[8 + i];
     const float inv = 1.0f / den;
-    for (int c = tid; c < a.kvrp; c += 256) {
-        const float* po = a.part_o + (size_t)h * a.kvrp + c;
-        float o = 0.f;
-#pragma unroll 8
-        for (int k = 0; k < a.nsplit; ++k) if (wgt[k] != 0.f) o = fmaf(wgt[k], __ldcg(po + (size_t)k * a.heads * a.kvrp), o);
-        lf_smem[c] = o * inv;
+    if (ncl > 1) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    for (int cb = rank * cw; cb < (rank + 1) * cw && cb < a.kvrp; cb += 128) {
+        const int c = cb + lane * 4;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (cb != rank * cw) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k) pre[k] = c < a.kvrp && warp + 8 * k < a.nsplit ? __ldcg(reinterpret_cast<const float4*>(po + (warp + 8 * k) * ps + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        auto acc = [&](float f, float4 v) { o.x = fmaf(f, v.x, o.x); o.y = fmaf(f, v.y, o.y); o.z = fmaf(f, v.z, o.z); o.w = fmaf(f, v.w, o.w); };
+#pragma unroll
+        for (int k = 0; k < 8; ++k) if (warp + 8 * k < a.nsplit) acc(wgt[warp + 8 * k], pre[k]);
+        if (c < a.kvrp)
+            for (int k = warp + 64; k < a.nsplit; k += 8) acc(wgt[k], __ldcg(reinterpret_cast<const float4*>(po + k * ps + c)));
+        reinterpret_cast<float4*>(mrg[warp])[lane] = o;
+        __syncthreads();
+        if (tid < 128 && cb + tid < a.kvrp) {
+            float v = 0.f;
+#pragma unroll
+            for (int k = 0; k < 8; ++k) v += mrg[k][tid];
+            v *= inv;
+            if (ncl == 1) lf_smem[cb + tid] = v;
+            else
+                for (int r = 0; r < ncl; ++r) {
+                    uint32_t dst;
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(smem_u32(lf_smem + cb + tid)), "r"(r));
+                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(v) : "memory");
+                }
+        }
+        __syncthreads();
     }
-    __syncthreads();
+    if (ncl > 1) asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int v = v0 + i;
@@ -286,7 +325,18 @@ static int ld_go(const LatentDecodeArgs& a, const LaunchCfg& cfg) {
 int launch_latent_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done) {
     if (a.crow % 8 || a.kvrp % 8 || a.kvrp > 1024 || a.nsplit < 1 || a.nsplit > kLdMaxSplit || a.heads < 1) return done((int)cudaErrorInvalidValue, "latent_decode");
     if (int r = done(a.kvrp <= 128 ? ld_go<1>(a, cfg) : a.kvrp <= 512 ? ld_go<4>(a, cfg) : ld_go<8>(a, cfg), "latent_partial")) return r;
-    return done(st_launch(latent_fold_kernel, dim3(a.heads, (a.vdim + kLfRows - 1) / kLfRows), dim3(256), (size_t)a.kvrp * 4, cfg, a), "latent_fold");
+    const int slices = (a.vdim + kLfRows - 1) / kLfRows;
+    LatentDecodeArgs f = a;
+    f.ncl = slices <= 8 ? slices : 1;
+    cudaLaunchConfig_t lc = {};
+    lc.gridDim = dim3(a.heads, slices); lc.blockDim = dim3(256); lc.dynamicSmemBytes = (size_t)a.kvrp * 4; lc.stream = cfg.stream;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = 1; at[0].val.clusterDim.y = f.ncl; at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    lc.attrs = at; lc.numAttrs = cfg.pdl ? 2 : 1;
+    return done((int)cudaLaunchKernelEx(&lc, latent_fold_kernel, f), "latent_fold");
 }
 
 }  // namespace cq

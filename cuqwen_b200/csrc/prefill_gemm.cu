@@ -107,7 +107,7 @@ template <int Q, int NT>
 __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __grid_constant__ PfGemmArgs a) {
     extern __shared__ unsigned char pf_smem_raw[];
     const uint32_t base = (smem_u32(pf_smem_raw) + 1023u) & ~1023u;
-    constexpr int NA = pf_na(Q), NB = pf_nb(Q), kRawBytes = pf_raw_bytes(Q, NT), kPfBBytes = NT * 128;
+    constexpr int NA = pf_na(Q, NT), NB = pf_nb(Q, NT), kRawBytes = pf_raw_bytes(Q, NT), kPfBBytes = NT * 128;
     constexpr bool kRaw = Q == Q_I4 || Q == Q_I8;              // weights that are widened on the way
     constexpr uint32_t kPfIdesc = Q == Q_BF16 ? umma_idesc_bf16(kPfM, NT, 0) : umma_idesc_f16(kPfM, NT, 0);
     constexpr int kASlot = kPfMH * kPfABytes;                  // X tiles of one slot
@@ -387,10 +387,11 @@ int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     a.mh = a.T > kPfM ? kPfMH : 1;
-    const int mtiles = (a.T + kPfM * a.mh - 1) / (kPfM * a.mh);
+    int mtiles = (a.T + kPfM * a.mh - 1) / (kPfM * a.mh);
     int wide = 0;
     for (int i = 0; i < nmat; ++i) wide += (m[i].rows + kPfN - 1) / kPfN;
     const int nt = (sms > 0 && wide * mtiles * 4 <= sms) ? kPfN / 4 : (sms > 0 && wide * mtiles * 2 <= sms) ? kPfN / 2 : kPfN;
+    if (nt == kPfN / 4 && a.mh == 2) { a.mh = 1; mtiles = (a.T + kPfM - 1) / kPfM; }       // few rows: a token half per CTA, twice the CTAs
     const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
     if (int r = pf_map(&a.tx, x, bf, 2, (size_t)a.T, (size_t)a.K, kPfKB, kPfM, true, (size_t)ldx)) return r;
     int tiles = 0;

@@ -34,10 +34,10 @@ constexpr int kPfABytes = kPfM * 128;          // one X tile of a stage
 // cover, so their ring is the deep one; a widened B tile is consumed by the very next MMAs, two slots suffice.
 // fp16 weights have no raw form: their B tile arrives by TMA, NB = NA.
 __host__ __device__ constexpr int pf_raw_bytes(int quant, int nt) { return quant == 2 ? nt * 32 : quant == 1 ? nt * 64 : 0; }
-__host__ __device__ constexpr int pf_na(int quant) { return quant == 2 ? 4 : 3; }
-__host__ __device__ constexpr int pf_nb(int quant) { return quant == 0 || quant == 3 ? 3 : 2; }
+__host__ __device__ constexpr int pf_na(int quant, int nt = kPfN) { return quant == 3 ? (nt == 256 ? 3 : nt == 128 ? 4 : 5) : quant == 2 ? 4 : 3; }      // bfloat16: narrow tiles leave room for more
+__host__ __device__ constexpr int pf_nb(int quant, int nt = kPfN) { return quant == 3 ? pf_na(3, nt) : quant == 0 ? 3 : 2; }
 __host__ __device__ constexpr int pf_smem_bytes(int quant, int nt) {
-    return pf_na(quant) * (kPfMH * kPfABytes + pf_raw_bytes(quant, nt)) + pf_nb(quant) * nt * 128 + 1024 /* alignment slack */ + 256 /* barriers, TMEM address */;
+    return pf_na(quant, nt) * (kPfMH * kPfABytes + pf_raw_bytes(quant, nt)) + pf_nb(quant, nt) * nt * 128 + 1024 /* alignment slack */ + 256 /* barriers, TMEM address */;
 }
 
 enum PfMode : int {

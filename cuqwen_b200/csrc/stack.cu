@@ -384,16 +384,23 @@ struct Pass {
             if (stop && !own) return CUQWEN_OK;
             if (int r = norms(y, y_w, l.norm1, l.ff && !stop ? l.norm2 : nullptr)) return r;
             const int c_off = l.qrp, g_off = c_off + (own ? l.crow : 0), ldraw = g_off + (a.gate ? a.heads * l.vdimp : 0);
+            if (stop) {
+                const StMat* kv[1] = {&l.dkv};
+                if (int r = product(LIN_F32, w->xn1, s->wp, kv, 1, w->raw + c_off, ldraw, T)) return r;
+                LatentRowsArgs lr = latent_rows(l, ldraw);
+                lr.dq = nullptr;
+                GO(launch_st_latent_rows(s->act, lr, T, cfg));
+                return CUQWEN_OK;
+            }
             const StMat* first[3]; int nf = 0;
             first[nf++] = &l.dq;
             if (own) first[nf++] = &l.dkv;
-            if (a.gate && !stop) first[nf++] = &l.g;
+            if (a.gate) first[nf++] = &l.g;
             if (int r = product(LIN_F32, w->xn1, s->wp, first, nf, w->raw, ldraw, T)) return r;
             const StMat *up[1] = {&l.up}, *uq[1] = {&l.uq}, *o[1] = {&l.o}, *sg[1] = {&l.side_gate}, *sp1[1] = {&l.side_proj};
-            if (l.ff && !stop) if (int r = product(LIN_RELU2, w->xn2, s->wp, up, 1, w->h, l.up.rows, T)) return r;
+            if (l.ff) if (int r = product(LIN_RELU2, w->xn2, s->wp, up, 1, w->h, l.up.rows, T)) return r;
             LatentRowsArgs lr = latent_rows(l, ldraw);
             GO(launch_st_latent_rows(s->act, lr, T, cfg));
-            if (stop) return CUQWEN_OK;
             if (int r = product(LIN_F32, w->cq, l.qrp, uq, 1, w->qf, l.uq.rows, T)) return r;
             if (int r = attention(l, a.gate ? w->raw + g_off : nullptr, ldraw)) return r;
             if (int r = product(LIN_ADD, w->att, a.heads * l.vdimp, o, 1, w->x, s->wp, T, w->h, l.up.rows, l.ff ? &l.down : nullptr)) return r;

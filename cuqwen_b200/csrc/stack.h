@@ -40,7 +40,7 @@ int launch_st_narrow(int act, const float* x, int ldx, void* out, int ldo, int T
 // Per row: the query latent and the cache row of a token from the raw projections.
 //   cq[t] = dq / rms(dq) * dq_w;  cache row pos = [ckv / rms(ckv) * dkv_w | rotated key part]
 struct LatentRowsArgs {
-    const float* dq; int ld; const float* dq_w; void* cq; int ldcq; int q_rank;
+    const float* dq; int ld; const float* dq_w; void* cq; int ldcq; int q_rank;      // dq null: only the cache row
     const float* dkv;                                   // null: the layer has no latent projection of its own
     const float* dkv_w; void* cache; int ldc, kv_rank, kr_off, rot_dim;      // kr_off: where the rotated part starts, in dkv rows and in cache rows
     const float2* rot;                                  // (cos, sin) [position][rot_dim / 2]
@@ -107,6 +107,7 @@ struct LatentDecodeArgs {
     const bf16* cache; int kvrp;                         // rows [crow]; the values are their first kvrp places
     const float* sink; int heads, window; float scale; const int* pos_ptr;
     int nsplit; float* part_o; float* part_ml;           // [nsplit][heads][kvrp], [nsplit][heads][2]
+    int ncl;                                             // set by the launcher: CTAs of a head that share the merge
     const bf16* wv; int pitch, vdim, vdimp, kv_rank; const float* gate; int g_hs; bf16* out; int o_hs;
 };
 // Splits that launch_latent_decode wants for a cache of max_seq rows; 0 = sizes it does not cover.

@@ -26,6 +26,10 @@ __device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
 }
 __device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), v); }
 
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf(v.x, v.y), pack_bf(v.z, v.w)); }
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w; }
+
 // Sum over the CTA, returned to every thread.  `red`: 33 floats of shared memory; safe to call again at once.
 __device__ __forceinline__ float cta_sum(float v, float* red) {
     v = warp_sum(v);

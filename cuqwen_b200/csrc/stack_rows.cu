@@ -4,7 +4,12 @@
 namespace cq {
 
 __device__ __forceinline__ void embed_row(const bf16* src, float* dst, int width) {
-    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = __bfloat162float(src[i]);
+    for (int i = threadIdx.x; i < (width + 7) / 8; i += blockDim.x) {      // rows are padded with zeros to a multiple of eight
+        float v[8];
+        unpack8(ldg_stream(src + 8 * i), v);
+        store4(dst + 8 * i, make_float4(v[0], v[1], v[2], v[3]));
+        store4(dst + 8 * i + 4, make_float4(v[4], v[5], v[6], v[7]));
+    }
 }
 __global__ void __launch_bounds__(256) st_embed_kernel(const bf16* __restrict__ table, int pitch, const int* __restrict__ tokens, float* __restrict__ x, int ldx, int width) {
     pdl_launch_dependents(); pdl_wait();
@@ -32,32 +37,67 @@ int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, i
 }
 
 // ---- x += rmsnorm(y), then one or two norms of x ------------------------------------------------------------------------
-// One CTA per row; a thread keeps its elements (one in 256) in registers up to a width of 8192 and re-reads them beyond.
-template <typename A>
+// One CTA per row, the row in registers: a thread owns the float4 units tid, tid + 256, ... (NV of them at the most; rows are
+// padded with zeros to a multiple of eight).  NV = 0: any width, the row re-read from memory instead.
+template <typename A, int NV>
 __global__ void __launch_bounds__(256) st_norms_kernel(const NormRowsArgs a) {
     __shared__ float red[40];
     pdl_launch_dependents(); pdl_wait();
-    const int t = blockIdx.x;
-    float* x = a.x + (size_t)(a.rows ? a.rows[t] : t) * a.ldx;
-    if (a.y) {
-        const float* y = a.y + (size_t)t * a.ldy;
-        float ss = 0.f;
-        for (int i = threadIdx.x; i < a.width; i += 256) ss += y[i] * y[i];
-        const float inv = inv_rms(cta_sum(ss, red), a.width, a.eps);
-        for (int i = threadIdx.x; i < a.width; i += 256) x[i] += y[i] * inv * a.y_w[i];      // the same thread reads it below
+    const int t = blockIdx.x, tid = threadIdx.x, n4 = (a.width + 3) / 4, o4 = a.ldo / 4;
+    float4* x = reinterpret_cast<float4*>(a.x + (size_t)(a.rows ? a.rows[t] : t) * a.ldx);
+    const float4* y = a.y ? reinterpret_cast<const float4*>(a.y + (size_t)t * a.ldy) : nullptr;
+    constexpr int N = NV > 0 ? NV : 1;
+    float4 v[N];
+    float ss = 0.f;
+    if (NV > 0) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = i * 256 + tid < n4 ? x[i * 256 + tid] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (y) {
+        const float4* yw = reinterpret_cast<const float4*>(a.y_w);
+        auto add = [&](float4 p, float4 u, float inv, float4 w) { return make_float4(p.x + u.x * inv * w.x, p.y + u.y * inv * w.y, p.z + u.z * inv * w.z, p.w + u.w * inv * w.w); };
+        float sy = 0.f;
+        if (NV > 0) {
+            float4 u[N];
+#pragma unroll
+            for (int i = 0; i < N; ++i) { u[i] = i * 256 + tid < n4 ? y[i * 256 + tid] : make_float4(0.f, 0.f, 0.f, 0.f); sy += dot4(u[i], u[i]); }
+            const float inv = inv_rms(cta_sum(sy, red), a.width, a.eps);
+#pragma unroll
+            for (int i = 0; i < N; ++i) if (i * 256 + tid < n4) { v[i] = add(v[i], u[i], inv, yw[i * 256 + tid]); x[i * 256 + tid] = v[i]; }
+        } else {
+            for (int i = tid; i < n4; i += 256) sy += dot4(y[i], y[i]);
+            const float inv = inv_rms(cta_sum(sy, red), a.width, a.eps);
+            for (int i = tid; i < n4; i += 256) x[i] = add(x[i], y[i], inv, yw[i]);          // the same thread reads it below
+        }
     }
     if (a.n_out == 0) return;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < a.width; i += 256) ss += x[i] * x[i];
+    if (NV > 0) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) ss += dot4(v[i], v[i]);
+    } else for (int i = tid; i < n4; i += 256) ss += dot4(x[i], x[i]);
     const float inv = inv_rms(cta_sum(ss, red), a.width, a.eps);
     for (int k = 0; k < a.n_out; ++k) {
         A* o = reinterpret_cast<A*>(a.out[k]) + (size_t)t * a.ldo;
-        for (int i = threadIdx.x; i < a.ldo; i += 256) o[i] = to_act<A>(i < a.width ? x[i] * inv * a.w[k][i] : 0.f);
+        const float4* w = reinterpret_cast<const float4*>(a.w[k]);
+        auto put = [&](int i, float4 p) {
+            if (i < n4) { const float4 g = w[i]; p = make_float4(p.x * inv * g.x, p.y * inv * g.y, p.z * inv * g.z, p.w * inv * g.w); }
+            if (i < o4) store4(o + 4 * i, p);
+        };
+        if (NV > 0) {
+#pragma unroll
+            for (int i = 0; i < N; ++i) put(i * 256 + tid, v[i]);
+        } else for (int i = tid; i < o4; i += 256) put(i, i < n4 ? x[i] : make_float4(0.f, 0.f, 0.f, 0.f));
     }
 }
-int launch_st_norms(int act, const NormRowsArgs& a, int T, const LaunchCfg& cfg) {
-    return act == ACT_F32 ? st_launch(st_norms_kernel<float>, dim3(T), dim3(256), 0, cfg, a) : st_launch(st_norms_kernel<bf16>, dim3(T), dim3(256), 0, cfg, a);
+template <typename A>
+static int go_norms(const NormRowsArgs& a, int T, const LaunchCfg& cfg) {
+    const int nv = (a.ldo > a.width ? a.ldo : a.width) / 4;
+    if (nv <= 2 * 256) return st_launch(st_norms_kernel<A, 2>, dim3(T), dim3(256), 0, cfg, a);
+    if (nv <= 4 * 256) return st_launch(st_norms_kernel<A, 4>, dim3(T), dim3(256), 0, cfg, a);
+    if (nv <= 8 * 256) return st_launch(st_norms_kernel<A, 8>, dim3(T), dim3(256), 0, cfg, a);
+    return st_launch(st_norms_kernel<A, 0>, dim3(T), dim3(256), 0, cfg, a);
 }
+int launch_st_norms(int act, const NormRowsArgs& a, int T, const LaunchCfg& cfg) { return act == ACT_F32 ? go_norms<float>(a, T, cfg) : go_norms<bf16>(a, T, cfg); }
 
 template <typename A>
 __global__ void __launch_bounds__(256) st_narrow_kernel(const float* __restrict__ x, int ldx, A* __restrict__ out, int ldo) {
@@ -69,38 +109,41 @@ int launch_st_narrow(int act, const float* x, int ldx, void* out, int ldo, int T
 }
 
 // ---- query latent and cache row ---------------------------------------------------------------------------------------
+// One CTA of 128 threads per (row, half): blockIdx.y 0 the query latent, 1 the cache row.  A row of up to 2048 values stays in
+// registers (four float4 units a thread), a longer one is re-read.
 template <typename A>
-__global__ void __launch_bounds__(256) st_latent_rows_kernel(const LatentRowsArgs a) {
+__global__ void __launch_bounds__(128) st_latent_rows_kernel(const LatentRowsArgs a) {
     __shared__ float red[40];
     pdl_launch_dependents(); pdl_wait();
-    const int t = blockIdx.x;
-    if (blockIdx.y == 0) {
-        const float* q = a.dq + (size_t)t * a.ld;
-        float ss = 0.f;
-        for (int i = threadIdx.x; i < a.q_rank; i += 256) ss += q[i] * q[i];
-        const float inv = inv_rms(cta_sum(ss, red), a.q_rank, a.eps);
-        A* o = reinterpret_cast<A*>(a.cq) + (size_t)t * a.ldcq;
-        for (int i = threadIdx.x; i < a.ldcq; i += 256) o[i] = to_act<A>(i < a.q_rank ? q[i] * inv * a.dq_w[i] : 0.f);
-    } else {
-        const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
-        const float* kv = a.dkv + (size_t)t * a.ld;
-        float ss = 0.f;
-        for (int i = threadIdx.x; i < a.kv_rank; i += 256) ss += kv[i] * kv[i];
-        const float inv = inv_rms(cta_sum(ss, red), a.kv_rank, a.eps);
-        A* o = reinterpret_cast<A*>(a.cache) + (size_t)pos * a.ldc;
-        for (int i = threadIdx.x; i < a.kv_rank; i += 256) o[i] = to_act<A>(kv[i] * inv * a.dkv_w[i]);
-        const int half = a.rot_dim / 2;
-        for (int i = threadIdx.x; i < half; i += 256) {
-            const float2 cs = a.rot[(size_t)pos * half + i];
-            const float u = kv[a.kr_off + i], v = kv[a.kr_off + half + i];
-            o[a.kr_off + i] = to_act<A>(u * cs.x - v * cs.y);
-            o[a.kr_off + half + i] = to_act<A>(v * cs.x + u * cs.y);
-        }
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const bool kv = a.dq == nullptr || blockIdx.y == 1;
+    const int n = kv ? a.kv_rank : a.q_rank, n4 = (n + 3) / 4;
+    const float* src = (kv ? a.dkv : a.dq) + (size_t)t * a.ld;
+    const float4 *s4 = reinterpret_cast<const float4*>(src), *w4 = reinterpret_cast<const float4*>(kv ? a.dkv_w : a.dq_w);
+    const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
+    A* o = kv ? reinterpret_cast<A*>(a.cache) + (size_t)pos * a.ldc : reinterpret_cast<A*>(a.cq) + (size_t)t * a.ldcq;
+    float4 v[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { v[i] = i * 128 + tid < n4 ? s4[i * 128 + tid] : make_float4(0.f, 0.f, 0.f, 0.f); ss += dot4(v[i], v[i]); }
+    for (int i = 512 + tid; i < n4; i += 128) ss += dot4(s4[i], s4[i]);
+    const float inv = inv_rms(cta_sum(ss, red), n, a.eps);
+    auto put = [&](int i, float4 p) { const float4 g = w4[i]; store4(o + 4 * i, make_float4(p.x * inv * g.x, p.y * inv * g.y, p.z * inv * g.z, p.w * inv * g.w)); };
+#pragma unroll
+    for (int i = 0; i < 4; ++i) if (i * 128 + tid < n4) put(i * 128 + tid, v[i]);
+    for (int i = 512 + tid; i < n4; i += 128) put(i, s4[i]);
+    if (!kv) return;
+    const int half = a.rot_dim / 2;
+    for (int i = tid; i < half; i += 128) {
+        const float2 cs = a.rot[(size_t)pos * half + i];
+        const float p = src[a.kr_off + i], q = src[a.kr_off + half + i];
+        o[a.kr_off + i] = to_act<A>(p * cs.x - q * cs.y);
+        o[a.kr_off + half + i] = to_act<A>(q * cs.x + p * cs.y);
     }
 }
 int launch_st_latent_rows(int act, const LatentRowsArgs& a, int T, const LaunchCfg& cfg) {
-    const dim3 grid(T, a.dkv ? 2 : 1);
-    return act == ACT_F32 ? st_launch(st_latent_rows_kernel<float>, grid, dim3(256), 0, cfg, a) : st_launch(st_latent_rows_kernel<bf16>, grid, dim3(256), 0, cfg, a);
+    const dim3 grid(T, a.dkv && a.dq ? 2 : 1);
+    return act == ACT_F32 ? st_launch(st_latent_rows_kernel<float>, grid, dim3(128), 0, cfg, a) : st_launch(st_latent_rows_kernel<bf16>, grid, dim3(128), 0, cfg, a);
 }
 
 // ---- rotation of the query heads --------------------------------------------------------------------------------------
