@@ -81,6 +81,11 @@ SIGNATURES = {
     "cuqwen_k_penalty": (_i, [_i, _vp, _vp, _vp, _i, _f, _vp]),
     "cuqwen_k_argmax": (_i, [_i, _vp, _vp, _i, _vp]),
     "cuqwen_k_dequant": (_i, [_i, _i, _vp, _vp, _vp, _l, _l]),
+    "cuqwen_k_linear": (_i, [_i, _i, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _vp, _i, _i, _vp]),
+    "cuqwen_k_norm_rows": (_i, [_i, _i, _vp, _i] + [_vp] * 6 + [_i, _i, _f, _i]),
+    "cuqwen_k_latent_rows": (_i, [_i, _i, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _f, _i, _i]),
+    "cuqwen_k_rot_table": (_i, [_i, _vp, _i, _i, C.c_double]),
+    "cuqwen_k_latent_attention": (_i, [_i, _i, _i] + [_vp] * 7 + [_i] * 8 + [_f]),
     "cuqwen_strerror": (C.c_char_p, [_i]),
     "cuqwen_last_error": (C.c_char_p, []),
 }

@@ -24,6 +24,8 @@
 #include "launch.h"
 #include "prefill.cuh"
 #include "prefill_gemm.cuh"
+#include "gemv_seg.cuh"
+#include "stack.h"
 #include "stack_host.h"
 #include "tp_plan.h"
 
@@ -1299,5 +1301,93 @@ extern "C" int cuqwen_k_tp_sum(int device, const void* x, void* x_next, const vo
         return fail(CUQWEN_ERR_ARG, "unsupported tp_sum arguments");
     NOT_NULL(x, x_next, slots, d_step_no);
     KK(launch_tp_sum((const __half*)x, (__half*)x_next, slots, n_ranks, dim, d_step_no, seq_index, t_err, wait_cycles, cfg));
+    return CUQWEN_OK;
+}
+
+// ---- kernels of the layer-list designs ----------------------------------------------------------------------------------
+static bool bad_act(int act) { return act != CUQWEN_ACT_BF16 && act != CUQWEN_ACT_F32; }
+extern "C" int cuqwen_k_linear(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, const void* x2, int ldx2, const void* w2, int pitch2,
+                               int cols2, int n_tokens, int rows, void* out, int ldo, const void* side, int side_pitch, int side_dim, const int* d_tokens) {
+    DEV(device);
+    NOT_NULL(x, w, out);
+    if (bad_act(act) || epi < LIN_F32 || epi > LIN_GELU_SIDE || n_tokens < 1 || rows < 8 || rows % 8 || cols < 8 || cols % 8 || pitch % 128 || pitch < cols || ldx % 8 || ldx < cols || ldo % 8 || ldo < rows)
+        return fail(CUQWEN_ERR_ARG, "linear: rows, cols and row strides are multiples of 8, the weight pitch of 128");
+    if (x2 && (!w2 || cols2 < 8 || cols2 % 8 || pitch2 % 128 || pitch2 < cols2 || ldx2 % 8 || ldx2 < cols2)) return fail(CUQWEN_ERR_ARG, "linear: bad second product");
+    if (epi == LIN_GELU_SIDE) { NOT_NULL(side, d_tokens); if (side_dim < 1 || side_dim > rows) return fail(CUQWEN_ERR_ARG, "linear: side_dim out of range"); }
+    if (act == CUQWEN_ACT_BF16 && n_tokens > 1) {
+        PfGemmArgs g; memset(&g, 0, sizeof g);
+        const PfBf16Mat m{w, rows, pitch}, m2{w2, rows, pitch2};
+        const int modes[5] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE};
+        g.T = n_tokens; g.K = cols; g.K2 = cols2; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = t_err; g.mode = modes[epi];
+        g.side = (const bf16*)side; g.side_pitch = side_pitch; g.side_dim = side_dim; g.tokens = d_tokens;
+        KK(launch_prefill_gemm_bf16(g, x, ldx, &m, 1, x2, ldx2, x2 ? &m2 : nullptr, dc->stream));
+        return CUQWEN_OK;
+    }
+    if (act == CUQWEN_ACT_BF16) {
+        SegGemvArgs g; memset(&g, 0, sizeof g);
+        g.stage = SEG_PLAIN; g.xb[0] = (const bf16*)x; g.klen[0] = cols; g.kp[0] = pitch; g.err = t_err; g.nvar = 1; g.epi[0] = epi; g.out[0] = out;
+        if (x2) { g.xb[1] = (const bf16*)x2; g.klen[1] = cols2; g.kp[1] = pitch2; }
+        g.K = g.kp[0] + g.kp[1];
+        g.side = (const bf16*)side; g.side_pitch = side_pitch; g.side_dim = side_dim; g.tokens = d_tokens;
+        const SegMat m[2] = {{(const bf16*)w, rows, pitch}, {(const bf16*)w2, rows, pitch2}};
+        KK(launch_gemv_seg(g, m, x2 ? 2 : 1, cfg));
+        return CUQWEN_OK;
+    }
+    LinArgs a{};
+    a.x = x; a.ldx = ldx; a.w = (const bf16*)w; a.pitch = pitch; a.K = cols; a.x2 = x2; a.ldx2 = ldx2; a.w2 = x2 ? (const bf16*)w2 : nullptr; a.pitch2 = pitch2; a.K2 = cols2;
+    a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.side = (const bf16*)side; a.side_pitch = side_pitch; a.side_dim = side_dim; a.tokens = d_tokens;
+    KK(launch_st_linear(act, a, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_norm_rows(int device, int act, float* x, int ldx, const float* y, const float* y_w, const float* w0, void* out0, const float* w1, void* out1, int ldo, int width, float eps,
+                                  int n_rows) {
+    DEV(device);
+    NOT_NULL(x);
+    if (y) NOT_NULL(y_w);
+    if (w0) NOT_NULL(out0);
+    if (w1) NOT_NULL(w0, out1);
+    if (bad_act(act) || width < 1 || n_rows < 1 || ldx % 8 || ldx < width || (w0 && (ldo % 8 || ldo < width))) return fail(CUQWEN_ERR_ARG, "norm_rows: row strides are multiples of 8");
+    NormRowsArgs a{};
+    a.x = x; a.ldx = ldx; a.y = y; a.ldy = ldx; a.y_w = y_w; a.ldo = ldo; a.width = width; a.eps = eps;
+    if (w0) { a.w[0] = w0; a.out[0] = out0; a.n_out = 1; }
+    if (w1) { a.w[1] = w1; a.out[1] = out1; a.n_out = 2; }
+    KK(launch_st_norms(act, a, n_rows, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_latent_rows(int device, int act, const float* raw, int ld, const float* dq_w, void* cq, int ldcq, int q_rank, const float* dkv, const float* dkv_w, void* cache, int ldc,
+                                    int kv_rank, int kr_off, int rot_dim, const void* rot, float eps, int pos0, int n_rows) {
+    DEV(device);
+    NOT_NULL(dkv, dkv_w, cache, rot);
+    if (raw) NOT_NULL(dq_w, cq);
+    if (bad_act(act) || n_rows < 1 || pos0 < 0 || ld % 8 || ldc % 8 || kv_rank < 1 || kr_off % 8 || kr_off < kv_rank || rot_dim < 2 || rot_dim % 2 || ldc < kr_off + rot_dim || ld < kr_off + rot_dim ||
+        (raw && (q_rank < 1 || ldcq % 8 || ldcq < q_rank || ld < q_rank)))
+        return fail(CUQWEN_ERR_ARG, "latent_rows: unsupported shape");
+    LatentRowsArgs a{};
+    a.dq = raw; a.ld = ld; a.dq_w = dq_w; a.cq = cq; a.ldcq = ldcq; a.q_rank = q_rank; a.dkv = dkv; a.dkv_w = dkv_w; a.cache = cache; a.ldc = ldc; a.kv_rank = kv_rank; a.kr_off = kr_off;
+    a.rot_dim = rot_dim; a.rot = (const float2*)rot; a.eps = eps; a.pos0 = pos0;
+    KK(launch_st_latent_rows(act, a, n_rows, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_rot_table(int device, void* table, int n_pos, int dims, double base) {
+    DEV(device);
+    NOT_NULL(table);
+    if (n_pos < 1 || dims < 2 || dims % 2 || !(base > 0)) return fail(CUQWEN_ERR_ARG, "rot_table: unsupported shape");
+    KK(launch_rot_table((float2*)table, n_pos, dims, base, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_latent_attention(int device, int act, int impl, const void* q, const void* kn, const void* kr, const void* v, const float* sink, const float* gate, void* out, int n_tokens,
+                                         int pos0, int n_keys, int heads, int dim, int rot_dim, int vdim, int window, float scale) {
+    DEV(device);
+    NOT_NULL(q, kn, kr, v, out);
+    if (bad_act(act) || impl < 0 || impl > 1 || (impl == 0 && act != CUQWEN_ACT_BF16) || n_tokens < 1 || pos0 < 0 || pos0 + n_tokens > n_keys || heads < 1 || dim < 8 || dim % 8 || rot_dim < 8 || rot_dim % 8 ||
+        vdim < 8 || vdim % 8 || window < 0)
+        return fail(CUQWEN_ERR_ARG, "latent_attention: lengths are multiples of 8; impl 0 (tensor cores) is bfloat16 only");
+    LatentAttnArgs t{};
+    const int es = act == CUQWEN_ACT_F32 ? 4 : 2;
+    t.qn = q; t.qn_hs = dim + rot_dim; t.ldqn = heads * t.qn_hs; t.dn = dim; t.qr = (const uint8_t*)q + (size_t)dim * es; t.ldqr = t.ldqn; t.qr_hs = t.qn_hs; t.dr = rot_dim;
+    t.kn = kn; t.ldkn = heads * dim; t.kn_hs = dim; t.kr = kr; t.ldkr = rot_dim; t.v = v; t.ldv = heads * vdim; t.v_hs = vdim; t.dv = vdim; t.sink = sink; t.gate = gate; t.ldg = heads * vdim; t.g_hs = vdim;
+    t.out = out; t.ldo = heads * vdim; t.o_hs = vdim; t.T = n_tokens; t.heads = heads; t.window = window; t.scale = scale; t.pos0 = pos0;
+    if (impl == 0) KK(launch_latent_prefill_attn(t, n_keys, (size_t)n_keys, t_err, cfg));
+    else KK(launch_latent_attn(act, t, cfg));
     return CUQWEN_OK;
 }

@@ -154,15 +154,18 @@ __global__ void __launch_bounds__(256) st_rope_q_kernel(const RopeQArgs a) {
     const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
     const float* in = a.in + (size_t)t * a.ld;
     A* out = reinterpret_cast<A*>(a.out) + (size_t)t * a.ld;
-    for (int i = threadIdx.x; i < a.heads * a.head_pitch; i += 256) {
-        const int c = i % a.head_pitch, r = c - a.rot_off;
-        if (r < 0 || r >= a.rot_dim) out[i] = to_act<A>(in[i]);
-        else if (r < half) {
-            const float2 cs = a.rot[(size_t)pos * half + r];
-            const float u = in[i], v = in[i + half];
-            out[i] = to_act<A>(u * cs.x - v * cs.y);
-            out[i + half] = to_act<A>(v * cs.x + u * cs.y);
-        }
+    // rot_off and head_pitch are multiples of eight; the padding behind the rotated part is never read
+    const int units = a.rot_off / 4;
+    for (int i = threadIdx.x; i < a.heads * units; i += 256) {
+        const int o = i / units * a.head_pitch + i % units * 4;
+        store4(out + o, *reinterpret_cast<const float4*>(in + o));
+    }
+    for (int i = threadIdx.x; i < a.heads * half; i += 256) {
+        const int r = i % half, o = i / half * a.head_pitch + a.rot_off + r;
+        const float2 cs = a.rot[(size_t)pos * half + r];
+        const float u = in[o], v = in[o + half];
+        out[o] = to_act<A>(u * cs.x - v * cs.y);
+        out[o + half] = to_act<A>(v * cs.x + u * cs.y);
     }
 }
 int launch_st_rope_q(int act, const RopeQArgs& a, int T, const LaunchCfg& cfg) {

@@ -190,6 +190,19 @@ class Engine:
                                        out.ctypes.data_as(C.POINTER(C.c_float))))
         return out
 
+    def generate(self, prompt, n: int, pos0: int = 0, penalise: bool = False) -> np.ndarray:
+        """n greedy tokens after the prompt: batched prefill of all but its last token, then the decode step with its result
+        fed back (on the device, or - with the repetition penalty over everything seen so far - through the host)."""
+        seen = [int(t) for t in prompt]
+        at = pos0 + len(seen) - 1
+        if len(seen) > 1:
+            self.prefill(seen[:-1], pos0)
+        if not penalise:
+            return self.decode_n(seen[-1], at, n)
+        for i in range(n):
+            seen.append(self.step(seen[-1], at + i, seen))
+        return np.array(seen[len(seen) - n:], dtype=np.int32)
+
     @property
     def last_decode_ms(self) -> float:
         return float(_abi.lib().cuqwen_last_decode_ms(self._h))

@@ -131,3 +131,32 @@ def capture_replay(replays: int, device=0) -> float:
     ms = C.c_float()
     check(_abi.lib().cuqwen_capture_replay(device, replays, C.byref(ms)))
     return ms.value
+
+
+# ---- kernels of the layer-list designs (act: 0 bfloat16, 1 float32 activations) ----
+LIN_F32, LIN_ACT, LIN_RELU2, LIN_ADD, LIN_GELU_SIDE = range(5)
+
+
+def linear(act, epi, x, ldx, w, pitch, cols, n_tokens, rows, out, ldo, second=None, side=None, device=0):
+    """cuqwen_k_linear; second = (x2, ldx2, w2, pitch2, cols2), side = (table, pitch, dim, d_tokens)."""
+    x2, ldx2, w2, p2, c2 = second or (None, 0, None, 0, 0)
+    sp, spitch, sdim, tok = side or (None, 0, 0, None)
+    check(_abi.lib().cuqwen_k_linear(device, act, epi, _p(x), ldx, _p(w), pitch, cols, _p(x2), ldx2, _p(w2), p2, c2, n_tokens, rows, _p(out), ldo, _p(sp), spitch, sdim, _p(tok)))
+
+
+def norm_rows(act, x, ldx, width, eps, n_rows, y=None, y_w=None, outs=(), ldo=0, device=0):
+    """cuqwen_k_norm_rows; outs = up to two (weight, out) pairs."""
+    o = list(outs) + [(None, None)] * (2 - len(outs))
+    check(_abi.lib().cuqwen_k_norm_rows(device, act, _p(x), ldx, _p(y), _p(y_w), _p(o[0][0]), _p(o[0][1]), _p(o[1][0]), _p(o[1][1]), ldo, width, eps, n_rows))
+
+
+def latent_rows(act, raw, ld, dq_w, cq, ldcq, q_rank, dkv, dkv_w, cache, ldc, kv_rank, kr_off, rot_dim, rot, eps, pos0, n_rows, device=0):
+    check(_abi.lib().cuqwen_k_latent_rows(device, act, _p(raw), ld, _p(dq_w), _p(cq), ldcq, q_rank, _p(dkv), _p(dkv_w), _p(cache), ldc, kv_rank, kr_off, rot_dim, _p(rot), eps, pos0, n_rows))
+
+
+def rot_table(table, n_pos, dims, base, device=0):
+    check(_abi.lib().cuqwen_k_rot_table(device, _p(table), n_pos, dims, base))
+
+
+def latent_attention(act, impl, q, kn, kr, v, sink, gate, out, n_tokens, pos0, n_keys, heads, dim, rot_dim, vdim, window, scale, device=0):
+    check(_abi.lib().cuqwen_k_latent_attention(device, act, impl, _p(q), _p(kn), _p(kr), _p(v), _p(sink), _p(gate), _p(out), n_tokens, pos0, n_keys, heads, dim, rot_dim, vdim, window, scale))

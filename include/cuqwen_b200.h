@@ -285,6 +285,28 @@ int cuqwen_k_dequant(int device, int quant, const void* w, const void* scale, vo
 int cuqwen_k_tp_sum(int device, const void* x, void* x_next, const void* slots, int n_ranks, int dim, const int* d_step_no, int seq_index,
                     long long wait_cycles);
 
+/* ---- kernels of the layer-list designs (cuqwen_open; none has a counterpart in the reference).  act: CUQWEN_ACT_* of the
+ * activations; weights are bfloat16 [rows][pitch]; norm weights, sinks, gates and residual rows are float32. ---- */
+/* out[t][r] = epilogue(sum_k x[t][k] w[r][k] + sum_k x2[t][k] w2[r][k]), the second product optional (x2 null).  epi: 0 float32 out, 1 out in the
+ * activation type, 2 max(acc, 0)^2 in the activation type, 3 float32 out += acc, 4 gelu_tanh(acc) * side[d_tokens[t]][r] in the
+ * activation type (side rows of side_pitch bfloat16 values; rows from side_dim on give 0).  bfloat16: the tcgen05 GEMM for
+ * several tokens, the segmented GEMV for one; float32: CUDA cores. */
+int cuqwen_k_linear(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, const void* x2, int ldx2, const void* w2, int pitch2,
+                    int cols2, int n_tokens, int rows, void* out, int ldo, const void* side, int side_pitch, int side_dim, const int* d_tokens);
+/* Per row: x += y / rms(y) * y_w (y may be null), then out_i = x / rms(x) * w_i for the given weights; eps inside the root. */
+int cuqwen_k_norm_rows(int device, int act, float* x, int ldx, const float* y, const float* y_w, const float* w0, void* out0, const float* w1, void* out1, int ldo, int width, float eps,
+                       int n_rows);
+/* Per row t: cq[t] = norm of raw[t] (q_rank values; raw null: left out), cache row pos0 + t = [norm of dkv[t] (kv_rank) | dkv[t] from kr_off on, rotated]. */
+int cuqwen_k_latent_rows(int device, int act, const float* raw, int ld, const float* dq_w, void* cq, int ldcq, int q_rank, const float* dkv, const float* dkv_w, void* cache, int ldc,
+                         int kv_rank, int kr_off, int rot_dim, const void* rot, float eps, int pos0, int n_rows);
+/* (cos, sin) float32 pairs [n_pos][dims / 2] of position * base^(-2 i / dims). */
+int cuqwen_k_rot_table(int device, void* table, int n_pos, int dims, double base);
+/* Attention of queries at positions pos0 .. over keys 0 .. n_keys: q [t][heads][dim + rot_dim], kn [key][heads][dim], kr [key][rot_dim] shared by
+ * the heads, v [key][heads][vdim]; query p sees keys p - window + 1 .. p (window 0: 0 .. p); sink [heads] or null: one more term
+ * exp(sink) in the denominator; gate [t][heads][vdim] or null: out *= sigmoid(gate).  impl 0: tcgen05, impl 1: CUDA cores. */
+int cuqwen_k_latent_attention(int device, int act, int impl, const void* q, const void* kn, const void* kr, const void* v, const float* sink, const float* gate, void* out, int n_tokens,
+                              int pos0, int n_keys, int heads, int dim, int rot_dim, int vdim, int window, float scale);
+
 const char* cuqwen_strerror(int code);
 const char* cuqwen_last_error(void);
 
