@@ -18,7 +18,7 @@ struct RotarySpec { int dims = 0; double base = 0; };
 // [normed latent (kv_rank) | rotated key part shared by all heads (rot_dim)].
 struct LatentAttnSpec {
     int heads = 0, dim = 0, rot_dim = 0, vdim = 0, q_rank = 0, kv_rank = 0;
-    int window = 0;          // a query sees itself and the window - 1 tokens before it; 0 = everything before it
+    int window = 0;          // length of the stretch of positions, ending with its own, that a query sees; 0 = all up to its own
     int kv_from = -1;        // >= 0: attends to the rows that layer's latent projection cached; no projection of its own
     double scale = 0;
     RotarySpec rot;

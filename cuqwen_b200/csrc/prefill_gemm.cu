@@ -388,16 +388,12 @@ int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     a.mh = a.T > kPfM ? kPfMH : 1;
     int mtiles = (a.T + kPfM * a.mh - 1) / (kPfM * a.mh);
-    auto ctas = [&](int w) { int n = 0; for (int i = 0; i < nmat; ++i) n += (m[i].rows + w - 1) / w; return n * mtiles; };
-    // 64 or 128 rows a tile where wider ones would leave most SMs idle, as in launch_prefill_gemm; and 128 where the last wave of
-    // 256-row tiles would be nearly empty (a 128-row tile costs a little more than half of one).
-    const int wide = ctas(kPfN);
-    int nt = kPfN;
-    if (sms > 0) {
-        const int w256 = (wide + sms - 1) / sms, w128 = (ctas(kPfN / 2) + sms - 1) / sms;
-        if (wide * 4 <= sms) nt = kPfN / 4;
-        else if (wide * 2 <= sms || w128 * 59 < w256 * 100) nt = kPfN / 2;
-    }
+    int wide = 0;
+    for (int i = 0; i < nmat; ++i) wide += (m[i].rows + kPfN - 1) / kPfN;
+    wide *= mtiles;
+    // 64 or 128 rows a tile where wider ones would leave most SMs idle, as in launch_prefill_gemm.  (128-row tiles where the
+    // last wave of 256-row tiles is nearly empty: measured, no gain - a tile's cost is its share of L2 traffic, not its MMAs.)
+    const int nt = (sms > 0 && wide * 4 <= sms) ? kPfN / 4 : (sms > 0 && wide * 2 <= sms) ? kPfN / 2 : kPfN;
     if (nt == kPfN / 4 && a.mh == 2) { a.mh = 1; mtiles = (a.T + kPfM - 1) / kPfM; }       // few rows: a token half per CTA, twice the CTAs
     const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
     if (int r = pf_map(&a.tx, x, bf, 2, (size_t)a.T, (size_t)a.K, kPfKB, kPfM, true, (size_t)ldx)) return r;

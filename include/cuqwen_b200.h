@@ -293,7 +293,7 @@ int cuqwen_k_tp_sum(int device, const void* x, void* x_next, const void* slots, 
  * several tokens, the segmented GEMV for one; float32: CUDA cores. */
 int cuqwen_k_linear(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, const void* x2, int ldx2, const void* w2, int pitch2,
                     int cols2, int n_tokens, int rows, void* out, int ldo, const void* side, int side_pitch, int side_dim, const int* d_tokens);
-/* Per row: x += y / rms(y) * y_w (y may be null), then out_i = x / rms(x) * w_i for the given weights; eps inside the root. */
+/* Per row: x += y / rms(y) * y_w (y may be null), then out_i = x / rms(x) * w_i for the given weights; rms(v) = sqrt(mean(v^2) + eps). */
 int cuqwen_k_norm_rows(int device, int act, float* x, int ldx, const float* y, const float* y_w, const float* w0, void* out0, const float* w1, void* out1, int ldo, int width, float eps,
                        int n_rows);
 /* Per row t: cq[t] = norm of raw[t] (q_rank values; raw null: left out), cache row pos0 + t = [norm of dkv[t] (kv_rank) | dkv[t] from kr_off on, rotated]. */

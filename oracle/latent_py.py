@@ -13,7 +13,7 @@ import numpy as np
 
 
 def rms_norm(x, weight, eps):
-    """Divide by the root mean square (eps under the root), then scale element by element."""
+    """x over sqrt(mean x^2 + eps), scaled element by element."""
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * weight
 
 
@@ -47,7 +47,7 @@ def rotate_half(x, pos, base, dims):
 
 
 def window_mask(n_q, n_k, size, pos0=0):
-    """True where query pos0 + i may see key j: not in its future, at most size - 1 tokens back."""
+    """True where query pos0 + i may see key j: the last `size` positions up to its own."""
     d = (pos0 + np.arange(n_q))[:, None] - np.arange(n_k)[None, :]
     return (d >= 0) & (d < size)
 

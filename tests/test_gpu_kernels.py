@@ -323,7 +323,7 @@ def test_penalty_and_argmax(built):
         print(f"NaN logit at 1234: this library {mine}, reference kernel {theirs}, oracle {O.argmax(nanv)}")
         assert mine == theirs
     else:
-            assert mine in (O.argmax(nanv), int(np.nanargmax(nanv.astype(np.float32))))      # measured against it earlier: the compiled kernels pass a NaN over
+        assert mine in (O.argmax(nanv), int(np.nanargmax(nanv.astype(np.float32))))      # measured against it earlier: the compiled kernels pass a NaN over
 
 
 def test_embedding_lookup(built):
