@@ -105,9 +105,88 @@ int parse_falivik(const Json& cfg, StackSpec* s) {
     return CUQWEN_OK;
 }
 
+int parse_rotary(const Fields& f, const std::string& where, int dim, RotarySpec* r) {
+    if (f.absent("rot")) return CUQWEN_OK;
+    Fields rot(f.get("rot"), where + ".rot");
+    r->base = rot.number("base"); r->dims = rot.integer("dims", 0);
+    if (!rot.bad.empty()) return config_error(rot.bad);
+    if (r->dims % 2 || r->dims > dim || !(r->base > 0)) return config_error(where + ".rot: an even number of dims, at most the head's, and a positive base");
+    return CUQWEN_OK;
+}
+int parse_clamped_glu(const Json* mlp, const std::string& where, double slope, DenseMlpSpec* m) {
+    Fields f(mlp, where);
+    const Json* kind = f.get("kind");
+    if (!kind || kind->kind != Json::Str || kind->str != "dense") return config_error(where + ".kind: this design has dense feed-forwards only");
+    m->kind = MLP_CLAMPED_GLU; m->ff = f.integer("ff"); m->limit = f.number("limit"); m->slope = slope;
+    if (!f.bad.empty()) return config_error(f.bad);
+    if (!(m->limit > 0)) return config_error(where + ".limit must be positive");
+    return CUQWEN_OK;
+}
+int parse_parallel(const Json* mixer, const std::string& where, LayerSpec* L) {
+    Fields f(mixer, where);
+    L->kind = MIX_PARALLEL;
+    L->left_scale = f.number("left_scale"); L->right_scale = f.number("right_scale");
+    if (!f.bad.empty()) return config_error(f.bad);
+    Fields l(f.get("left"), where + ".left"), r(f.get("right"), where + ".right");
+    GroupedAttnSpec& a = L->left;
+    a.heads = l.integer("heads"); a.kv_heads = l.integer("kv_heads"); a.dim = l.integer("dim"); a.vdim = l.integer("vdim"); a.scale = l.number("scale");
+    if (!l.bad.empty()) return config_error(l.bad);
+    if (a.heads % a.kv_heads) return config_error(where + ".left.heads must be a multiple of kv_heads");
+    if (int e = parse_rotary(l, where + ".left", a.dim, &a.rot)) return e;
+    L->right.heads = r.integer("heads"); L->right.dim = r.integer("dim");
+    return r.bad.empty() ? (int)CUQWEN_OK : config_error(r.bad);
+}
+int parse_delta(const Json* mixer, const std::string& where, LayerSpec* L) {
+    Fields f(mixer, where);
+    L->kind = MIX_DELTA;
+    DeltaSpec& d = L->delta;
+    d.heads = f.integer("heads"); d.kv_heads = f.integer("kv_heads"); d.dim = f.integer("dim"); d.vdim = f.integer("vdim"); d.conv = f.integer("conv");
+    if (!f.bad.empty()) return config_error(f.bad);
+    if (d.heads % d.kv_heads) return config_error(where + ".heads must be a multiple of kv_heads");
+    return CUQWEN_OK;
+}
+
+// Gipotar: sequential pre-norm layers (norm weights stored about zero) whose mixer is either softmax attention beside time
+// mixing or a gated delta rule; clamped gated feed-forward or none; scaled embedding, soft-capped logits.
+int parse_gipotar(const Json& cfg, StackSpec* s) {
+    constexpr double kSlope = 1.702;
+    Fields top(&cfg, "model");
+    s->sequential = true; s->norm_offset = 1;
+    s->vocab = top.integer("vocab"); s->width = top.integer("width");
+    if (!top.absent("residual_mult")) s->residual_mult = top.number("residual_mult");
+    if (!top.absent("logit_softcap")) s->logit_softcap = top.number("logit_softcap");
+    if (!top.bad.empty()) return config_error(top.bad);
+    if (s->logit_softcap < 0) return config_error("logit_softcap must not be negative");
+    Fields norm(top.get("norm"), "norm");
+    s->norm_eps = norm.number("eps");
+    if (!norm.bad.empty()) return config_error(norm.bad);
+    if (!top.absent("embedding")) {
+        Fields e(top.get("embedding"), "embedding");
+        if (!e.absent("scale")) s->embed_scale = e.number("scale");
+        if (!e.bad.empty()) return config_error(e.bad);
+    }
+    const Json* layers = top.get("layers");
+    if (!layers || layers->kind != Json::Arr || layers->arr.empty()) return config_error("layers must be a list");
+    for (size_t i = 0; i < layers->arr.size(); ++i) {
+        const std::string where = "layers[" + std::to_string(i) + "]";
+        Fields f(&layers->arr[i], where);
+        if (!f.bad.empty()) return config_error(f.bad);
+        const Json* type = f.get("type");
+        const std::string t = type && type->kind == Json::Str ? type->str : "";
+        LayerSpec L;
+        if (t == "parallel") { if (int r = parse_parallel(f.get("mixer"), where + ".mixer", &L)) return r; }
+        else if (t == "delta") { if (int r = parse_delta(f.get("mixer"), where + ".mixer", &L)) return r; }
+        else return config_error(where + ".type: this design has the mixers parallel and delta");
+        if (!f.absent("mlp")) if (int r = parse_clamped_glu(f.get("mlp"), where + ".mlp", kSlope, &L.mlp)) return r;
+        s->layers.push_back(L);
+    }
+    return CUQWEN_OK;
+}
+
 struct Design { const char* name; int (*parse)(const Json&, StackSpec*); };
 const Design kDesigns[] = {
     {"Falivik", parse_falivik},
+    {"Gipotar", parse_gipotar},
 };
 
 bool read_file(const std::string& path, std::string* out) {
@@ -136,14 +215,41 @@ int read_model_config(const char* dir, StackSpec* out) {
     return config_error("unknown architecture \"" + a->str + "\"");
 }
 
+int read_model_shapes(const char* dir, StackSpec* spec) {
+    Safetensors st;
+    bool opened = false;
+    for (size_t i = 0; i < spec->layers.size(); ++i) {
+        LayerSpec& L = spec->layers[i];
+        if (L.kind != MIX_PARALLEL) continue;
+        if (!opened) { if (int r = st.open((std::string(dir) + "/model.safetensors").c_str())) return r; opened = true; }
+        const std::string name = "l" + std::to_string(i) + ".mix.right.w1";
+        const Safetensors::Tensor* t = st.find(name);
+        if (!t) return report_error(CUQWEN_ERR_DIMS, "tensor %s is missing", name.c_str());
+        if (t->shape.size() != 2 || t->shape[0] < 1 || t->shape[0] > (1 << 20)) return report_error(CUQWEN_ERR_DIMS, "tensor %s is no matrix", name.c_str());
+        L.right.rank = (int)t->shape[0];
+    }
+    return CUQWEN_OK;
+}
+
 std::string describe_spec(const StackSpec& s) {
-    char b[512];
+    char b[640];
     snprintf(b, sizeof b, "design %s\nvocab %d\nwidth %d\nlayers %zu\nnorm_eps %.9g\nside_dim %d\n", s.design.c_str(), s.vocab, s.width, s.layers.size(), s.norm_eps, s.side_dim);
     std::string t = b;
+    if (s.sequential) {
+        snprintf(b, sizeof b, "residual_mult %.9g\nembed_scale %.9g\nlogit_softcap %.9g\n", s.residual_mult, s.embed_scale, s.logit_softcap);
+        t += b;
+    }
     for (size_t i = 0; i < s.layers.size(); ++i) {
-        const LatentAttnSpec& a = s.layers[i].attn;
-        snprintf(b, sizeof b, "layer %zu latent_attention heads %d dim %d rot_dim %d vdim %d q_rank %d kv_rank %d window %d kv_from %d scale %.9g rot_base %.9g sink %d gate %d ff %d\n",
-                 i, a.heads, a.dim, a.rot_dim, a.vdim, a.q_rank, a.kv_rank, a.window, a.kv_from, a.scale, a.rot.base, a.sink, a.gate, s.layers[i].mlp.ff);
+        const LayerSpec& L = s.layers[i];
+        if (L.kind == MIX_LATENT) {
+            const LatentAttnSpec& a = L.attn;
+            snprintf(b, sizeof b, "layer %zu latent_attention heads %d dim %d rot_dim %d vdim %d q_rank %d kv_rank %d window %d kv_from %d scale %.9g rot_base %.9g sink %d gate %d ff %d\n",
+                     i, a.heads, a.dim, a.rot_dim, a.vdim, a.q_rank, a.kv_rank, a.window, a.kv_from, a.scale, a.rot.base, a.sink, a.gate, L.mlp.ff);
+        } else if (L.kind == MIX_PARALLEL)
+            snprintf(b, sizeof b, "layer %zu parallel left_heads %d left_kv_heads %d left_dim %d left_vdim %d score_scale %.9g rot_dims %d rot_base %.9g right_heads %d right_dim %d left_scale %.9g right_scale %.9g ff %d limit %.9g\n",
+                     i, L.left.heads, L.left.kv_heads, L.left.dim, L.left.vdim, L.left.scale, L.left.rot.dims, L.left.rot.base, L.right.heads, L.right.dim, L.left_scale, L.right_scale, L.mlp.ff, L.mlp.limit);
+        else
+            snprintf(b, sizeof b, "layer %zu delta heads %d kv_heads %d dim %d vdim %d conv %d ff %d limit %.9g\n", i, L.delta.heads, L.delta.kv_heads, L.delta.dim, L.delta.vdim, L.delta.conv, L.mlp.ff, L.mlp.limit);
         t += b;
     }
     return t;
