@@ -12,7 +12,7 @@ __global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(const LatentAtt
     __shared__ float red[40];
     float *q = la_smem, *acc = q + a.dn + a.dr, *pr = acc + a.dv;
     pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x;
+    const int h = blockIdx.x, hk = a.kv_group > 1 ? h / a.kv_group : h, t = blockIdx.y, tid = threadIdx.x;
     const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
     const A* qn = reinterpret_cast<const A*>(a.qn) + (size_t)t * a.ldqn + (size_t)h * a.qn_hs;
     const A* qr = reinterpret_cast<const A*>(a.qr) + (size_t)t * a.ldqr + (size_t)h * a.qr_hs;
@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(const LatentAtt
         const int k = k0 + tid;
         float s = -INFINITY;
         if (k <= pos) {
-            const A* kn = reinterpret_cast<const A*>(a.kn) + (size_t)(k - a.kbase) * a.ldkn + (size_t)h * a.kn_hs;
+            const A* kn = reinterpret_cast<const A*>(a.kn) + (size_t)(k - a.kbase) * a.ldkn + (size_t)hk * a.kn_hs;
             const A* kr = reinterpret_cast<const A*>(a.kr) + (size_t)k * a.ldkr;
             float d = 0.f;
             for (int i = 0; i < a.dn; ++i) d = fmaf(q[i], act_f(kn[i]), d);
@@ -47,13 +47,13 @@ __global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(const LatentAtt
         l = l * alpha + cta_sum(p, red);                 // barriers inside: pr is complete
         const int n = pos - k0 + 1 < kLaThreads ? pos - k0 + 1 : kLaThreads;
         for (int c = tid; c < a.dv; c += kLaThreads) {
-            const A* v = reinterpret_cast<const A*>(a.v) + (size_t)(k0 - a.kbase) * a.ldv + (size_t)h * a.v_hs + c;
+            const A* v = reinterpret_cast<const A*>(a.v) + (size_t)(k0 - a.kbase) * a.ldv + (size_t)hk * a.v_hs + c;
             float o = acc[c] * alpha;
             for (int j = 0; j < n; ++j) o = fmaf(pr[j], act_f(v[(size_t)j * a.ldv]), o);
             acc[c] = o;
         }
     }
-    const float inv = 1.0f / l;
+    const float inv = a.out_scale / l;
     for (int c = tid; c < a.dv; c += kLaThreads) {
         float o = acc[c] * inv;
         if (a.gate) o *= sigmoid_f(a.gate[(size_t)t * a.ldg + (size_t)h * a.g_hs + c]);

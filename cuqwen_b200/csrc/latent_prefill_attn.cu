@@ -27,7 +27,8 @@ struct LatentPrefillArgs {
     int T, pos0, kbase, window, vdim, vcols;        // vcols: value columns written (vdim rounded up to eight)
     int nbn, nbr, nbv, kn_steps, kr_steps;          // 64-column blocks of each part, 16-column steps of the key parts
     int nks, nvs;                                   // ring slots
-    float scale_log2;
+    float scale_log2, out_scale;
+    int kv_group;                                   // query heads to a key / value head
     uint32_t tmem_cols;
     unsigned* err;
 };
@@ -41,7 +42,7 @@ __global__ void __launch_bounds__(kLpThreads, 2) latent_prefill_attn_kernel(cons
     const uint32_t sQ = base, sK = sQ + nbk * kLpQBlk, sV = sK + a.nks * kslot, sP = sV + a.nvs * vslot, bars = sP + kLpPTile;
     const uint32_t b_q = bars, b_kfull = bars + 8, b_kfree = bars + 24, b_vfull = bars + 40, b_vfree = bars + 56, b_sfull = bars + 72, b_p = bars + 88, b_pv = bars + 96,
                    tmem_slot = bars + 104;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y, hkv = head / a.kv_group;
     const int q0 = (gridDim.x - 1 - blockIdx.x) * kLpBM;                 // the longest rows first
     const int p_first = a.pos0 + q0, p_last = a.pos0 + min(q0 + kLpBM, a.T) - 1;
     const int k_first = a.window > 0 && p_first - a.window + 1 > 0 ? p_first - a.window + 1 : 0;
@@ -71,11 +72,11 @@ __global__ void __launch_bounds__(kLpThreads, 2) latent_prefill_attn_kernel(cons
                 const int ks = j % a.nks, vs = j % a.nvs; const uint32_t kp = (uint32_t)(j / a.nks) & 1u, vp = (uint32_t)(j / a.nvs) & 1u;
                 if (!mbar_wait(b_kfree + 8 * ks, kp ^ 1u)) { failed = true; break; }
                 mbar_expect_tx(b_kfull + 8 * ks, (uint32_t)kslot);
-                for (int b = 0; b < a.nbn; ++b) tma_load_3d(sK + ks * kslot + b * kLpKBlk, &a.tkn, 64 * b, head, key - a.kbase, b_kfull + 8 * ks);
+                for (int b = 0; b < a.nbn; ++b) tma_load_3d(sK + ks * kslot + b * kLpKBlk, &a.tkn, 64 * b, hkv, key - a.kbase, b_kfull + 8 * ks);
                 for (int b = 0; b < a.nbr; ++b) tma_load_2d(sK + ks * kslot + (a.nbn + b) * kLpKBlk, &a.tkr, 64 * b, key, b_kfull + 8 * ks);
                 if (!mbar_wait(b_vfree + 8 * vs, vp ^ 1u)) { failed = true; break; }
                 mbar_expect_tx(b_vfull + 8 * vs, (uint32_t)vslot);
-                for (int b = 0; b < a.nbv; ++b) tma_load_3d(sV + vs * vslot + b * kLpKBlk, &a.tv, 64 * b, head, key - a.kbase, b_vfull + 8 * vs);
+                for (int b = 0; b < a.nbv; ++b) tma_load_3d(sV + vs * vslot + b * kLpKBlk, &a.tv, 64 * b, hkv, key - a.kbase, b_vfull + 8 * vs);
             }
         }
     } else if (warp == 1) {
@@ -180,7 +181,7 @@ __global__ void __launch_bounds__(kLpThreads, 2) latent_prefill_attn_kernel(cons
         if (hsel == 1) l = mxbuf[128 + r];
         if (!failed && !mbar_wait(b_pv, (uint32_t)(nj - 1) & 1u)) failed = true;
         tc_fence_after();
-        const float inv = 1.0f / l;
+        const float inv = a.out_scale / l;
         const int t = q0 + r;
 #pragma unroll 1
         for (int c = hsel; c < nch; c += 2) {
@@ -242,18 +243,19 @@ bool latent_prefill_fits(int dn, int dr, int dv) {
     return dv <= 256 && lp_smem_bytes((dn + 63) / 64 + (dr + 63) / 64, (dv + 63) / 64, 1, 1) <= 225 * 1024;
 }
 int launch_latent_prefill_attn(const LatentAttnArgs& t, int n_keys, size_t cache_rows, unsigned* err, const LaunchCfg& cfg) {
-    if (t.T < 1 || t.heads < 1 || t.pos_ptr || t.out_f32 || n_keys < 1 || !latent_prefill_fits(t.dn, t.dr, t.dv) || ((t.ldqn | t.qn_hs | t.ldqr | t.qr_hs | t.ldkn | t.kn_hs | t.ldkr | t.ldv | t.v_hs | t.ldo | t.o_hs) & 7))
+    if (t.T < 1 || t.heads < 1 || t.pos_ptr || t.out_f32 || n_keys < 1 || (t.kv_group > 1 && t.heads % t.kv_group) || !latent_prefill_fits(t.dn, t.dr, t.dv) || ((t.ldqn | t.qn_hs | t.ldqr | t.qr_hs | t.ldkn | t.kn_hs | t.ldkr | t.ldv | t.v_hs | t.ldo | t.o_hs) & 7))
         return (int)cudaErrorInvalidValue;
     LatentPrefillArgs a{};
     if (int r = lp_map(&a.tqn, t.qn, t.dn, t.heads, t.qn_hs, (size_t)t.T, t.ldqn, kLpBM)) return r;
-    if (int r = lp_map(&a.tqr, t.qr, t.dr, t.heads, t.qr_hs, (size_t)t.T, t.ldqr, kLpBM)) return r;
-    if (int r = lp_map(&a.tkn, t.kn, t.dn, t.heads, t.kn_hs, (size_t)n_keys, t.ldkn, kLpBN)) return r;
-    if (int r = lp_map(&a.tkr, t.kr, t.dr, 0, 0, cache_rows, t.ldkr, kLpBN)) return r;
-    if (int r = lp_map(&a.tv, t.v, t.dv, t.heads, t.v_hs, (size_t)n_keys, t.ldv, kLpBN)) return r;
+    if (t.dr > 0) if (int r = lp_map(&a.tqr, t.qr, t.dr, t.heads, t.qr_hs, (size_t)t.T, t.ldqr, kLpBM)) return r;
+    const int grp = t.kv_group > 1 ? t.kv_group : 1, kvh = t.heads / grp;
+    if (int r = lp_map(&a.tkn, t.kn, t.dn, kvh, t.kn_hs, (size_t)n_keys, t.ldkn, kLpBN)) return r;
+    if (t.dr > 0) if (int r = lp_map(&a.tkr, t.kr, t.dr, 0, 0, cache_rows, t.ldkr, kLpBN)) return r;
+    if (int r = lp_map(&a.tv, t.v, t.dv, kvh, t.v_hs, (size_t)n_keys, t.ldv, kLpBN)) return r;
     a.out = (bf16*)t.out; a.ldo = t.ldo; a.o_hs = t.o_hs; a.gate = t.gate; a.ldg = t.ldg; a.g_hs = t.g_hs; a.sink = t.sink;
     a.T = t.T; a.pos0 = t.pos0; a.kbase = t.kbase; a.window = t.window; a.vdim = t.dv; a.vcols = (t.dv + 7) / 8 * 8;
     a.nbn = (t.dn + 63) / 64; a.nbr = (t.dr + 63) / 64; a.nbv = (t.dv + 63) / 64; a.kn_steps = (t.dn + 15) / 16; a.kr_steps = (t.dr + 15) / 16;
-    a.scale_log2 = t.scale * 1.4426950408889634f; a.err = err;
+    a.scale_log2 = t.scale * 1.4426950408889634f; a.out_scale = t.out_scale; a.kv_group = grp; a.err = err;
     a.tmem_cols = t.dv <= 128 ? 256u : 512u;
     // two slots each if two CTAs still fit an SM (and its TMEM), else one each if that lets them; a CTA that has the SM to itself takes two
     const int nbk = a.nbn + a.nbr, half = 113 * 1024;

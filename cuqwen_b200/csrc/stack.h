@@ -19,10 +19,10 @@ typedef __nv_bfloat16 bf16;
 enum Act : int { ACT_BF16 = 0, ACT_F32 = 1 };
 
 // ---- row kernels (stack_rows.cu) ---------------------------------------------------------------------------------------
-// x[t] = embed[tokens[t]]
-int launch_st_embed(const bf16* table, int pitch, const int* tokens, float* x, int ldx, int width, int T, const LaunchCfg& cfg);
+// x[t] = scale * embed[tokens[t]]
+int launch_st_embed(const bf16* table, int pitch, const int* tokens, float* x, int ldx, int width, float scale, int T, const LaunchCfg& cfg);
 // The first launch of a decode step: takes over the mailbox, then the same for ctl->token.
-int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, int width, const LaunchCfg& cfg);
+int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, int width, float scale, const LaunchCfg& cfg);
 
 // Per row: x += y / rms(y) * y_w (y may be null), then n_out copies x / rms(x) * w[i] -> out[i].
 struct NormRowsArgs {
@@ -58,8 +58,10 @@ enum LinEpi : int {
     LIN_F32 = 0,          // out (float) = acc
     LIN_ACT = 1,          // out (activation type) = acc
     LIN_RELU2 = 2,        // out (activation type) = max(acc, 0)^2
-    LIN_ADD = 3,          // out (float) += acc
-    LIN_GELU_SIDE = 4     // out (activation type) = gelu_tanh(acc) * side[tokens[t]][r]
+    LIN_ADD = 3,          // out (float) += c0 * acc
+    LIN_GELU_SIDE = 4,    // out (activation type) = gelu_tanh(acc) * side[tokens[t]][r]
+    LIN_CAP = 5,          // out (float) = c0 * tanh(acc / c0)
+    LIN_GLU = 6           // out (activation type) = clamped_glu(gate, up, limit c0, slope c1); rows come as eight of the gate, eight of the up matrix in turn
 };
 struct LinArgs {
     const void* x; int ldx; const bf16* w; int pitch, K;
@@ -67,13 +69,16 @@ struct LinArgs {
     int T, R, epi;
     void* out; int ldo;
     const bf16* side; int side_pitch, side_dim; const int* tokens; // LIN_GELU_SIDE
+    float c0, c1;                                                  // constants of the epilogue
 };
+// LIN_GLU is not among its epilogues: LIN_F32, then launch_st_glu_rows.
 int launch_st_linear(int act, const LinArgs& a, const LaunchCfg& cfg);
 
 // ---- latent attention (latent_attn.cu) -------------------------------------------------------------------------------
 // Softmax attention over [unrotated | rotated] keys with a window, a sink and an output gate.  Keys and values either
 // per head (prefill: k = W_uk c, v = W_uv c of every key in reach) or the latents themselves (decode: queries carried
-// into the latent space by absorb_q, values left there for uv_gate).
+// into the latent space by absorb_q, values left there for uv_gate).  Grouped attention is the same with one key part (dr 0)
+// and several query heads to a key / value head (kv_group).
 struct LatentAttnArgs {
     const void *qn, *qr; int ldqn, qn_hs, dn, ldqr, qr_hs, dr;      // unrotated and rotated query parts: row stride, head stride, length
     const void* kn; int ldkn, kn_hs;                                // unrotated keys; row 0 is key `kbase`
@@ -87,6 +92,8 @@ struct LatentAttnArgs {
     int T, heads, window;                                           // window 0: all earlier keys
     float scale;
     const int* pos_ptr; int pos0;
+    int kv_group;                                                   // query heads that share a key / value head (0 and 1: none)
+    float out_scale;                                                // factor of the output
 };
 int launch_latent_attn(int act, const LatentAttnArgs& a, const LaunchCfg& cfg);
 // The same for bfloat16 portions on the tensor cores (latent_prefill_attn.cu), where the sizes fit: keys and values hold n_keys
@@ -109,13 +116,94 @@ struct LatentDecodeArgs {
     int nsplit; float* part_o; float* part_ml;           // [nsplit][heads][kvrp], [nsplit][heads][2]
     int ncl;                                             // set by the launcher: CTAs of a head that share the merge
     const bf16* wv; int pitch, vdim, vdimp, kv_rank; const float* gate; int g_hs; bf16* out; int o_hs;
+    // Grouped attention: a cache of rows [key kdim | value kvrp] per key / value head, group query heads to each, kv_stride
+    // elements from head to head; group 0: one cache for all heads whose rows are key and value at once.
+    int group, kdim; size_t kv_stride; float out_scale;
 };
 // Splits that launch_latent_decode wants for a cache of max_seq rows; 0 = sizes it does not cover.
 int latent_decode_splits(int heads, int crow, int kvrp, int window, int max_seq, int sm_count);
 int launch_latent_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done);
+// The grouped form; the fold writes the merged heads times out_scale.
+int grouped_decode_splits(int heads, int kv_heads, int kdim, int vdimp, int max_seq, int sm_count);
+int launch_grouped_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done);
 // att[h][v] = sigmoid(g[h][v]) * sum_r W_uv[h][v][r] o[h][r].  o float [heads][ldo].
 struct UvGateArgs { const float* o; int ldo; const bf16* wv; int pitch, heads, vdim, vdimp, kv_rank; const float* gate; int g_hs; void* out; int o_hs; };
 int launch_uv_gate(int act, const UvGateArgs& a, const LaunchCfg& cfg);
+
+// ---- grouped attention (grouped_attn.cu) -------------------------------------------------------------------------------
+// Rows of raw projections [q heads x dimp | k kv_heads x dimp | v kv_heads x vdimp]: rotated queries to q, [rotated key | value]
+// to the cache [kv_heads][max_seq][dimp + vdimp] at the rows' positions.
+struct QkvRowsArgs {
+    const float* raw; int ld, k_off, v_off;
+    int heads, kv_heads, dim, dimp, vdimp;
+    void* q; int ldq; void* cache; int max_seq;
+    const float2* rot; int rot_dims;                                // rot_dims 0: no rotation
+    const int* pos_ptr; int pos0;
+};
+int launch_qkv_rows(int act, const QkvRowsArgs& a, int T, const LaunchCfg& cfg);
+
+// ---- recurrent mixers ---------------------------------------------------------------------------------------------------
+// States live from token to token: float32, zero at position 0.  Everything that enters a recurrence is float32 as well.
+//
+// h = norm(x); out variant 0 = h, variant i = h + (previous token's h - h) * mu[i - 1].  prev: ring of two rows by position
+// parity; the last row's h goes to `tail` (launch_tail_rows puts it into the ring once every row has been read).
+struct ShiftRowsArgs {
+    const float* x; int ldx; const float* w; int width; float eps;
+    void* out; int ldo; size_t var_stride; const float* mu; int ldmu, n_mix;
+    const float* prev; int ldprev; float* tail;
+    const int* pos_ptr; int pos0;
+};
+int launch_shift_rows(int act, const ShiftRowsArgs& a, int T, const LaunchCfg& cfg);
+// The last min(T, keep) rows of src (row t at position pos0 + t) into ring rows by position (mod slots).
+struct TailRowsArgs { const float* src; int lds, T; float* ring; int ldr, n, slots, keep; const int* pos_ptr; int pos0; };
+int launch_tail_rows(const TailRowsArgs& a, const LaunchCfg& cfg);
+// out = tanh(raw) in the activation type; bfloat16: as two parts whose sum carries it to 16 bits (the second part_stride elements on).
+int launch_tanh_rows(int act, const float* raw, int ld, void* out, int ldo, size_t part_stride, int n, int T, const LaunchCfg& cfg);
+// out[t][i] = clamped_glu of the pair (gate, up) i of a row laid out as LIN_GLU's.
+int launch_st_glu_rows(int act, const float* raw, int ld, void* out, int ldo, int ff, float limit, float slope, int T, const LaunchCfg& cfg);
+// out[t][h] = o[t][h] / rms(o[t][h]) * w[h] * silu(gate[t][h]) * scale, heads of n values np apart.
+struct HeadNormArgs { const float* o; int ldo, heads, n, np; const float* w; int w_hs; const float* gate; int ldg; float eps, scale; void* out; int ldout; };
+int launch_head_norm_gate(int act, const HeadNormArgs& a, int T, const LaunchCfg& cfg);
+
+constexpr int kRecurMaxDim = 512;                                   // key channels of a head
+
+// Time mixing (time_mix.cu).  State [heads][dimp (value channel)][dimp (key channel)].
+// time_mix_rows: z -> exp(-exp(z + w0)) in place; bonus[t][h] = sum_i r_i u_i k_i.
+struct TimeMixArgs {
+    const float *r, *k, *v; int ld;                                 // heads dimp apart
+    float* z; int ldz; const float *w0, *u; float* bonus;
+    int heads, dim, dimp, T;
+    float* state; float* o; int ldo;
+    const int* pos_ptr; int pos0;
+};
+int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg);
+int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg);
+// One token in bfloat16: low-rank decay, recurrence, head norm, gate - and, in the same launch, the token's qkv rows (qkv.raw null: none).
+struct TimeMixStepArgs {
+    const float *r, *k, *v, *g, *w1;                                // raw projections
+    const bf16* w2; int w2_pitch, rank; const float *w0, *u, *norm;
+    int heads, dim, dimp; float* state; float eps, scale; bf16* out;
+    const int* pos_ptr;
+    QkvRowsArgs qkv;
+};
+int launch_time_mix_step(const TimeMixStepArgs& a, const LaunchCfg& cfg);
+
+// Gated delta rule (delta_rule.cu).  State [heads][vdimp][dimp]; ring [taps][channels]: raw projections by position.
+// delta_rows: convolution, silu, unit vectors; per value head decay and step size.
+struct DeltaArgs {
+    const float* raw; int ld, k_off, v_off, g_off, a_off, b_off;    // raw rows [q | k | v | g | a | b]
+    const float* conv; int taps; float* ring;                       // conv [channels][taps], channels = g_off
+    const float *a_exp, *dt;                                        // exp(A_log), dt_bias [heads]
+    int heads, kv_heads, dim, dimp, vdim, vdimp, T;
+    float* qk; float* v; float4* sc;                                // [T][kv_heads][q dimp | k dimp], [T][heads * vdimp], [T][heads] (decay, step, k . q, -)
+    float* state; float* o; int ldo;
+    const int* pos_ptr; int pos0;
+};
+int launch_delta_rows(const DeltaArgs& a, const LaunchCfg& cfg);
+int launch_delta_scan(const DeltaArgs& a, const LaunchCfg& cfg);
+// One token in bfloat16: all of it, head norm and gate included.
+struct DeltaStepArgs { DeltaArgs d; const float* norm; float eps, scale; bf16* out; };
+int launch_delta_step(const DeltaStepArgs& a, const LaunchCfg& cfg);
 
 // (cos, sin) of pos * freq for every position; freq in double.
 int launch_rot_table(float2* table, int n_pos, int dims, double base, const LaunchCfg& cfg);

@@ -11,7 +11,8 @@ __device__ __forceinline__ void lin_store(const LinArgs& a, int t, int r, float 
         case LIN_F32: reinterpret_cast<float*>(a.out)[o] = v; break;
         case LIN_ACT: reinterpret_cast<A*>(a.out)[o] = to_act<A>(v); break;
         case LIN_RELU2: { const float p = fmaxf(v, 0.f); reinterpret_cast<A*>(a.out)[o] = to_act<A>(p * p); break; }
-        case LIN_ADD: reinterpret_cast<float*>(a.out)[o] += v; break;
+        case LIN_ADD: reinterpret_cast<float*>(a.out)[o] += a.c0 * v; break;
+        case LIN_CAP: reinterpret_cast<float*>(a.out)[o] = a.c0 * tanhf(v / a.c0); break;
         case LIN_GELU_SIDE: {
             const float e = r < a.side_dim ? __bfloat162float(a.side[(size_t)a.tokens[t] * a.side_pitch + r]) : 0.f;
             reinterpret_cast<A*>(a.out)[o] = to_act<A>(gelu_tanh_f(v) * e);
@@ -78,7 +79,7 @@ __global__ void __launch_bounds__(256) st_gemm_kernel(const LinArgs a) {
 }
 
 int launch_st_linear(int act, const LinArgs& a, const LaunchCfg& cfg) {
-    if (a.T < 1 || a.R < 1 || a.K < 1 || !a.x || !a.w || !a.out) return (int)cudaErrorInvalidValue;
+    if (a.T < 1 || a.R < 1 || a.K < 1 || !a.x || !a.w || !a.out || a.epi == LIN_GLU) return (int)cudaErrorInvalidValue;
     if (a.T == 1) {
         const dim3 grid((a.R + 7) / 8);
         return act == ACT_F32 ? st_launch(st_gemv_kernel<float>, grid, dim3(256), 0, cfg, a) : st_launch(st_gemv_kernel<bf16>, grid, dim3(256), 0, cfg, a);

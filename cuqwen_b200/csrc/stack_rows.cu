@@ -3,25 +3,27 @@
 
 namespace cq {
 
-__device__ __forceinline__ void embed_row(const bf16* src, float* dst, int width) {
+__device__ __forceinline__ void embed_row(const bf16* src, float* dst, int width, float scale) {
     for (int i = threadIdx.x; i < (width + 7) / 8; i += blockDim.x) {      // rows are padded with zeros to a multiple of eight
         float v[8];
         unpack8(ldg_stream(src + 8 * i), v);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] *= scale;
         store4(dst + 8 * i, make_float4(v[0], v[1], v[2], v[3]));
         store4(dst + 8 * i + 4, make_float4(v[4], v[5], v[6], v[7]));
     }
 }
-__global__ void __launch_bounds__(256) st_embed_kernel(const bf16* __restrict__ table, int pitch, const int* __restrict__ tokens, float* __restrict__ x, int ldx, int width) {
+__global__ void __launch_bounds__(256) st_embed_kernel(const bf16* __restrict__ table, int pitch, const int* __restrict__ tokens, float* __restrict__ x, int ldx, int width, float scale) {
     pdl_launch_dependents(); pdl_wait();
-    embed_row(table + (size_t)tokens[blockIdx.x] * pitch, x + (size_t)blockIdx.x * ldx, width);
+    embed_row(table + (size_t)tokens[blockIdx.x] * pitch, x + (size_t)blockIdx.x * ldx, width, scale);
 }
-int launch_st_embed(const bf16* table, int pitch, const int* tokens, float* x, int ldx, int width, int T, const LaunchCfg& cfg) {
-    return st_launch(st_embed_kernel, dim3(T), dim3(256), 0, cfg, table, pitch, tokens, x, ldx, width);
+int launch_st_embed(const bf16* table, int pitch, const int* tokens, float* x, int ldx, int width, float scale, int T, const LaunchCfg& cfg) {
+    return st_launch(st_embed_kernel, dim3(T), dim3(256), 0, cfg, table, pitch, tokens, x, ldx, width, scale);
 }
 
 // One CTA: thread 0 takes over what the host left in the mailbox before any dependent launch is released (as
 // embed_step_kernel does for the models of the table).
-__global__ void __launch_bounds__(256) st_embed_step_kernel(const bf16* __restrict__ table, int pitch, StepCtl* ctl, float* __restrict__ x, int width) {
+__global__ void __launch_bounds__(256) st_embed_step_kernel(const bf16* __restrict__ table, int pitch, StepCtl* ctl, float* __restrict__ x, int width, float scale) {
     if (threadIdx.x == 0 && ctl->hio && !ctl->auto_advance) {
         int sq, tk, ps, hl;
         asm volatile("ld.volatile.global.v4.s32 {%0,%1,%2,%3}, [%4];" : "=r"(sq), "=r"(tk), "=r"(ps), "=r"(hl) : "l"(ctl->hio) : "memory");
@@ -30,10 +32,10 @@ __global__ void __launch_bounds__(256) st_embed_step_kernel(const bf16* __restri
     }
     __syncthreads();
     pdl_launch_dependents();
-    embed_row(table + (size_t)(*(volatile int*)&ctl->token) * pitch, x, width);
+    embed_row(table + (size_t)(*(volatile int*)&ctl->token) * pitch, x, width, scale);
 }
-int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, int width, const LaunchCfg& cfg) {
-    return st_launch(st_embed_step_kernel, dim3(1), dim3(256), 0, cfg, table, pitch, ctl, x, width);
+int launch_st_embed_step(const bf16* table, int pitch, StepCtl* ctl, float* x, int width, float scale, const LaunchCfg& cfg) {
+    return st_launch(st_embed_step_kernel, dim3(1), dim3(256), 0, cfg, table, pitch, ctl, x, width, scale);
 }
 
 // ---- x += rmsnorm(y), then one or two norms of x ------------------------------------------------------------------------
