@@ -1,0 +1,203 @@
+// Time mixing: state S of a head with a decay per key channel, S <- diag(w) S + k v^T, read out before the update with a bonus
+// for the current token: o = S^T r + (sum_i r_i u_i k_i) v.  All of it in float32.
+//
+// Portions: the row kernel turns the low-rank products into decays and takes the bonus sums; the scan walks the tokens with the
+// state in registers (recur.cuh), r, k, decays and values brought a tile of tokens at a time by cp.async.  Value channels are
+// independent of one another, so a head is cut into CTAs of a few of them.
+#include "qkv_rows.cuh"
+#include "recur.cuh"
+
+namespace cq {
+
+// A warp per (row, head).
+__global__ void __launch_bounds__(256) time_mix_rows_kernel(const TimeMixArgs a) {
+    pdl_launch_dependents(); pdl_wait();
+    const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = blockIdx.x;
+    if (h >= a.heads) return;
+    const size_t o = (size_t)h * a.dimp;
+    const float *r = a.r + (size_t)t * a.ld + o, *k = a.k + (size_t)t * a.ld + o, *u = a.u + o, *w0 = a.w0 + o;
+    float* z = a.z + (size_t)t * a.ldz + o;
+    float b = 0.f;
+    for (int i = lane; i < a.dimp; i += 32) {
+        z[i] = expf(-expf(z[i] + w0[i]));
+        b = fmaf(r[i] * u[i], k[i], b);                 // padded places hold zeros
+    }
+    b = warp_sum(b);
+    if (lane == 0) a.bonus[(size_t)t * a.heads + h] = b;
+}
+int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg) {
+    return st_launch(time_mix_rows_kernel, dim3(a.T, (a.heads + 7) / 8), dim3(256), 0, cfg, a);
+}
+
+constexpr int kTmTile = 16;                             // tokens brought at a time
+// CTA: head x CB value channels, NC of them to a thread.
+template <int LPC, int NV, int NC, int CB>
+__global__ void __launch_bounds__(CB / NC * LPC) time_mix_scan_kernel(const TimeMixArgs a) {
+    constexpr int D = LPC * NV * 4, NT = CB / NC * LPC, ROW = 3 * D + CB + 4;            // r | k | w | v | bonus
+    extern __shared__ __align__(16) float tm_smem[];    // [2][kTmTile][ROW]
+    pdl_launch_dependents(); pdl_wait();
+    const int h = blockIdx.x, c0 = blockIdx.y * CB, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC;
+    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0, nc = min(CB, a.dimp - c0);
+    const size_t ho = (size_t)h * a.dimp;
+    for (int i = tid; i < 2 * kTmTile * ROW; i += NT) tm_smem[i] = 0.f;                 // what no copy reaches stays zero
+    __syncthreads();
+    auto bring = [&](int t0, int b) {
+        const int n = min(kTmTile, a.T - t0), du = a.dimp / 4, cu = nc / 4, per = 3 * du + cu;
+        for (int i = tid; i < n * per; i += NT) {
+            const int t = i / per, u = i - t * per, tt = t0 + t;
+            float* dst = tm_smem + (b * kTmTile + t) * ROW;
+            if (u < du) cp_async16(dst + 4 * u, a.r + (size_t)tt * a.ld + ho + 4 * u);
+            else if (u < 2 * du) cp_async16(dst + D + 4 * (u - du), a.k + (size_t)tt * a.ld + ho + 4 * (u - du));
+            else if (u < 3 * du) cp_async16(dst + 2 * D + 4 * (u - 2 * du), a.z + (size_t)tt * a.ldz + ho + 4 * (u - 2 * du));
+            else cp_async16(dst + 3 * D + 4 * (u - 3 * du), a.v + (size_t)tt * a.ld + ho + c0 + 4 * (u - 3 * du));
+        }
+        for (int t = tid; t < n; t += NT) tm_smem[(b * kTmTile + t) * ROW + 3 * D + CB] = a.bonus[(size_t)(t0 + t) * a.heads + h];
+        cp_async_commit();
+    };
+    bring(0, 0);
+    StateCol<LPC, NV> s[NC];
+    float* st[NC];
+#pragma unroll
+    for (int j = 0; j < NC; ++j) {
+        const int c = c0 + cg * NC + j;
+        st[j] = a.state + (ho + c) * a.dimp;
+        if (c < a.dimp && first > 0) s[j].load(st[j], l, a.dimp); else s[j].zero();
+    }
+    for (int t0 = 0, b = 0; t0 < a.T; t0 += kTmTile, b ^= 1) {
+        if (t0 + kTmTile < a.T) { bring(t0 + kTmTile, b ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
+        __syncthreads();
+        const int n = min(kTmTile, a.T - t0);
+#pragma unroll 2
+        for (int t = 0; t < n; ++t) {
+            const float* row = tm_smem + (b * kTmTile + t) * ROW;
+            f32x2 r[2 * NV], k[2 * NV], w[2 * NV];
+            lane_units<LPC, NV>(row, l, r); lane_units<LPC, NV>(row + D, l, k); lane_units<LPC, NV>(row + 2 * D, l, w);
+            const float bonus = row[3 * D + CB];
+            float o[NC];
+#pragma unroll
+            for (int j = 0; j < NC; ++j) {
+                const float v = row[3 * D + cg * NC + j];
+                const f32x2 v2 = pack2(v, v);
+                f32x2 acc = 0ull, acc1 = 0ull;
+#pragma unroll
+                for (int i = 0; i < 2 * NV; i += 2) {
+                    acc = fma2(s[j].s[i], r[i], acc); acc1 = fma2(s[j].s[i + 1], r[i + 1], acc1);
+                    s[j].s[i] = fma2(s[j].s[i], w[i], mul2(k[i], v2)); s[j].s[i + 1] = fma2(s[j].s[i + 1], w[i + 1], mul2(k[i + 1], v2));
+                }
+                o[j] = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v;
+            }
+            if (l == 0) {
+#pragma unroll
+                for (int j = 0; j < NC; ++j) { const int c = c0 + cg * NC + j; if (c < a.dimp) a.o[(size_t)(t0 + t) * a.ldo + ho + c] = o[j]; }
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int j = 0; j < NC; ++j) if (c0 + cg * NC + j < a.dimp) s[j].store(st[j], l, a.dimp);
+}
+template <int LPC, int NV>
+static int tm_go(const TimeMixArgs& a, const LaunchCfg& cfg) {
+    constexpr int NC = 2, CB = 32, D = LPC * NV * 4;
+    const size_t smem = (size_t)2 * kTmTile * (3 * D + CB + 4) * 4;
+    static bool once = false;
+    if (!once) {
+        const cudaError_t e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e != cudaSuccess) return (int)e;
+        once = true;
+    }
+    return st_launch(time_mix_scan_kernel<LPC, NV, NC, CB>, dim3(a.heads, (a.dimp + CB - 1) / CB), dim3(CB / NC * LPC), smem, cfg, a);
+}
+int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg) {
+    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.ld % 4 || a.ldz % 4) return (int)cudaErrorInvalidValue;
+#define GO(L, N) tm_go<L, N>(a, cfg)
+    return RECUR_DISPATCH(a.dimp, GO);
+#undef GO
+}
+
+// ---- one token --------------------------------------------------------------------------------------------------------
+// CTA = head; the three CTAs behind the heads put the token's q, k and v rows in place.  The state of the first value channels is
+// on its way before the dependency wait (it was written by an earlier step).
+constexpr int kTsThreads = 512, kTsHold = 2;            // channels of a thread held at a time
+template <int LPC, int NV>
+__global__ void __launch_bounds__(kTsThreads) time_mix_step_kernel(const TimeMixStepArgs a) {
+    constexpr int D = LPC * NV * 4, CH = kTsThreads / LPC;                               // value channels at a time
+    extern __shared__ __align__(16) float ts_smem[];    // r [D], k [D], w [D], tanh [rank], o [dimp]
+    __shared__ float red[40];
+    pdl_launch_dependents();
+    const int h = blockIdx.x, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC, pos = *a.pos_ptr;      // written before the step's first kernel released its dependents
+    if (h >= a.heads) {
+        pdl_wait();
+        qkv_section<bf16>(a.qkv, 0, pos, h - a.heads, tid, kTsThreads);
+        return;
+    }
+    float *r = ts_smem, *k = r + D, *w = k + D, *o = w + D, *th = o + a.dimp;
+    const size_t ho = (size_t)h * a.dimp;
+    StateCol<LPC, NV> s[kTsHold];
+    auto fetch = [&](int c0) {
+#pragma unroll
+        for (int j = 0; j < kTsHold; ++j) {
+            const int c = c0 + j * CH + cg;
+            if (c < a.dimp && pos > 0) s[j].load(a.state + (ho + c) * a.dimp, l, a.dimp); else s[j].zero();
+        }
+    };
+    fetch(0);
+    pdl_wait();
+    float b = 0.f;
+    for (int i = tid; i < D; i += kTsThreads) {
+        const bool in = i < a.dimp;
+        const float rv = in ? __ldcg(a.r + ho + i) : 0.f, kv = in ? __ldcg(a.k + ho + i) : 0.f;
+        r[i] = rv; k[i] = kv; w[i] = 0.f;
+        if (in) b = fmaf(rv * a.u[ho + i], kv, b);
+    }
+    for (int i = tid; i < a.rank; i += kTsThreads) th[i] = tanhf(__ldcg(a.w1 + i));
+    const float bonus = cta_sum(b, red);                // barriers inside
+    // decays: a warp per key channel
+    for (int i = tid >> 5; i < a.dimp; i += kTsThreads / 32) {
+        const bf16* row = a.w2 + (ho + i) * a.w2_pitch;
+        float z = 0.f;
+        for (int q = tid & 31; q < a.rank; q += 32) z = fmaf(th[q], __bfloat162float(row[q]), z);
+        z = warp_sum(z);
+        if ((tid & 31) == 0) w[i] = expf(-expf(z + a.w0[ho + i]));
+    }
+    __syncthreads();
+    f32x2 rr[2 * NV], kk[2 * NV], ww[2 * NV];
+    lane_units<LPC, NV>(r, l, rr); lane_units<LPC, NV>(k, l, kk); lane_units<LPC, NV>(w, l, ww);
+    float ss = 0.f;
+    for (int c0 = 0; c0 < a.dimp; c0 += kTsHold * CH) {
+        if (c0) fetch(c0);
+#pragma unroll
+        for (int j = 0; j < kTsHold; ++j) {
+            const int c = c0 + j * CH + cg;
+            const float v = c < a.dimp ? __ldcg(a.v + ho + c) : 0.f;
+            const f32x2 v2 = pack2(v, v);
+            f32x2 acc = 0ull, acc1 = 0ull;
+#pragma unroll
+            for (int i = 0; i < 2 * NV; i += 2) {
+                acc = fma2(s[j].s[i], rr[i], acc); acc1 = fma2(s[j].s[i + 1], rr[i + 1], acc1);
+                s[j].s[i] = fma2(s[j].s[i], ww[i], mul2(kk[i], v2)); s[j].s[i + 1] = fma2(s[j].s[i + 1], ww[i + 1], mul2(kk[i + 1], v2));
+            }
+            const float x = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v;
+            if (c < a.dimp) {
+                s[j].store(a.state + (ho + c) * a.dimp, l, a.dimp);
+                if (l == 0) { o[c] = x; ss = fmaf(x, x, ss); }
+            }
+        }
+    }
+    const float inv = inv_rms(cta_sum(ss, red), a.dim, a.eps) * a.scale;
+    for (int c = tid; c < a.dimp; c += kTsThreads) a.out[ho + c] = __float2bfloat16_rn(c < a.dim ? o[c] * inv * a.norm[ho + c] * silu_f(__ldcg(a.g + ho + c)) : 0.f);
+}
+template <int LPC, int NV>
+static int ts_go(const TimeMixStepArgs& a, const LaunchCfg& cfg) {
+    const size_t smem = (size_t)(3 * LPC * NV * 4 + a.dimp + a.rank) * 4;
+    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+    return st_launch(time_mix_step_kernel<LPC, NV>, dim3(a.heads + (a.qkv.raw ? 3 : 0)), dim3(kTsThreads), smem, cfg, a);
+}
+int launch_time_mix_step(const TimeMixStepArgs& a, const LaunchCfg& cfg) {
+    if (a.heads < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.rank < 1 || (a.qkv.raw && !qkv_rows_ok(a.qkv))) return (int)cudaErrorInvalidValue;
+#define GO(L, N) ts_go<L, N>(a, cfg)
+    return RECUR_DISPATCH(a.dimp, GO);
+#undef GO
+}
+
+}  // namespace cq
