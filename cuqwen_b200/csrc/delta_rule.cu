@@ -12,11 +12,10 @@ constexpr float kUnitEps = 1e-6f;                       // added to the sum of s
 
 // One channel's convolution and silu at row t (position pos): earlier rows of the portion, before them the ring.
 __device__ __forceinline__ float delta_conv(const DeltaArgs& a, int t, int pos, int ch) {
-    const float* w = a.conv + (size_t)ch * a.taps;
     float s = 0.f;
     for (int j = 0; j < a.taps && j <= pos; ++j) {      // j rows back
         const float x = t - j >= 0 ? __ldcg(a.raw + (size_t)(t - j) * a.ld + ch) : a.ring[(size_t)((pos - j) % a.taps) * a.g_off + ch];
-        s = fmaf(w[a.taps - 1 - j], x, s);
+        s = fmaf(a.conv[(size_t)(a.taps - 1 - j) * a.g_off + ch], x, s);
     }
     return silu_f(s);
 }

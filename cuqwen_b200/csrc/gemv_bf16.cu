@@ -44,7 +44,7 @@ __device__ __forceinline__ float seg_inv_rms(float ss, int n, float eps, float* 
 
 // The input vector as bfloat16 in shared memory.  A thread owns the float4 units tid, tid + 256, ... of the vector from the
 // first load to the last store, so only the sums need barriers.
-__device__ __forceinline__ void seg_stage(const SegGemvArgs& a, unsigned char* sm, const SegLayout& L, bool first) {
+__device__ __forceinline__ void seg_stage(const SegGemvArgs& a, unsigned char* sm, const SegLayout& L, bool first, unsigned vars) {
     const int tid = threadIdx.x;
     if (a.stage == SEG_PLAIN) {
         uint4* xs = reinterpret_cast<uint4*>(sm + L.off_x);
@@ -90,8 +90,35 @@ __device__ __forceinline__ void seg_stage(const SegGemvArgs& a, unsigned char* s
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
     }
-    const bool norm = a.stage == SEG_NORM;
+    const bool norm = a.stage == SEG_NORM || a.stage == SEG_MIX;
     const float inv = norm ? seg_inv_rms(ss, a.width, a.eps, red) : 1.f;
+    if (a.stage == SEG_MIX) {
+        const int pos = *a.pos_ptr;
+        const float4 *w = reinterpret_cast<const float4*>(a.nw[0]), *prev = reinterpret_cast<const float4*>(a.prev + (size_t)((pos + 1) & 1) * a.ldprev);
+        float4* keep = reinterpret_cast<float4*>(a.prev + (size_t)(pos & 1) * a.ldprev);
+#pragma unroll 2
+        for (int i = tid; i < k4; i += kSgNC) {
+            float4 h = make_float4(0.f, 0.f, 0.f, 0.f), p = h;
+            if (i < n4) {
+                h = xf[i];
+                const float4 g = __ldg(w + i);
+                if (pos > 0) p = __ldcg(prev + i);
+                h.x *= inv * g.x; h.y *= inv * g.y; h.z *= inv * g.z; h.w *= inv * g.w;
+                if (first) keep[i] = h;
+            }
+            for (int k = 0; k < a.nvar; ++k) {
+                if (!(vars >> k & 1u)) continue;
+                float4 v = h;
+                if (k > 0 && i < n4) {
+                    const float4 m = __ldg(reinterpret_cast<const float4*>(a.mu + (size_t)(k - 1) * a.ldmu) + i);
+                    v = make_float4(fmaf(p.x - h.x, m.x, h.x), fmaf(p.y - h.y, m.y, h.y), fmaf(p.z - h.z, m.z, h.z), fmaf(p.w - h.w, m.w, h.w));
+                }
+                reinterpret_cast<uint2*>(sm + L.off_x + k * a.K * 2)[i] = make_uint2(pack_bf(v.x, v.y), pack_bf(v.z, v.w));
+            }
+        }
+        consumer_sync(kSgNC);
+        return;
+    }
     for (int k = 0; k < a.nvar; ++k) {
         uint2* o = reinterpret_cast<uint2*>(sm + L.off_x + k * a.K * 2);
         const float4* w = reinterpret_cast<const float4*>(a.nw[k]);
@@ -114,9 +141,14 @@ __device__ __forceinline__ void seg_finish(const SegGemvArgs& a, int seg, int ro
         case LIN_F32: reinterpret_cast<float*>(a.out[seg])[row] = v; break;
         case LIN_ACT: reinterpret_cast<bf16*>(a.out[seg])[row] = __float2bfloat16_rn(v); break;
         case LIN_RELU2: { const float p = fmaxf(v, 0.f); reinterpret_cast<bf16*>(a.out[seg])[row] = __float2bfloat16_rn(p * p); break; }
-        case LIN_ADD: reinterpret_cast<float*>(a.out[seg])[row] = pre + v; break;
+        case LIN_ADD: reinterpret_cast<float*>(a.out[seg])[row] = pre + a.c0 * v; break;
+        case LIN_CAP: reinterpret_cast<float*>(a.out[seg])[row] = a.c0 * tanhf(v / a.c0); break;
         case LIN_GELU_SIDE: reinterpret_cast<bf16*>(a.out[seg])[row] = __float2bfloat16_rn(gelu_tanh_f(v) * pre); break;
     }
+}
+// Row `row` of the gate and row + 8 of the up matrix (LIN_GLU: eight rows of each in turn).
+__device__ __forceinline__ void seg_finish_glu(const SegGemvArgs& a, int seg, int row, float gate, float up) {
+    reinterpret_cast<bf16*>(a.out[seg])[(row >> 4) * 8 + (row & 7)] = __float2bfloat16_rn(clamped_glu_f(gate, up, a.c0, a.c1));
 }
 // The epilogue's operand from global memory, fetched before the block's arithmetic.
 __device__ __forceinline__ float seg_fetch(const SegGemvArgs& a, int seg, int row, int row_end) {
@@ -183,7 +215,14 @@ __global__ void __launch_bounds__(kSgThreads, 1) gemv_seg_kernel(const __grid_co
         return;
     }
     pdl_wait();
-    seg_stage(a, sg_smem, L, blockIdx.x == 0);
+    unsigned vars = 0;                                          // copies of the input that this CTA's segments read
+    if (a.stage == SEG_MIX)
+        for (int blk = blockIdx.x; blk < a.nblk; blk += ncta) {
+            int seg = 0;
+            while (seg + 1 < a.nseg && blk >= a.seg_blk0[seg + 1]) ++seg;
+            vars |= 1u << a.seg_var[seg];
+        }
+    seg_stage(a, sg_smem, L, blockIdx.x == 0, vars);
     float* red = reinterpret_cast<float*>(sg_smem + L.off_red);
     const int g = lane >> 2, t = lane & 3, rwi = warp % a.rw, kwi = warp / a.rw;
     const int cstride = a.brows * kChunkBytes;
@@ -221,22 +260,31 @@ __global__ void __launch_bounds__(kSgThreads, 1) gemv_seg_kernel(const __grid_co
         if (kw > 1) {
             if (t == 0) { red[warp * 16 + g] = vA; red[warp * 16 + g + 8] = vB; }
             consumer_sync(kSgNC);
-            if (kwi == 0 && lane < 16 && row0 + lane < row_end) {
+            if (a.epi[seg] == LIN_GLU) {
+                if (kwi == 0 && lane < 8 && row0 + lane < row_end) {
+                    float v = 0.f, u = 0.f;
+                    for (int k = 0; k < kw; ++k) { v += red[(k * a.rw + rwi) * 16 + lane]; u += red[(k * a.rw + rwi) * 16 + lane + 8]; }
+                    seg_finish_glu(a, seg, row0 + lane, v, u);
+                }
+            } else if (kwi == 0 && lane < 16 && row0 + lane < row_end) {
                 float v = 0.f;
                 for (int k = 0; k < kw; ++k) v += red[(k * a.rw + rwi) * 16 + lane];
                 seg_finish(a, seg, row0 + lane, v, preA);
             }
             consumer_sync(kSgNC);
         } else if (t == 0 && live) {
-            if (row0 + g < row_end) seg_finish(a, seg, row0 + g, vA, preA);
-            if (row0 + g + 8 < row_end) seg_finish(a, seg, row0 + g + 8, vB, preB);
+            if (a.epi[seg] == LIN_GLU) { if (row0 + g < row_end) seg_finish_glu(a, seg, row0 + g, vA, vB); }
+            else {
+                if (row0 + g < row_end) seg_finish(a, seg, row0 + g, vA, preA);
+                if (row0 + g + 8 < row_end) seg_finish(a, seg, row0 + g + 8, vB, preB);
+            }
         }
     }
 }
 
 int launch_gemv_seg(SegGemvArgs& a, const SegMat* mats, int nmat, const LaunchCfg& cfg) {
     const bool two = a.stage == SEG_PLAIN && a.kp[1] > 0;
-    if (nmat < 1 || nmat > 4 || (two && nmat != 2) || a.K < 128 || a.K % 128 || (a.stage == SEG_PLAIN && a.K != a.kp[0] + a.kp[1])) return (int)cudaErrorInvalidValue;
+    if (nmat < 1 || nmat > kSegMax || (two && nmat != 2) || a.K < 128 || a.K % 128 || (a.stage == SEG_PLAIN && a.K != a.kp[0] + a.kp[1])) return (int)cudaErrorInvalidValue;
     a.nseg = two ? 1 : nmat;
     int total = 0;
     for (int s = 0; s < a.nseg; ++s) { a.seg_rows[s] = mats[s].rows; total += mats[s].rows; }
@@ -245,8 +293,12 @@ int launch_gemv_seg(SegGemvArgs& a, const SegMat* mats, int nmat, const LaunchCf
     const int rounds = (total + 128 * sms - 1) / (128 * sms);
     int brows = (total + rounds * sms - 1) / (rounds * sms);
     if (brows < 8) brows = 8;
+    bool glu = false;                                // its pairs of rows lie in one 16-row tile
+    for (int s = 0; s < a.nseg; ++s) if (a.epi[s] == LIN_GLU) { glu = true; if (mats[s].rows % 16) return (int)cudaErrorInvalidValue; }
+    const int step = glu ? 16 : 1;
+    brows = (brows + step - 1) / step * step;
     auto blocks = [&](int br) { int n = 0; for (int s = 0; s < a.nseg; ++s) n += (mats[s].rows + br - 1) / br; return n; };
-    while (brows < 128 && blocks(brows) > rounds * sms) ++brows;
+    while (brows < 128 && blocks(brows) > rounds * sms) brows += step;
     a.brows = brows;
     a.nblk = 0;
     for (int s = 0; s < a.nseg; ++s) { a.seg_blk0[s] = a.nblk; a.nblk += (mats[s].rows + brows - 1) / brows; }

@@ -8,6 +8,10 @@
 // latent_fold_kernel: grid (heads, slices of 32 value rows): merges the ranges and the sink - up to eight slices of a head
 // form a cluster whose CTAs merge a share of the columns each and exchange them through distributed shared memory -
 // multiplies the head's latent output with W_uv, applies the gate.
+//
+// Grouped attention runs the same partial kernel over a cache per key / value head whose rows are [key | value]: the groups of
+// sixteen are cut from the query heads of one key / value head, the score stops at the key's end, P V starts there.
+// grouped_fold_kernel merges the ranges.
 #include "stack_dev.cuh"
 #include "tma.cuh"
 
@@ -54,13 +58,17 @@ __global__ void __launch_bounds__(kLdThreads) latent_partial_kernel(const Latent
     bf16* P = reinterpret_cast<bf16*>(S + kLdHeads * (kLdTile + 2));                             // [16][72]
     float* rowf = reinterpret_cast<float*>(P + kLdHeads * (kLdTile + 8));                        // rescale factor, max, sum per head
     const uint32_t sp = smem_u32(P);
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h0 = blockIdx.y * kLdHeads;
-    const int nh = min(kLdHeads, a.heads - h0);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tiles16 = (a.group + kLdHeads - 1) / kLdHeads, kvh = a.group ? blockIdx.y / tiles16 : 0, sub = a.group ? blockIdx.y % tiles16 * kLdHeads : 0;
+    const int h0 = a.group ? kvh * a.group + sub : blockIdx.y * kLdHeads;
+    const int nh = min(kLdHeads, a.group ? a.group - sub : a.heads - h0);
+    const bf16* cache = a.cache + (size_t)kvh * a.kv_stride;
+    const int qrow = a.group ? a.kdim : a.crow, qunits = qrow / 8;
     pdl_launch_dependents();
     const int pos = *a.pos_ptr;                 // written before the step's first kernel released its dependents
     int lo, hi;
     ld_range(a, pos, blockIdx.x, lo, hi);
-    const int units = a.crow / 8, ksteps = (a.crow + 15) / 16;
+    const int units = a.crow / 8, ksteps = (qrow + 15) / 16;
     if (lo >= hi) {                             // an empty range: the fold skips it
         pdl_wait();
         if (tid < nh) { float* ml = a.part_ml + ((size_t)blockIdx.x * a.heads + h0 + tid) * 2; ml[0] = -INFINITY; ml[1] = 0.f; }
@@ -75,7 +83,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_partial_kernel(const Latent
             const int r = i / units, u = i - r * units, k = k0 + r;
             const uint32_t dst = sk + (b * kLdTile + r) * pb + u * 16;
             if (k >= hi) { if (only != 2) *reinterpret_cast<uint4*>(ld_raw + (dst - sk)) = make_uint4(0u, 0u, 0u, 0u); }
-            else if (only == 0 || (only == 2) == (k == pos)) ld_cp16(dst, a.cache + (size_t)k * a.crow + u * 8);
+            else if (only == 0 || (only == 2) == (k == pos)) ld_cp16(dst, cache + (size_t)k * a.crow + u * 8);
         }
     };
     load(lo, 0, 1);
@@ -85,7 +93,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_partial_kernel(const Latent
     for (int i = tid; i < kLdHeads * units; i += kLdThreads) {
         const int r = i / units, u = i - r * units;
         unsigned char* dst = ld_raw + (size_t)(2 * kLdTile + r) * pb + u * 16;
-        if (r < nh) ld_cp16(smem_u32(dst), a.q + (size_t)(h0 + r) * a.crow + u * 8);
+        if (r < nh && u < qunits) ld_cp16(smem_u32(dst), a.q + (size_t)(h0 + r) * qrow + u * 8);
         else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
     }
     ld_commit();
@@ -158,7 +166,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_partial_kernel(const Latent
         for (int ks = 0; ks < kLdTile / 16; ++ks) {
             uint32_t pf[4];
             ld_sm4(sp + (lane & 15) * (kLdTile + 8) * 2 + (ks * 16 + (lane >> 4) * 8) * 2, pf);
-            const uint32_t va = sk + (b * kLdTile + ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pb + (lane >> 4) * 16;
+            const uint32_t va = sk + (b * kLdTile + ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pb + (lane >> 4) * 16 + (a.group ? a.kdim * 2 : 0);
 #pragma unroll
             for (int p = 0; p < MAXP; ++p) {
                 const int pair = warp + p * 8;
@@ -302,10 +310,67 @@ __global__ void __launch_bounds__(256) latent_fold_kernel(const LatentDecodeArgs
     }
 }
 
+// CTA = (head, 128 value columns): a warp takes every eighth key range, a lane four columns.
+__global__ void __launch_bounds__(256) grouped_fold_kernel(const LatentDecodeArgs a) {
+    __shared__ float wgt[kLdMaxSplit];
+    __shared__ float red[16];
+    __shared__ __align__(16) float mrg[8][128];
+    const int h = blockIdx.x, cb = blockIdx.y * 128, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c = cb + lane * 4;
+    pdl_launch_dependents(); pdl_wait();
+    const float* po = a.part_o + (size_t)h * a.kvrp;
+    const size_t ps = (size_t)a.heads * a.kvrp;
+    float4 pre[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) pre[k] = c < a.kvrp && warp + 8 * k < a.nsplit ? __ldcg(reinterpret_cast<const float4*>(po + (warp + 8 * k) * ps + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float m = -INFINITY, l = 0.f;
+    if (tid < a.nsplit) {
+        const float2 v = __ldcg(reinterpret_cast<const float2*>(a.part_ml) + (size_t)tid * a.heads + h);
+        m = v.x; l = v.y;
+    }
+    float mx = m;
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+    if (lane == 0) red[warp] = mx;
+    __syncthreads();
+    mx = red[0];
+#pragma unroll
+    for (int i = 1; i < 8; ++i) mx = fmaxf(mx, red[i]);
+    const float e = m == -INFINITY ? 0.f : expf(m - mx);                // a range without keys weighs nothing (its partials are an earlier step's, finite)
+    const float s = warp_sum(e * l);
+    if (lane == 0) red[8 + warp] = s;
+    if (tid < a.nsplit) wgt[tid] = e;
+    __syncthreads();
+    float den = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) den += red[8 + i];
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto acc = [&](float f, float4 v) { o.x = fmaf(f, v.x, o.x); o.y = fmaf(f, v.y, o.y); o.z = fmaf(f, v.z, o.z); o.w = fmaf(f, v.w, o.w); };
+#pragma unroll
+    for (int k = 0; k < 8; ++k) if (warp + 8 * k < a.nsplit) acc(wgt[warp + 8 * k], pre[k]);
+    if (c < a.kvrp)
+        for (int k = warp + 64; k < a.nsplit; k += 8) acc(wgt[k], __ldcg(reinterpret_cast<const float4*>(po + k * ps + c)));
+    reinterpret_cast<float4*>(mrg[warp])[lane] = o;
+    __syncthreads();
+    if (tid < 128 && cb + tid < a.kvrp) {
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += mrg[k][tid];
+        a.out[(size_t)h * a.o_hs + cb + tid] = __float2bfloat16_rn(v * (a.out_scale / den));
+    }
+}
+
 int latent_decode_splits(int heads, int crow, int kvrp, int window, int max_seq, int sm_count) {
     if (ld_smem(crow) > 225 * 1024 || kvrp > 1024) return 0;
     const int groups = (heads + kLdHeads - 1) / kLdHeads;
     const int keys = window > 0 && window < max_seq ? window : max_seq, tiles = (keys + kLdTile - 1) / kLdTile;
+    int n = sm_count / groups;
+    if (n > kLdMaxSplit) n = kLdMaxSplit;
+    if (n > tiles) n = tiles;
+    return n < 1 ? 1 : n;
+}
+int grouped_decode_splits(int heads, int kv_heads, int kdim, int vdimp, int max_seq, int sm_count) {
+    if (ld_smem(kdim + vdimp) > 225 * 1024 || vdimp > 1024) return 0;
+    const int groups = kv_heads * ((heads / kv_heads + kLdHeads - 1) / kLdHeads), tiles = (max_seq + kLdTile - 1) / kLdTile;
     int n = sm_count / groups;
     if (n > kLdMaxSplit) n = kLdMaxSplit;
     if (n > tiles) n = tiles;
@@ -320,11 +385,17 @@ static int ld_go(const LatentDecodeArgs& a, const LaunchCfg& cfg) {
         if (e != cudaSuccess) return (int)e;
         once = true;
     }
-    return st_launch(latent_partial_kernel<MAXP>, dim3(a.nsplit, (a.heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads), (size_t)ld_smem(a.crow), cfg, a);
+    return st_launch(latent_partial_kernel<MAXP>, dim3(a.nsplit, a.group ? a.heads / a.group * ((a.group + kLdHeads - 1) / kLdHeads) : (a.heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads), (size_t)ld_smem(a.crow), cfg, a);
+}
+static int ld_partial(const LatentDecodeArgs& a, const LaunchCfg& cfg) { return a.kvrp <= 128 ? ld_go<1>(a, cfg) : a.kvrp <= 512 ? ld_go<4>(a, cfg) : ld_go<8>(a, cfg); }
+int launch_grouped_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done) {
+    if (a.group < 1 || a.heads % a.group || a.kdim % 8 || a.kvrp % 8 || a.crow != a.kdim + a.kvrp || a.kvrp > 1024 || a.nsplit < 1 || a.nsplit > kLdMaxSplit) return done((int)cudaErrorInvalidValue, "grouped_decode");
+    if (int r = done(ld_partial(a, cfg), "grouped_partial")) return r;
+    return done(st_launch(grouped_fold_kernel, dim3(a.heads, (a.kvrp + 127) / 128), dim3(256), 0, cfg, a), "grouped_fold");
 }
 int launch_latent_decode(const LatentDecodeArgs& a, const LaunchCfg& cfg, const std::function<int(int, const char*)>& done) {
-    if (a.crow % 8 || a.kvrp % 8 || a.kvrp > 1024 || a.nsplit < 1 || a.nsplit > kLdMaxSplit || a.heads < 1) return done((int)cudaErrorInvalidValue, "latent_decode");
-    if (int r = done(a.kvrp <= 128 ? ld_go<1>(a, cfg) : a.kvrp <= 512 ? ld_go<4>(a, cfg) : ld_go<8>(a, cfg), "latent_partial")) return r;
+    if (a.group || a.crow % 8 || a.kvrp % 8 || a.kvrp > 1024 || a.nsplit < 1 || a.nsplit > kLdMaxSplit || a.heads < 1) return done((int)cudaErrorInvalidValue, "latent_decode");
+    if (int r = done(ld_partial(a, cfg), "latent_partial")) return r;
     const int slices = (a.vdim + kLfRows - 1) / kLfRows;
     LatentDecodeArgs f = a;
     f.ncl = slices <= 8 ? slices : 1;

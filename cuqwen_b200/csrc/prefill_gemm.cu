@@ -74,8 +74,29 @@ __device__ __forceinline__ void pf_store_bf16(const PfGemmArgs& a, const float (
         for (int i = 0; i < 32; i += 4)
             if (r + i < R) {
                 float4 o = *reinterpret_cast<float4*>(dst + i);
-                o.x += v[i]; o.y += v[i + 1]; o.z += v[i + 2]; o.w += v[i + 3];
+                o.x = fmaf(a.c0, v[i], o.x); o.y = fmaf(a.c0, v[i + 1], o.y); o.z = fmaf(a.c0, v[i + 2], o.z); o.w = fmaf(a.c0, v[i + 3], o.w);
                 *reinterpret_cast<float4*>(dst + i) = o;
+            }
+        return;
+    }
+    if (a.mode == PF_CAP_F32) {
+        float* dst = a.out_f + (size_t)token * a.ldo + coff + r;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4)
+            if (r + i < R)
+                *reinterpret_cast<float4*>(dst + i) = make_float4(a.c0 * tanhf(v[i] / a.c0), a.c0 * tanhf(v[i + 1] / a.c0), a.c0 * tanhf(v[i + 2] / a.c0), a.c0 * tanhf(v[i + 3] / a.c0));
+        return;
+    }
+    if (a.mode == PF_BF16_GLU) {
+        __nv_bfloat16* dst = a.out_b + (size_t)token * a.ldo + r / 2;
+#pragma unroll
+        for (int i = 0; i < 32; i += 16)
+            if (r + i < R) {
+                uint32_t o[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    o[k] = pack_bf(clamped_glu_f(v[i + 2 * k], v[i + 8 + 2 * k], a.c0, a.c1), clamped_glu_f(v[i + 2 * k + 1], v[i + 9 + 2 * k], a.c0, a.c1));
+                *reinterpret_cast<uint4*>(dst + i / 2) = make_uint4(o[0], o[1], o[2], o[3]);
             }
         return;
     }
@@ -124,7 +145,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
     if (!swiglu)
         while (seg + 1 < a.nseg && tseg >= (a.seg_rows[seg] + NT - 1) / NT) { tseg -= (a.seg_rows[seg] + NT - 1) / NT; coff += a.seg_rows[seg]; ++seg; }
     const int row0 = tseg * rows_mat;                         // first row inside the matrix
-    const int R = a.seg_rows[seg];
+    const int R = a.seg_rows[seg], xrow = Q == Q_BF16 ? a.seg_xrow[seg] : 0;
     const int nk1 = (a.K + kPfKB - 1) / kPfKB, nkb = Q == Q_BF16 ? nk1 + (a.K2 + kPfKB - 1) / kPfKB : nk1;      // columns past the end arrive as zeros
     constexpr int kRawKb = Q == Q_I4 ? 32 : 64;               // raw bytes of one row in one K block
     bool failed = false;
@@ -155,7 +176,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) prefill_gemm_kernel(const __gri
                     continue;
                 }
                 for (int h = 0; h < mh; ++h)        // a half that lies past the last token arrives as zeros
-                    tma_load_2d(ring_a + sa * kASlot + h * kPfABytes, &a.tx, kb * kPfKB, (tm * mh + h) * kPfM, bar_full + 8 * sa);
+                    tma_load_2d(ring_a + sa * kASlot + h * kPfABytes, &a.tx, kb * kPfKB, xrow + (tm * mh + h) * kPfM, bar_full + 8 * sa);
                 for (int m = 0; m < nmat; ++m) {
                     if (!kRaw) tma_load_2d(ring_b + sb * kPfBBytes + m * rows_mat * 128, &a.tw[seg + m], kb * kPfKB, row0, bar_full + 8 * sa);    // NB == NA: freed together
                     else tma_load_2d(ring_raw + sa * kRawBytes + m * rows_mat * kRawKb, &a.tw[seg + m], kb * kRawKb, row0, bar_full + 8 * sa);
@@ -380,7 +401,7 @@ int launch_prefill_gemm(int quant, PfGemmArgs& a, const void* x, const void* con
 }
 
 int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16Mat* m, int nmat, const void* x2, int ldx2, const PfBf16Mat* m2, cudaStream_t stream) {
-    if (a.T <= 0 || a.K <= 0 || a.K % 8 || a.ldo % 8 || ldx % 8 || nmat < 1 || nmat > 3 || (a.mode != PF_OUT_F32 && a.mode < PF_BF16) || (x2 && (nmat != 1 || !m2 || m2->rows != m->rows || a.K2 % 8 || ldx2 % 8)))
+    if (a.T <= 0 || a.K <= 0 || a.K % 8 || a.ldo % 8 || ldx % 8 || nmat < 1 || nmat > kPfMaxMat || (a.mode != PF_OUT_F32 && a.mode < PF_BF16) || (a.mode == PF_BF16_GLU && (nmat != 1 || m->rows % 16)) || (x2 && (nmat != 1 || !m2 || m2->rows != m->rows || a.K2 % 8 || ldx2 % 8)))
         return (int)cudaErrorInvalidValue;
     if (!x2) a.K2 = 0;
     int sms = 0, dev = 0;
@@ -396,10 +417,16 @@ int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16
     const int nt = (sms > 0 && wide * 4 <= sms) ? kPfN / 4 : (sms > 0 && wide * 2 <= sms) ? kPfN / 2 : kPfN;
     if (nt == kPfN / 4 && a.mh == 2) { a.mh = 1; mtiles = (a.T + kPfM - 1) / kPfM; }       // few rows: a token half per CTA, twice the CTAs
     const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-    if (int r = pf_map(&a.tx, x, bf, 2, (size_t)a.T, (size_t)a.K, kPfKB, kPfM, true, (size_t)ldx)) return r;
+    int xrows = a.T;
+    for (int i = 0; i < nmat; ++i) {
+        if (m[i].xrow < 0) return (int)cudaErrorInvalidValue;
+        if (m[i].xrow + a.T > xrows) xrows = m[i].xrow + a.T;
+    }
+    if (int r = pf_map(&a.tx, x, bf, 2, (size_t)xrows, (size_t)a.K, kPfKB, kPfM, true, (size_t)ldx)) return r;
     int tiles = 0;
     a.R = 0;
     for (int i = 0; i < nmat; ++i) {
+        a.seg_xrow[i] = m[i].xrow;
         if (!m[i].w || m[i].rows <= 0 || m[i].rows % 8 || m[i].pitch % 8 || m[i].pitch < a.K) return (int)cudaErrorInvalidValue;
         if (int r = pf_map(&a.tw[i], m[i].w, bf, 2, (size_t)m[i].rows, (size_t)a.K, kPfKB, nt, true, (size_t)m[i].pitch)) return r;
         a.seg_rows[i] = m[i].rows;

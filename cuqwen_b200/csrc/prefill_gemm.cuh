@@ -48,18 +48,22 @@ enum PfMode : int {
     // bfloat16 weights and activations (Q_BF16; PF_OUT_F32 as well)
     PF_BF16 = 4,            // out_b[t][r] = acc
     PF_BF16_RELU2 = 5,      // out_b[t][r] = max(acc, 0)^2
-    PF_ADD_F32 = 6,         // out_f[t][r] += acc
-    PF_BF16_GELU_SIDE = 7   // out_b[t][r] = gelu_tanh(acc) * side[tokens[t]][r], r < side_dim, else 0
+    PF_ADD_F32 = 6,         // out_f[t][r] += c0 * acc
+    PF_BF16_GELU_SIDE = 7,  // out_b[t][r] = gelu_tanh(acc) * side[tokens[t]][r], r < side_dim, else 0
+    PF_CAP_F32 = 8,         // out_f[t][r] = c0 * tanh(acc / c0)
+    PF_BF16_GLU = 9         // out_b[t][i] = clamped_glu(gate row i, up row i; limit c0, slope c1), rows as eight of each in turn
 };
+constexpr int kPfMaxMat = 6;
 
 struct PfGemmArgs {
     CUtensorMap tx;            // X as [T][K] fp16, box 64 x 128, 128-byte swizzle
-    CUtensorMap tw[3];         // weights: bytes [rows][row bytes], box (raw bytes of a K block) x rows; fp16: box 64 x rows, swizzled
+    CUtensorMap tw[kPfMaxMat];         // weights: bytes [rows][row bytes], box (raw bytes of a K block) x rows; fp16: box 64 x rows, swizzled
     const __half* s[3];        // scales [rows][K / 128] (quantised formats)
     // Plain modes: up to three matrices over the same X side by side in one launch (q, k and v: 16-CTA launches of
     // their own would leave most of the GPU idle); matrix i owns ceil(seg_rows[i] / NT) row tiles and the output
     // columns after those of the matrices before it.  PF_SWIGLU: tw[0] / tw[1] are gate and up, nseg = 1.
-    int seg_rows[3];
+    int seg_rows[kPfMaxMat];
+    int seg_xrow[kPfMaxMat];   // Q_BF16: row of X at which matrix i's input starts (several inputs stacked); 0 = all read the same
     int nseg;
     const __half* bias;        // PF_OUT_F16, may be null
     __half* out_h;
@@ -73,6 +77,7 @@ struct PfGemmArgs {
     CUtensorMap tx2, tw2;      // a second product summed into the same rows (K2 = 0: none)
     int K2;
     const __nv_bfloat16* side; int side_pitch, side_dim; const int* tokens;
+    float c0, c1;              // constants of the epilogue
 };
 
 // Fills the tensor maps and launches.  PF_SWIGLU: w = {gate, up}, nmat = 2, rows[0] = rows of each.  Other modes: nmat
@@ -80,8 +85,8 @@ struct PfGemmArgs {
 int launch_prefill_gemm(int quant, PfGemmArgs& a, const void* x, const void* const* w, const int* rows, int nmat, cudaStream_t stream);
 
 // bfloat16 form: x [T][ldx], matrices of rows[i] stored rows (multiples of 8) of pitch[i] columns, of which the first a.K
-// (any multiple of 8) count; x2 / w2: the second product (its rows = rows[0], columns a.K2).
-struct PfBf16Mat { const void* w; int rows, pitch; };
+// (any multiple of 8) count; x2 / w2: the second product (its rows = rows[0], columns a.K2).  xrow: seg_xrow.
+struct PfBf16Mat { const void* w; int rows, pitch, xrow = 0; };
 int launch_prefill_gemm_bf16(PfGemmArgs& a, const void* x, int ldx, const PfBf16Mat* m, int nmat, const void* x2, int ldx2, const PfBf16Mat* m2, cudaStream_t stream);
 
 }  // namespace cq

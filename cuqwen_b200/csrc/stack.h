@@ -192,7 +192,7 @@ int launch_time_mix_step(const TimeMixStepArgs& a, const LaunchCfg& cfg);
 // delta_rows: convolution, silu, unit vectors; per value head decay and step size.
 struct DeltaArgs {
     const float* raw; int ld, k_off, v_off, g_off, a_off, b_off;    // raw rows [q | k | v | g | a | b]
-    const float* conv; int taps; float* ring;                       // conv [channels][taps], channels = g_off
+    const float* conv; int taps; float* ring;                       // conv [taps][channels], channels = g_off
     const float *a_exp, *dt;                                        // exp(A_log), dt_bias [heads]
     int heads, kv_heads, dim, dimp, vdim, vdimp, T;
     float* qk; float* v; float4* sc;                                // [T][kv_heads][q dimp | k dimp], [T][heads * vdimp], [T][heads] (decay, step, k . q, -)
