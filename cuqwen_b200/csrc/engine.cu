@@ -274,6 +274,7 @@ extern "C" int cuqwen_open(const char* dir, const cuqwen_open_params* pin, cuqwe
     if (o.max_seq_len < 0) return fail(CUQWEN_ERR_ARG, "max_seq_len must be positive (or 0 for the default)");
     StackSpec spec;
     if (int r = read_model_config(dir, &spec)) return r;
+    if (int r = read_model_shapes(dir, &spec)) return r;
     CK(cudaSetDevice(o.device));
     cuqwen_engine* e = new cuqwen_engine();
     e->p.max_seq_len = o.max_seq_len > 0 ? o.max_seq_len : 32768;
@@ -642,6 +643,7 @@ extern "C" int cuqwen_step(cuqwen_engine* e, int token, int pos, const int* hist
         return fail(CUQWEN_ERR_ARG, "token %d / pos %d / history_len %d out of range", token, pos, history_len);
     CK(cudaSetDevice(e->p.device));
     if (int r = ensure_graph(e)) return r;
+    if (e->stack) if (int r = stack_begin(e->stack, pos)) return r;
     const int hist_len = (history && history_len > 0) ? history_len : 0;
     if (e->ctl_dirty) {         // after cuqwen_decode_n / a profile run / an error: the device block is put back into the host-fed state once
         StepCtl c{}; c.pad[1] = e->steps_done; c.io_seq = e->io_seq; c.hio = e->hio_dev;
@@ -676,6 +678,7 @@ extern "C" int cuqwen_step(cuqwen_engine* e, int token, int pos, const int* hist
         tok = e->h_out[0]; err = e->h_out[1];
     }
     if (err) { e->ctl_dirty = true; return fail(CUQWEN_ERR_TIMEOUT, "a bounded device-side wait expired (code %d)", err); }
+    if (e->stack) stack_end(e->stack, pos + 1);
     if (out_token) *out_token = tok;
     return CUQWEN_OK;
 }
@@ -706,6 +709,7 @@ static int check_tokens(const cuqwen_engine* e, const int* tokens, int n_tokens,
 static int stack_portion(cuqwen_engine* e, const int* tokens, int n_tokens, int pos0, const int* want, int n_want, float* logits) {
     const int C = stack_chunk();
     CK(cudaSetDevice(e->p.device));
+    if (int r = stack_begin(e->stack, pos0)) return r;
     t_err = reinterpret_cast<unsigned*>(&e->ctl->pad[0]);
     if (!e->pf_tok) CK(cudaMalloc((void**)&e->pf_tok, (size_t)C * 4));
     CK(cudaMemsetAsync(&e->ctl->pad[0], 0, 4, e->stream));
@@ -726,6 +730,7 @@ static int stack_portion(cuqwen_engine* e, const int* tokens, int n_tokens, int 
     CK(cudaStreamSynchronize(e->stream));
     if (e->h_out[0]) return fail(CUQWEN_ERR_TIMEOUT, "a bounded device-side wait expired (code %d)", e->h_out[0]);
     CK(cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1));
+    stack_end(e->stack, pos0 + n_tokens);
     return CUQWEN_OK;
 }
 
@@ -840,6 +845,7 @@ extern "C" int cuqwen_decode_n(cuqwen_engine* e, int first_token, int start_pos,
         return fail(CUQWEN_ERR_ARG, "decode_n arguments out of range");
     CK(cudaSetDevice(e->p.device));
     if (int r = ensure_graph(e)) return r;
+    if (e->stack) if (int r = stack_begin(e->stack, start_pos)) return r;
     StepCtl c{}; c.token = first_token; c.pos = start_pos; c.auto_advance = 1; c.pad[1] = e->steps_done; c.io_seq = e->io_seq; c.hio = e->hio_dev;
     e->ctl_dirty = true;
     *e->h_ctl = c;
@@ -853,6 +859,7 @@ extern "C" int cuqwen_decode_n(cuqwen_engine* e, int first_token, int start_pos,
     CK(cudaStreamSynchronize(e->stream));
     if (e->h_out[n]) return fail(CUQWEN_ERR_TIMEOUT, "a bounded device-side wait expired (code %d)", e->h_out[n]);
     CK(cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1));
+    if (e->stack) stack_end(e->stack, start_pos + n);
     if (out_tokens) memcpy(out_tokens, e->h_out, (size_t)n * 4);
     return CUQWEN_OK;
 }
@@ -865,6 +872,7 @@ extern "C" int cuqwen_step_profile(cuqwen_engine* e, int token, int pos, float* 
     if (e->tp > 1 && !e->comm) return fail(CUQWEN_ERR_STATE, "cuqwen_step_profile before cuqwen_tp_init");
     if (token < 0 || token >= e->p.vocab_size || pos < 0 || pos >= e->p.max_seq_len) return fail(CUQWEN_ERR_ARG, "token / pos out of range");
     CK(cudaSetDevice(e->p.device));
+    if (e->stack) if (int r = stack_begin(e->stack, pos)) return r;
     StepCtl c{}; c.token = token; c.pos = pos; c.pad[1] = e->steps_done; c.io_seq = e->io_seq; c.hio = e->hio_dev;
     e->ctl_dirty = true;
     *e->h_ctl = c;
@@ -881,6 +889,7 @@ extern "C" int cuqwen_step_profile(cuqwen_engine* e, int token, int pos, float* 
     for (cudaEvent_t ev : evs) cudaEventDestroy(ev);
     if (r) return r;
     CK(ce);
+    if (e->stack) stack_end(e->stack, pos + 1);
     if (n_out) *n_out = n;
     return CUQWEN_OK;
 }
@@ -1317,9 +1326,9 @@ extern "C" int cuqwen_k_linear(int device, int act, int epi, const void* x, int 
     if (act == CUQWEN_ACT_BF16 && n_tokens > 1) {
         PfGemmArgs g; memset(&g, 0, sizeof g);
         const PfBf16Mat m{w, rows, pitch}, m2{w2, rows, pitch2};
-        const int modes[5] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE};
+        const int modes[] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE};
         g.T = n_tokens; g.K = cols; g.K2 = cols2; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = t_err; g.mode = modes[epi];
-        g.side = (const bf16*)side; g.side_pitch = side_pitch; g.side_dim = side_dim; g.tokens = d_tokens;
+        g.side = (const bf16*)side; g.side_pitch = side_pitch; g.side_dim = side_dim; g.tokens = d_tokens; g.c0 = 1.f;
         KK(launch_prefill_gemm_bf16(g, x, ldx, &m, 1, x2, ldx2, x2 ? &m2 : nullptr, dc->stream));
         return CUQWEN_OK;
     }
@@ -1327,7 +1336,7 @@ extern "C" int cuqwen_k_linear(int device, int act, int epi, const void* x, int 
         SegGemvArgs g; memset(&g, 0, sizeof g);
         g.stage = SEG_PLAIN; g.xb[0] = (const bf16*)x; g.klen[0] = cols; g.kp[0] = pitch; g.err = t_err; g.nvar = 1; g.epi[0] = epi; g.out[0] = out;
         if (x2) { g.xb[1] = (const bf16*)x2; g.klen[1] = cols2; g.kp[1] = pitch2; }
-        g.K = g.kp[0] + g.kp[1];
+        g.K = g.kp[0] + g.kp[1]; g.c0 = 1.f;
         g.side = (const bf16*)side; g.side_pitch = side_pitch; g.side_dim = side_dim; g.tokens = d_tokens;
         const SegMat m[2] = {{(const bf16*)w, rows, pitch}, {(const bf16*)w2, rows, pitch2}};
         KK(launch_gemv_seg(g, m, x2 ? 2 : 1, cfg));
@@ -1335,7 +1344,7 @@ extern "C" int cuqwen_k_linear(int device, int act, int epi, const void* x, int 
     }
     LinArgs a{};
     a.x = x; a.ldx = ldx; a.w = (const bf16*)w; a.pitch = pitch; a.K = cols; a.x2 = x2; a.ldx2 = ldx2; a.w2 = x2 ? (const bf16*)w2 : nullptr; a.pitch2 = pitch2; a.K2 = cols2;
-    a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.side = (const bf16*)side; a.side_pitch = side_pitch; a.side_dim = side_dim; a.tokens = d_tokens;
+    a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.side = (const bf16*)side; a.side_pitch = side_pitch; a.side_dim = side_dim; a.tokens = d_tokens; a.c0 = 1.f;
     KK(launch_st_linear(act, a, cfg));
     return CUQWEN_OK;
 }
@@ -1386,7 +1395,7 @@ extern "C" int cuqwen_k_latent_attention(int device, int act, int impl, const vo
     const int es = act == CUQWEN_ACT_F32 ? 4 : 2;
     t.qn = q; t.qn_hs = dim + rot_dim; t.ldqn = heads * t.qn_hs; t.dn = dim; t.qr = (const uint8_t*)q + (size_t)dim * es; t.ldqr = t.ldqn; t.qr_hs = t.qn_hs; t.dr = rot_dim;
     t.kn = kn; t.ldkn = heads * dim; t.kn_hs = dim; t.kr = kr; t.ldkr = rot_dim; t.v = v; t.ldv = heads * vdim; t.v_hs = vdim; t.dv = vdim; t.sink = sink; t.gate = gate; t.ldg = heads * vdim; t.g_hs = vdim;
-    t.out = out; t.ldo = heads * vdim; t.o_hs = vdim; t.T = n_tokens; t.heads = heads; t.window = window; t.scale = scale; t.pos0 = pos0;
+    t.out_scale = 1.f; t.out = out; t.ldo = heads * vdim; t.o_hs = vdim; t.T = n_tokens; t.heads = heads; t.window = window; t.scale = scale; t.pos0 = pos0;
     if (impl == 0) KK(launch_latent_prefill_attn(t, n_keys, (size_t)n_keys, t_err, cfg));
     else KK(launch_latent_attn(act, t, cfg));
     return CUQWEN_OK;

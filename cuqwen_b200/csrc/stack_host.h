@@ -20,6 +20,10 @@ void stack_residual(const Stack* s, void** ptr, size_t* bytes);
 // Algorithmic bytes of one decode step at context length ctx.
 uint64_t stack_step_bytes(const Stack* s, int ctx);
 
+// Around everything that runs tokens at positions pos0 .. pos - 1.  States of a recurrence cannot go back: a run begins at position 0 or
+// where the last one ended; after a failed run only position 0 is left.
+int stack_begin(Stack* s, int pos0);
+void stack_end(Stack* s, int pos);
 // The launches of one decode step from the embedding to the logits, for the token / position in e->ctl.  `after` is called
 // after every launch (launch counting, profiling events).
 int stack_record_step(cuqwen_engine* e, const LaunchCfg& cfg, const std::function<int()>& after);
