@@ -116,7 +116,7 @@ struct Pass {
     // bfloat16, the CUDA-core kernels in float32.
     int product(int epi, const void* x, int ldx, const StMat* const* m, int nm, void* out, int ldo, int n) { return product(epi, x, ldx, m, nm, out, ldo, n, With{}); }
     int product(int epi, const void* x, int ldx, const StMat* const* m, int nm, void* out, int ldo, int n, const With& o) {
-        if (s->act == ACT_BF16 && n > 1) {
+        if (s->act == ACT_BF16 && (n > 1 || epi == LIN_GLU)) {
             static const int modes[] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE, PF_CAP_F32, PF_BF16_GLU};
             PfGemmArgs g; memset(&g, 0, sizeof g);
             PfBf16Mat pm[kPfMaxMat], pm2{};
@@ -166,10 +166,10 @@ struct Pass {
     // sequential layers (stack_mixers.cu)
     int seq_layers(bool cache_only);
     int seq_fused_layers();
-    int first_products(const StLayer& l, bool stop);
     int parallel_mixer(const StLayer& l, bool stop);
     int delta_mixer(const StLayer& l, bool stop);
-    int glu(const StLayer& l);
+    int clamped_glu(const StLayer& l);
+    int grouped_attention(const StLayer& l);
     TimeMixArgs time_mix(const StLayer& l);
     DeltaArgs delta(const StLayer& l);
     QkvRowsArgs qkv(const StLayer& l);
