@@ -628,33 +628,65 @@ def run_prefill_sweep(a, rng):
           "how": "qwen_forward once per prompt token (src/main.cu:86-92): 32 calls at each of four positions, mean x prompt length"})
 
 
-# Layers of the sizes that the table's models have, for designs read from a model directory (--sweep stack): Falivik layers
-# with about as many weights as a layer of the table model named beside them.
+# Layers of the sizes that the table's models have, for designs read from a model directory (--sweep stack): layers with about as
+# many weights as a layer of the table model named beside them.  "gipotar": parallel and delta layers in turn.
 STACK_SIZES = {
     "1.5b": dict(width=1536, heads=12, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, window=1024, ff=13440, side=128,
+                 gipotar=dict(parallel=(12, 2, 128, 128, 64, 24, 64, 6400), delta=(12, 6, 128, 128, 4, 8064), rank=64),
                  table=dict(vocab=32000, dim=1536, inter=8960, heads=12, kv=2, hd=128, tied=False)),
     "7b": dict(width=3584, heads=28, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=4096, ff=25600, side=256,
+               gipotar=dict(parallel=(28, 4, 128, 128, 64, 56, 64, 12928), delta=(28, 14, 128, 128, 4, 16896), rank=64),
                table=dict(vocab=32000, dim=3584, inter=18944, heads=28, kv=4, hd=128, tied=False)),
 }
 
 
-def stack_model(size: str, layers: int) -> Path:
-    """Random-weight model directory of the given layers (every second pair of layers shares its latents), made once."""
+def stack_config(design: str, size: str, layers: int) -> dict:
     from cuqwen_b200 import stackfmt as F
     z = STACK_SIZES[size]
-    base = Path("/dev/shm") if os.access("/dev/shm", os.W_OK) else Path("/tmp")
-    d = base / f"cuqwen_bench_falivik_{size}_L{layers}_seed{SEED}"
-    if not (d / "done").exists():
+    if design == "falivik":                     # every second pair of layers shares its latents
         ls = [F.latent_layer(z["heads"], z["dim"], z["rot_dim"], z["vdim"], z["q_rank"], z["kv_rank"], z["window"], z["ff"], kv_from=i - 1 if i % 4 == 3 else None) for i in range(layers)]
-        cfg = F.falivik_config(z["table"]["vocab"], z["width"], z["side"], ls)
-        F.write_model_dir(d, cfg, F.random_weights(cfg, SEED, block=1 << 20))
+        return F.falivik_config(z["table"]["vocab"], z["width"], z["side"], ls)
+    g = z["gipotar"]
+    return F.gipotar_config(z["table"]["vocab"], z["width"], [F.delta_layer(*g["delta"]) if i % 2 == 0 else F.parallel_layer(*g["parallel"]) for i in range(layers)], residual_mult=0.4)
+
+
+def stack_model(design: str, size: str, layers: int) -> Path:
+    """Random-weight model directory of the given layers, made once."""
+    from cuqwen_b200 import stackfmt as F
+    base = Path("/dev/shm") if os.access("/dev/shm", os.W_OK) else Path("/tmp")
+    d = base / f"cuqwen_bench_{design}_{size}_L{layers}_seed{SEED}"
+    if not (d / "done").exists():
+        cfg = stack_config(design, size, layers)
+        F.write_model_dir(d, cfg, F.random_weights(cfg, SEED, block=1 << 20, rank=STACK_SIZES[size]["gipotar"]["rank"]))
         (d / "done").touch()
     return d
 
 
+def gipotar_flops(cfg, rank: int, n: int) -> tuple[float, float]:
+    """(matrix products, attention and recurrences) of a prefill of n tokens without logits: the last layer stops at what it leaves behind."""
+    W, gemm, rest = cfg["width"], 0.0, 0.0
+    for i, L in enumerate(cfg["layers"]):
+        m, last = L["mixer"], i + 1 == len(cfg["layers"])
+        if L["type"] == "parallel":
+            a, t = m["left"], m["right"]
+            R = t["heads"] * t["dim"]
+            gemm += W * ((a["heads"] + a["kv_heads"]) * a["dim"] + a["kv_heads"] * a["vdim"] + 4 * R + rank) + rank * R
+            rest += 6.0 * n * R * t["dim"]
+            if not last:
+                gemm += W * (a["heads"] * a["vdim"] + R)
+                rest += float(n) * (n + 1) * a["heads"] * (a["dim"] + a["vdim"])
+        else:
+            H, G, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            gemm += W * (2 * G * d + 2 * H * v + 2 * H) + (0 if last else W * H * v)
+            rest += 8.0 * n * H * d * v
+        if L["mlp"] and not last:
+            gemm += 3 * W * L["mlp"]["ff"]
+    return 2.0 * n * gemm, rest
+
+
 def run_stack_sweep(a):
-    """--sweep stack: decode and prefill of a Falivik model in bfloat16 (random weights) beside the table's model of about
-    equal layers in fp16, both cut to the same number of layers (default 8) and the same vocabulary.  --stack picks the
+    """--sweep stack: decode and prefill of a directory's design (--design) in bfloat16 (random weights) beside the table's model of
+    about equal layers in fp16, both cut to the same number of layers (default 8) and the same vocabulary.  --stack picks the
     size, --only one of the two arms (profiler runs)."""
     from cuqwen_b200 import binfmt, build
     from cuqwen_b200 import engine as E
@@ -663,7 +695,8 @@ def run_stack_sweep(a):
     tp = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
     tf = float(tp.get("bf16_tflops", 1590.0))
     toks = np.random.default_rng(SEED).integers(0, z["table"]["vocab"], size=max(n, ctx)).astype(np.int32)
-    W, H, t = z["width"], z["heads"], z["table"]
+    W, H, t, wu = z["width"], z["heads"], z["table"], max(a.warmup, 3)
+    room = max(n, ctx + wu + Kst + 64)
 
     def measure(name, eng, fill, gemm_flop, attn_flop, step_bytes):
         fill()
@@ -674,8 +707,8 @@ def run_stack_sweep(a):
                 eng.prefill(toks[:n], 0)
                 pms.append(eng.last_decode_ms)
             fill()
-            eng.decode_n(1234, ctx, max(a.warmup, 3))
-            eng.decode_n(1234, ctx, Kst)
+            eng.decode_n(1234, ctx, wu)
+            eng.decode_n(1234, ctx + wu, Kst)
         ms, p = eng.last_decode_ms / Kst, min(pms)
         emit({"sweep": "stack", "model": name, "layers": nl, "decode": {"ctx": ctx, "tok_s": round(1e3 / ms, 1), "ms_per_step": round(ms, 4), "launches": eng.step_launches, "algorithmic_bytes": step_bytes,
               "gbs": round(step_bytes / ms / 1e6, 1), "frac_of_measured_hbm": round(step_bytes / ms / 1e6 / hbm, 4)},
@@ -684,26 +717,29 @@ def run_stack_sweep(a):
               "l2": "no flush: a step streams more weights than L2 holds", "clocks": cs.result})
         eng.close()
 
-    if a.only in ("", "stack"):
-        d = stack_model(a.stack, nl)
-        eng = E.Engine.open(d, max_seq_len=max(n, ctx + Kst + 64))
+    if a.only in ("", "stack") and a.design == "gipotar":
+        eng = E.Engine.open(stack_model("gipotar", a.stack, nl), max_seq_len=room)
+        gemm, rest = gipotar_flops(stack_config("gipotar", a.stack, nl), z["gipotar"]["rank"], n)
+        measure(f"Gipotar {a.stack} layers, bfloat16", eng, lambda: eng.prefill(toks[:ctx], 0), gemm, rest, eng.step_bytes(ctx + wu + Kst // 2))
+    elif a.only in ("", "stack"):
+        eng = E.Engine.open(stack_model("falivik", a.stack, nl), max_seq_len=room)
         keys = sum(min(i + 1, z["window"]) for i in range(n))
         own = sum(1 for i in range(nl) if i % 4 != 3)
         # every layer; the last one of a prefill without logits stops after its cache row (or before, when it shares one)
         per = W * (z["q_rank"] + 2 * H * z["vdim"] + 2 * z["ff"] + 2 * z["side"]) + z["q_rank"] * H * (z["dim"] + z["rot_dim"]) + z["kv_rank"] * H * (z["dim"] + z["vdim"])
         measure(f"Falivik {a.stack} layers, bfloat16", eng, lambda: eng.prefill(toks[:ctx], 0), 2.0 * n * ((nl - 1) * per + own * W * (z["kv_rank"] + z["rot_dim"])),
-                2.0 * keys * H * (z["dim"] + z["rot_dim"] + z["vdim"]) * (nl - 1), eng.step_bytes(ctx + Kst // 2))
+                2.0 * keys * H * (z["dim"] + z["rot_dim"] + z["vdim"]) * (nl - 1), eng.step_bytes(ctx + wu + Kst // 2))
     if a.only in ("", "table"):
         cfg = dict(t, layers=nl)
         p = model_path(f"stack_{a.stack}", "fp16", nl)
         if not p.exists():
             build.build_gen()
             subprocess.run([str(build.GEN_BIN), "--out", str(p), "--dims", *[str(cfg[k]) for k in ("vocab", "dim", "inter", "layers", "heads", "kv", "hd")], "--quant", "fp16", "--seed", str(SEED), "--untied"], check=True)
-        eng = E.Engine(E.custom_params(cfg["vocab"], cfg["dim"], cfg["inter"], nl, cfg["heads"], cfg["kv"], cfg["hd"], "fp16", max_seq_len=max(n, ctx + Kst + 64)))
+        eng = E.Engine(E.custom_params(cfg["vocab"], cfg["dim"], cfg["inter"], nl, cfg["heads"], cfg["kv"], cfg["hd"], "fp16", max_seq_len=room))
         eng.load(str(p))
         qd, kd = cfg["heads"] * cfg["hd"], cfg["kv"] * cfg["hd"]
         gemm = 2.0 * n * (nl * cfg["dim"] * (qd + 2 * kd) + (nl - 1) * (qd * cfg["dim"] + 3 * cfg["dim"] * cfg["inter"]))
-        measure(f"Qwen2.5 {a.stack} layers, fp16", eng, lambda: eng.kv_fill_normal(ctx, SEED), gemm, 4.0 * qd * (n * (n + 1) / 2) * (nl - 1), eng.step_bytes(ctx + Kst // 2))
+        measure(f"Qwen2.5 {a.stack} layers, fp16", eng, lambda: eng.kv_fill_normal(ctx, SEED), gemm, 4.0 * qd * (n * (n + 1) / 2) * (nl - 1), eng.step_bytes(ctx + wu + Kst // 2))
 
 
 def main():
@@ -724,6 +760,7 @@ def main():
     ap.add_argument("--sweep", default="", choices=["", "gemv", "attention", "prefill", "stack"],
                     help="kernel-level sweeps of the other benchmark configurations; stack: a model directory's design beside the table's closest model")
     ap.add_argument("--stack", default="7b", choices=sorted(STACK_SIZES), help="--sweep stack: layer size")
+    ap.add_argument("--design", default="falivik", choices=["falivik", "gipotar"], help="--sweep stack: the model directory's design")
     ap.add_argument("--only", default="", choices=["", "stack", "table"], help="--sweep stack: one arm only")
     ap.add_argument("--repeat", type=int, default=3, help="--sweep stack: timed prefills (the best counts)")
     a = ap.parse_args()
