@@ -8,6 +8,7 @@
 #include "../../include/cuqwen_tokenizer.h"
 
 #include <algorithm>
+#include <cstdlib>
 #include <cstdint>
 #include <cstdio>
 #include <cstring>
@@ -262,7 +263,7 @@ struct JsonReader {
         if (p < end && (*p == '-' || *p == '+')) ++p;
         while (p < end && ((*p >= '0' && *p <= '9') || *p == '.' || *p == 'e' || *p == 'E' || *p == '-' || *p == '+')) ++p;
         if (p == s) bad("number expected");
-        return std::stod(std::string(s, p));
+        return std::strtod(std::string(s, p).c_str(), nullptr);      // not stod, which throws on subnormal values
     }
     void skip_value() {
         const char c = peek();
