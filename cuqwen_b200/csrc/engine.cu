@@ -1400,3 +1400,123 @@ extern "C" int cuqwen_k_latent_attention(int device, int act, int impl, const vo
     else KK(launch_latent_attn(act, t, cfg));
     return CUQWEN_OK;
 }
+
+extern "C" int cuqwen_k_linear_epi(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, int n_tokens, int rows, void* out, int ldo, float c0, float c1) {
+    DEV(device);
+    NOT_NULL(x, w, out);
+    if (bad_act(act) || (epi != LIN_ADD && epi != LIN_CAP && epi != LIN_GLU) || n_tokens < 1 || rows < 8 || rows % 8 || (epi == LIN_GLU && (rows % 16 || act == CUQWEN_ACT_F32)) || cols < 8 || cols % 8 || pitch % 128 ||
+        pitch < cols || ldx % 8 || ldx < cols || ldo % 8 || ldo < (epi == LIN_GLU ? rows / 2 : rows) || (epi == LIN_CAP && !(c0 > 0.f)))
+        return fail(CUQWEN_ERR_ARG, "linear_epi: rows, cols and row strides are multiples of 8, the weight pitch of 128; the gated unit has rows in sixteens and bfloat16");
+    if (act == CUQWEN_ACT_BF16 && n_tokens > 1) {
+        PfGemmArgs g; memset(&g, 0, sizeof g);
+        const PfBf16Mat m{w, rows, pitch};
+        g.T = n_tokens; g.K = cols; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = t_err; g.mode = epi == LIN_ADD ? PF_ADD_F32 : epi == LIN_CAP ? PF_CAP_F32 : PF_BF16_GLU; g.c0 = c0; g.c1 = c1;
+        KK(launch_prefill_gemm_bf16(g, x, ldx, &m, 1, nullptr, 0, nullptr, dc->stream));
+        return CUQWEN_OK;
+    }
+    if (act == CUQWEN_ACT_BF16) {
+        SegGemvArgs g; memset(&g, 0, sizeof g);
+        g.stage = SEG_PLAIN; g.xb[0] = (const bf16*)x; g.klen[0] = cols; g.kp[0] = pitch; g.K = pitch; g.err = t_err; g.nvar = 1; g.epi[0] = epi; g.out[0] = out; g.c0 = c0; g.c1 = c1;
+        const SegMat m[1] = {{(const bf16*)w, rows, pitch}};
+        KK(launch_gemv_seg(g, m, 1, cfg));
+        return CUQWEN_OK;
+    }
+    LinArgs a{};
+    a.x = x; a.ldx = ldx; a.w = (const bf16*)w; a.pitch = pitch; a.K = cols; a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.c0 = c0; a.c1 = c1;
+    KK(launch_st_linear(act, a, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_shift_mix(int device, int act, const float* x, int ldx, const float* w, int width, float eps, const float* mu, int n_mix, float* ring, float* tail, void* out, int pos0, int n_rows) {
+    DEV(device);
+    NOT_NULL(x, w, ring, tail, out);
+    if (n_mix > 0) NOT_NULL(mu);
+    if (bad_act(act) || width < 1 || ldx % 8 || ldx < width || n_mix < 0 || n_rows < 1 || pos0 < 0) return fail(CUQWEN_ERR_ARG, "shift_mix: the row stride is a multiple of 8");
+    ShiftRowsArgs a{};
+    a.x = x; a.ldx = ldx; a.w = w; a.width = width; a.eps = eps; a.out = out; a.ldo = ldx; a.var_stride = (size_t)n_rows * ldx; a.mu = mu; a.ldmu = ldx; a.n_mix = n_mix; a.prev = ring; a.ldprev = ldx; a.tail = tail; a.pos0 = pos0;
+    KK(launch_shift_rows(act, a, n_rows, cfg));
+    const TailRowsArgs t{tail, 0, 1, ring, ldx, ldx, 2, 1, nullptr, pos0 + n_rows - 1};
+    KK(launch_tail_rows(t, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_grouped_attention(int device, int act, int impl, const float* raw, void* q, void* cache, int max_seq, const void* rot, int rot_dims, void* out, float* scratch, int n_tokens, int pos0,
+                                          const int* d_pos, int heads, int kv_heads, int dim, int vdim, float scale, float out_scale) {
+    DEV(device);
+    NOT_NULL(raw, q, cache, out);
+    if (bad_act(act) || impl < 0 || impl > 2 || (impl != 1 && act != CUQWEN_ACT_BF16) || n_tokens < 1 || pos0 < 0 || pos0 + n_tokens > max_seq || heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 8 || dim % 8 ||
+        vdim < 8 || vdim % 8 || rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (impl == 0 && !latent_prefill_fits(dim, 0, vdim)) || (impl == 2 && n_tokens != 1))
+        return fail(CUQWEN_ERR_ARG, "grouped_attention: lengths are multiples of 8; impl 0 (tensor cores) and 2 (split, one token) are bfloat16 only");
+    if (rot_dims) NOT_NULL(rot);
+    if (impl == 2) NOT_NULL(scratch, d_pos);
+    const int es = act == CUQWEN_ACT_F32 ? 4 : 2, crow = dim + vdim;
+    QkvRowsArgs a{};
+    a.raw = raw; a.k_off = heads * dim; a.v_off = a.k_off + kv_heads * dim; a.ld = a.v_off + kv_heads * vdim; a.heads = heads; a.kv_heads = kv_heads; a.dim = a.dimp = dim; a.vdimp = vdim; a.q = q; a.ldq = heads * dim;
+    a.cache = cache; a.max_seq = max_seq; a.rot = (const float2*)rot; a.rot_dims = rot_dims; a.pos0 = pos0;
+    KK(launch_qkv_rows(act, a, n_tokens, cfg));
+    if (impl == 2) {
+        LatentDecodeArgs d{};
+        d.q = (const bf16*)q; d.crow = crow; d.cache = (const bf16*)cache; d.kvrp = vdim; d.heads = heads; d.scale = scale; d.pos_ptr = d_pos; d.nsplit = grouped_decode_splits(heads, kv_heads, dim, vdim, max_seq, cfg.sm_count);
+        if (d.nsplit < 1) return fail(CUQWEN_ERR_ARG, "grouped_attention: the split form does not cover these lengths");
+        d.part_ml = scratch; d.part_o = scratch + (size_t)(2 * d.nsplit * heads + 3) / 4 * 4; d.out = (bf16*)out; d.o_hs = vdim; d.group = heads / kv_heads; d.kdim = dim; d.kv_stride = (size_t)max_seq * crow; d.out_scale = out_scale;
+        return launch_grouped_decode(d, cfg, [](int err, const char* what) { return err ? fail(CUQWEN_ERR_CUDA, "%s: %s", what, cudaGetErrorString((cudaError_t)err)) : (int)CUQWEN_OK; });
+    }
+    LatentAttnArgs t{};
+    t.qn = q; t.ldqn = heads * dim; t.qn_hs = dim; t.dn = dim; t.qr = q; t.kn = cache; t.ldkn = crow; t.kn_hs = max_seq * crow; t.kr = cache; t.v = (const uint8_t*)cache + (size_t)dim * es; t.ldv = crow; t.v_hs = t.kn_hs; t.dv = vdim;
+    t.out = out; t.ldo = heads * vdim; t.o_hs = vdim; t.T = n_tokens; t.heads = heads; t.scale = scale; t.pos0 = pos0; t.kv_group = heads / kv_heads; t.out_scale = out_scale;
+    if (impl == 0) KK(launch_latent_prefill_attn(t, pos0 + n_tokens, (size_t)max_seq, t_err, cfg));
+    else KK(launch_latent_attn(act, t, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, float* z, const float* w0, const float* u, float* bonus, float* state, float* o, int heads, int dim, int n_tokens, int pos0) {
+    DEV(device);
+    NOT_NULL(r, k, v, z, w0, u, bonus, state, o);
+    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || n_tokens < 1 || pos0 < 0) return fail(CUQWEN_ERR_ARG, "time_mix: dim is a multiple of 8, at most %d", kRecurMaxDim);
+    TimeMixArgs a{};
+    a.r = r; a.k = k; a.v = v; a.ld = a.ldz = a.ldo = heads * dim; a.z = z; a.w0 = w0; a.u = u; a.bonus = bonus; a.heads = heads; a.dim = a.dimp = dim; a.T = n_tokens; a.state = state; a.o = o; a.pos0 = pos0;
+    KK(launch_time_mix_rows(a, cfg));
+    KK(launch_time_mix_scan(a, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_time_mix_step(int device, const float* raw, const void* w2, int w2_pitch, int rank, const float* w0, const float* u, const float* norm, float* state, void* out, int heads, int dim, float eps,
+                                      float scale, const int* d_pos) {
+    DEV(device);
+    NOT_NULL(raw, w2, w0, u, norm, state, out, d_pos);
+    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || rank < 1 || w2_pitch < rank) return fail(CUQWEN_ERR_ARG, "time_mix_step: dim is a multiple of 8, at most %d", kRecurMaxDim);
+    const int n = heads * dim;
+    TimeMixStepArgs a{};
+    a.r = raw; a.k = raw + n; a.v = raw + 2 * n; a.g = raw + 3 * n; a.w1 = raw + 4 * n; a.w2 = (const bf16*)w2; a.w2_pitch = w2_pitch; a.rank = rank; a.w0 = w0; a.u = u; a.norm = norm; a.heads = heads; a.dim = a.dimp = dim;
+    a.state = state; a.eps = eps; a.scale = scale; a.out = (bf16*)out; a.pos_ptr = d_pos;
+    KK(launch_time_mix_step(a, cfg));
+    return CUQWEN_OK;
+}
+static DeltaArgs delta_args(const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, float* state, int heads, int kv_heads, int dim, int vdim) {
+    DeltaArgs a{};
+    a.raw = raw; a.k_off = kv_heads * dim; a.v_off = 2 * a.k_off; a.g_off = a.v_off + heads * vdim; a.a_off = a.g_off + heads * vdim; a.b_off = a.a_off + (heads + 7) / 8 * 8; a.ld = a.b_off + (heads + 7) / 8 * 8;
+    a.conv = conv; a.taps = taps; a.ring = ring; a.a_exp = a_exp; a.dt = dt; a.heads = heads; a.kv_heads = kv_heads; a.dim = a.dimp = dim; a.vdim = a.vdimp = vdim; a.state = state; a.ldo = heads * vdim;
+    return a;
+}
+static bool delta_ok(int heads, int kv_heads, int dim, int vdim, int taps) {
+    return heads >= 1 && kv_heads >= 1 && heads % kv_heads == 0 && dim >= 8 && dim % 8 == 0 && dim <= kRecurMaxDim && vdim >= 8 && vdim % 8 == 0 && taps >= 1;
+}
+extern "C" int cuqwen_k_delta(int device, const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, float* qk, float* v, float* sc, float* state, float* o, int heads, int kv_heads, int dim,
+                              int vdim, int n_tokens, int pos0) {
+    DEV(device);
+    NOT_NULL(raw, conv, ring, a_exp, dt, qk, v, sc, state, o);
+    if (!delta_ok(heads, kv_heads, dim, vdim, taps) || n_tokens < 1 || pos0 < 0) return fail(CUQWEN_ERR_ARG, "delta: lengths are multiples of 8, dim at most %d", kRecurMaxDim);
+    DeltaArgs a = delta_args(raw, conv, taps, ring, a_exp, dt, state, heads, kv_heads, dim, vdim);
+    a.qk = qk; a.v = v; a.sc = (float4*)sc; a.o = o; a.T = n_tokens; a.pos0 = pos0;
+    KK(launch_delta_rows(a, cfg));
+    const TailRowsArgs t{raw, a.ld, n_tokens, ring, a.g_off, a.g_off, taps, taps - 1, nullptr, pos0};
+    if (taps > 1) KK(launch_tail_rows(t, cfg));
+    KK(launch_delta_scan(a, cfg));
+    return CUQWEN_OK;
+}
+extern "C" int cuqwen_k_delta_step(int device, const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, const float* norm, float* state, void* out, int heads, int kv_heads, int dim,
+                                   int vdim, float eps, const int* d_pos) {
+    DEV(device);
+    NOT_NULL(raw, conv, ring, a_exp, dt, norm, state, out, d_pos);
+    if (!delta_ok(heads, kv_heads, dim, vdim, taps)) return fail(CUQWEN_ERR_ARG, "delta_step: lengths are multiples of 8, dim at most %d", kRecurMaxDim);
+    DeltaStepArgs a{delta_args(raw, conv, taps, ring, a_exp, dt, state, heads, kv_heads, dim, vdim), norm, eps, 1.f, (bf16*)out};
+    a.d.T = 1; a.d.pos_ptr = d_pos;
+    KK(launch_delta_step(a, cfg));
+    return CUQWEN_OK;
+}

@@ -134,7 +134,7 @@ def capture_replay(replays: int, device=0) -> float:
 
 
 # ---- kernels of the layer-list designs (act: 0 bfloat16, 1 float32 activations) ----
-LIN_F32, LIN_ACT, LIN_RELU2, LIN_ADD, LIN_GELU_SIDE = range(5)
+LIN_F32, LIN_ACT, LIN_RELU2, LIN_ADD, LIN_GELU_SIDE, LIN_CAP, LIN_GLU = range(7)
 
 
 def linear(act, epi, x, ldx, w, pitch, cols, n_tokens, rows, out, ldo, second=None, side=None, device=0):
@@ -160,3 +160,15 @@ def rot_table(table, n_pos, dims, base, device=0):
 
 def latent_attention(act, impl, q, kn, kr, v, sink, gate, out, n_tokens, pos0, n_keys, heads, dim, rot_dim, vdim, window, scale, device=0):
     check(_abi.lib().cuqwen_k_latent_attention(device, act, impl, _p(q), _p(kn), _p(kr), _p(v), _p(sink), _p(gate), _p(out), n_tokens, pos0, n_keys, heads, dim, rot_dim, vdim, window, scale))
+
+
+# ---- kernels of the recurrent designs' layers: arguments as in include/cuqwen_b200.h, without the device ----
+def _forward(name):
+    def call(*args, device=0):
+        check(getattr(_abi.lib(), name)(device, *[_p(a) if a is None or hasattr(a, "ptr") else a for a in args]))
+    call.__name__, call.__doc__ = name.removeprefix("cuqwen_k_"), name
+    return call
+
+
+linear_epi, shift_mix, grouped_attention, time_mix, time_mix_step, delta, delta_step = map(_forward, (
+    "cuqwen_k_linear_epi", "cuqwen_k_shift_mix", "cuqwen_k_grouped_attention", "cuqwen_k_time_mix", "cuqwen_k_time_mix_step", "cuqwen_k_delta", "cuqwen_k_delta_step"))

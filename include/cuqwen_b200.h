@@ -307,6 +307,29 @@ int cuqwen_k_rot_table(int device, void* table, int n_pos, int dims, double base
 int cuqwen_k_latent_attention(int device, int act, int impl, const void* q, const void* kn, const void* kr, const void* v, const float* sink, const float* gate, void* out, int n_tokens,
                               int pos0, int n_keys, int heads, int dim, int rot_dim, int vdim, int window, float scale);
 
+/* Kernels of the recurrent designs' layers (no counterpart in the reference). */
+/* Matrix product with an epilogue of constants.  epi 3: out (float) += c0 * acc; 5: out (float) = c0 * tanh(acc / c0); 6 (bfloat16 only): rows are eight of a
+ * gate and eight of an up matrix in turn, g = min(gate, c0), u = clamp(up, -c0, c0), out[t][i] = g * sigmoid(c1 * g) * (u + 1). */
+int cuqwen_k_linear_epi(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, int n_tokens, int rows, void* out, int ldo, float c0, float c1);
+/* h = x / rms(x) * w per row; out [n_mix + 1][n_rows][ldx]: copy 0 = h, copy i = h + (h of the row before - h) * mu[i - 1].  ring: two rows by position parity, the
+ * h of the position before pos0 going in, the last row's coming out; tail: one row of scratch. */
+int cuqwen_k_shift_mix(int device, int act, const float* x, int ldx, const float* w, int width, float eps, const float* mu, int n_mix, float* ring, float* tail, void* out, int pos0, int n_rows);
+/* Raw rows [q heads x dim | k kv_heads x dim | v kv_heads x vdim] at positions pos0 ..: rotates q and k (their first rot_dims entries), puts [key | value] rows into
+ * cache [kv_heads][max_seq][dim + vdim], attends causally; out [t][heads][vdim] times out_scale.  impl 0: tcgen05, 1: CUDA cores, 2: one token, split over the
+ * keys (*d_pos = pos0; scratch: 148 * heads * (vdim + 4) floats). */
+int cuqwen_k_grouped_attention(int device, int act, int impl, const float* raw, void* q, void* cache, int max_seq, const void* rot, int rot_dims, void* out, float* scratch, int n_tokens, int pos0, const int* d_pos, int heads, int kv_heads, int dim, int vdim, float scale, float out_scale);
+/* Time mixing of a portion in float32: r, k, v, z [t][heads][dim]; z (the low-rank product) becomes the decay exp(-exp(z + w0)); o = S^T r + (sum r u k) v, then
+ * S = diag(decay) S + k v^T; state [heads][value][key] goes on from pos0 (zero at 0); bonus: heads * n_tokens floats of scratch. */
+int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, float* z, const float* w0, const float* u, float* bonus, float* state, float* o, int heads, int dim, int n_tokens, int pos0);
+/* One token: raw [r | k | v | g, heads x dim each | w1 product, rank]; decay through w2 [heads * dim][w2_pitch]; out = o / rms(o) * norm * silu(g) * scale (bfloat16). */
+int cuqwen_k_time_mix_step(int device, const float* raw, const void* w2, int w2_pitch, int rank, const float* w0, const float* u, const float* norm, float* state, void* out, int heads, int dim, float eps, float scale, const int* d_pos);
+/* Gated delta rule of a portion in float32: raw rows [q, k: kv_heads x dim | v, g: heads x vdim | a, b: heads rounded up to eight]; conv [taps][q | k | v channels], last tap
+ * = current token; ring [taps][channels] raw rows by position; a_exp = exp(A_log); qk [t][kv_heads][2 dim], v [t][heads * vdim], sc [t][heads][4] scratch; state
+ * [heads][value][key]; o [t][heads][vdim] before norm and gate. */
+int cuqwen_k_delta(int device, const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, float* qk, float* v, float* sc, float* state, float* o, int heads, int kv_heads, int dim, int vdim, int n_tokens, int pos0);
+/* One token of the same, with o / rms(o) * norm * silu(g) (bfloat16). */
+int cuqwen_k_delta_step(int device, const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, const float* norm, float* state, void* out, int heads, int kv_heads, int dim, int vdim, float eps, const int* d_pos);
+
 const char* cuqwen_strerror(int code);
 const char* cuqwen_last_error(void);
 
