@@ -1466,12 +1466,15 @@ extern "C" int cuqwen_k_grouped_attention(int device, int act, int impl, const f
     else KK(launch_latent_attn(act, t, cfg));
     return CUQWEN_OK;
 }
-extern "C" int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, float* z, const float* w0, const float* u, float* bonus, float* state, float* o, int heads, int dim, int n_tokens, int pos0) {
+extern "C" int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, float* z, const float* w0, const float* u, float* bonus, float* state, float* o, int heads, int dim, int n_tokens, int pos0,
+                                 int segment, float* seg_state, float* seg_decay) {
     DEV(device);
     NOT_NULL(r, k, v, z, w0, u, bonus, state, o);
-    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || n_tokens < 1 || pos0 < 0) return fail(CUQWEN_ERR_ARG, "time_mix: dim is a multiple of 8, at most %d", kRecurMaxDim);
+    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || n_tokens < 1 || pos0 < 0 || segment < 0 || (segment > 0 && (n_tokens + segment - 1) / segment > kTmMaxSeg)) return fail(CUQWEN_ERR_ARG, "time_mix: dim is a multiple of 8, at most %d", kRecurMaxDim);
     TimeMixArgs a{};
     a.r = r; a.k = k; a.v = v; a.ld = a.ldz = a.ldo = heads * dim; a.z = z; a.w0 = w0; a.u = u; a.bonus = bonus; a.heads = heads; a.dim = a.dimp = dim; a.T = n_tokens; a.state = state; a.o = o; a.pos0 = pos0;
+    a.seg_len = segment > 0 && segment < n_tokens ? segment : n_tokens; a.seg_state = seg_state; a.seg_decay = seg_decay;
+    if (a.seg_len < n_tokens) NOT_NULL(seg_state, seg_decay);
     KK(launch_time_mix_rows(a, cfg));
     KK(launch_time_mix_scan(a, cfg));
     return CUQWEN_OK;

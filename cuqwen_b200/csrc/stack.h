@@ -175,7 +175,10 @@ struct TimeMixArgs {
     int heads, dim, dimp, T;
     float* state; float* o; int ldo;
     const int* pos_ptr; int pos0;
+    int seg_len; float *seg_state, *seg_decay;                      // tokens of a segment (T: one segment, no scratch); scratch [kTmMaxSeg][state], [kTmMaxSeg][heads][dimp]
 };
+constexpr int kTmMaxSeg = 16;
+int time_mix_segment(int heads, int dimp, int T, int sm_count);    // a good seg_len
 int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg);
 int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg);
 // One token in bfloat16: low-rank decay, recurrence, head norm, gate - and, in the same launch, the token's qkv rows (qkv.raw null: none).

@@ -23,6 +23,7 @@ TimeMixArgs Pass::time_mix(const StLayer& l) {
     a.z = w->z; a.ldz = t.heads * l.rdimp; a.w0 = l.w0; a.u = l.u; a.bonus = (float*)w->sc;
     a.heads = t.heads; a.dim = t.dim; a.dimp = l.rdimp; a.T = T;
     a.state = (float*)at(l.state_off); a.o = w->ro; a.ldo = t.heads * l.rdimp; a.pos_ptr = pos_ptr; a.pos0 = pos0;
+    a.seg_len = T > 1 ? time_mix_segment(t.heads, l.rdimp, T, cfg.sm_count) : 1; a.seg_state = w->seg_state; a.seg_decay = w->seg_decay;
     return a;
 }
 DeltaArgs Pass::delta(const StLayer& l) {

@@ -59,7 +59,7 @@ struct Stack {
     struct Ws {
         int rows = 0, kv_rows = 0;
         float *x = nullptr, *x2 = nullptr, *raw = nullptr, *qf = nullptr, *y = nullptr, *o_lat = nullptr, *part_o = nullptr, *part_ml = nullptr;
-        float *z = nullptr, *qk = nullptr, *vv = nullptr, *ro = nullptr, *tail = nullptr; float4* sc = nullptr;      // recurrences: decays, convolution outputs, read-outs, head scalars
+        float *z = nullptr, *qk = nullptr, *vv = nullptr, *ro = nullptr, *tail = nullptr; float *seg_state = nullptr, *seg_decay = nullptr; float4* sc = nullptr;      // recurrences: segments of a portion, decays, convolution outputs, read-outs, head scalars
         void *zin = nullptr, *att2 = nullptr;
         void *xn1 = nullptr, *xn2 = nullptr, *cq = nullptr, *q = nullptr, *att = nullptr, *h = nullptr, *sg = nullptr, *kv = nullptr;
         uint8_t* arena = nullptr;
@@ -68,7 +68,7 @@ struct Stack {
     float* logits = nullptr;            // decode step
     float* logits_rows = nullptr; void* xn_rows = nullptr; int* want_rows = nullptr;
     int max_raw = 0, max_q = 0, max_att = 0, max_ff = 0, max_qr = 0, max_kv = 0, max_kvr = 0, max_heads = 0, max_split = 1;
-    int max_var = 1, max_z = 0, max_rank = 0, max_qk = 0, max_vv = 0, max_sc = 0, max_ro = 0, max_glu = 0;
+    int max_var = 1, max_z = 0, max_rank = 0, max_qk = 0, max_vv = 0, max_sc = 0, max_ro = 0, max_tm_state = 0;
     int next_pos = 0;                   // designs with a recurrence: the position that the states have reached (-1: none)
 };
 

@@ -3,7 +3,8 @@
 //
 // Portions: the row kernel turns the low-rank products into decays and takes the bonus sums; the scan walks the tokens with the
 // state in registers (recur.cuh), r, k, decays and values brought a tile of tokens at a time by cp.async.  Value channels are
-// independent of one another, so a head is cut into CTAs of a few of them.
+// independent of one another, so a head is cut into CTAs of a few of them; and since a segment of the portion acts on the state it
+// begins with by a factor per key channel and a sum, a long portion is also cut into segments.
 #include "qkv_rows.cuh"
 #include "recur.cuh"
 
@@ -30,86 +31,145 @@ int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg) {
 }
 
 constexpr int kTmTile = 16;                             // tokens brought at a time
-// CTA: head x CB value channels, NC of them to a thread.
-template <int LPC, int NV, int NC, int CB>
+// CTA: head x CB value channels x segment of the portion, NC channels to a thread.  A portion of several segments takes three passes:
+// every segment's state from zero and its decay product (STATE_ONLY), the states the segments begin with (time_mix_join_kernel), and the
+// segments' outputs.
+template <int LPC, int NV, int NC, int CB, bool STATE_ONLY>
 __global__ void __launch_bounds__(CB / NC * LPC) time_mix_scan_kernel(const TimeMixArgs a) {
-    constexpr int D = LPC * NV * 4, NT = CB / NC * LPC, ROW = 3 * D + CB + 4;            // r | k | w | v | bonus
+    constexpr int D = LPC * NV * 4, NT = CB / NC * LPC, ROW = 3 * D + CB + 4;            // k | w | r | v | bonus
     extern __shared__ __align__(16) float tm_smem[];    // [2][kTmTile][ROW]
     pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.x, c0 = blockIdx.y * CB, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC;
+    const int h = blockIdx.x, c0 = blockIdx.y * CB, seg = blockIdx.z, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC;
     const int first = a.pos_ptr ? *a.pos_ptr : a.pos0, nc = min(CB, a.dimp - c0);
-    const size_t ho = (size_t)h * a.dimp;
+    const int t_begin = seg * a.seg_len, t_end = min(t_begin + a.seg_len, a.T);
+    const size_t ho = (size_t)h * a.dimp, states = (size_t)a.heads * a.dimp * a.dimp;
     for (int i = tid; i < 2 * kTmTile * ROW; i += NT) tm_smem[i] = 0.f;                 // what no copy reaches stays zero
     __syncthreads();
+    // a warp brings whole tokens, a lane 16-byte units
     auto bring = [&](int t0, int b) {
-        const int n = min(kTmTile, a.T - t0), du = a.dimp / 4, cu = nc / 4, per = 3 * du + cu;
-        for (int i = tid; i < n * per; i += NT) {
-            const int t = i / per, u = i - t * per, tt = t0 + t;
+        const int n = min(kTmTile, t_end - t0), du = a.dimp / 4, cu = nc / 4;
+        for (int t = tid >> 5; t < n; t += NT / 32) {
+            const size_t tt = (size_t)(t0 + t);
             float* dst = tm_smem + (b * kTmTile + t) * ROW;
-            if (u < du) cp_async16(dst + 4 * u, a.r + (size_t)tt * a.ld + ho + 4 * u);
-            else if (u < 2 * du) cp_async16(dst + D + 4 * (u - du), a.k + (size_t)tt * a.ld + ho + 4 * (u - du));
-            else if (u < 3 * du) cp_async16(dst + 2 * D + 4 * (u - 2 * du), a.z + (size_t)tt * a.ldz + ho + 4 * (u - 2 * du));
-            else cp_async16(dst + 3 * D + 4 * (u - 3 * du), a.v + (size_t)tt * a.ld + ho + c0 + 4 * (u - 3 * du));
+            const float *k = a.k + tt * a.ld + ho, *w = a.z + tt * a.ldz + ho, *r = a.r + tt * a.ld + ho, *v = a.v + tt * a.ld + ho + c0;
+            for (int u = tid & 31; u < du; u += 32) {
+                cp_async16(dst + 4 * u, k + 4 * u); cp_async16(dst + D + 4 * u, w + 4 * u);
+                if (!STATE_ONLY) cp_async16(dst + 2 * D + 4 * u, r + 4 * u);
+            }
+            for (int u = tid & 31; u < cu; u += 32) cp_async16(dst + 3 * D + 4 * u, v + 4 * u);
+            if (!STATE_ONLY && (tid & 31) == 0) dst[3 * D + CB] = a.bonus[tt * a.heads + h];
         }
-        for (int t = tid; t < n; t += NT) tm_smem[(b * kTmTile + t) * ROW + 3 * D + CB] = a.bonus[(size_t)(t0 + t) * a.heads + h];
         cp_async_commit();
     };
-    bring(0, 0);
+    bring(t_begin, 0);
     StateCol<LPC, NV> s[NC];
-    float* st[NC];
+    f32x2 prod[2 * NV];
+#pragma unroll
+    for (int i = 0; i < 2 * NV; ++i) prod[i] = pack2(1.f, 1.f);
+    const bool joined = gridDim.z > 1;                  // every segment begins with its slot of seg_state (a.state itself is the last segment's to write)
+    const float* from = joined ? a.seg_state + (size_t)seg * states : a.state;
 #pragma unroll
     for (int j = 0; j < NC; ++j) {
         const int c = c0 + cg * NC + j;
-        st[j] = a.state + (ho + c) * a.dimp;
-        if (c < a.dimp && first > 0) s[j].load(st[j], l, a.dimp); else s[j].zero();
+        if (!STATE_ONLY && c < a.dimp && (joined || first > 0)) s[j].load(from + (ho + c) * a.dimp, l, a.dimp); else s[j].zero();
     }
-    for (int t0 = 0, b = 0; t0 < a.T; t0 += kTmTile, b ^= 1) {
-        if (t0 + kTmTile < a.T) { bring(t0 + kTmTile, b ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
+    for (int t0 = t_begin, b = 0; t0 < t_end; t0 += kTmTile, b ^= 1) {
+        if (t0 + kTmTile < t_end) { bring(t0 + kTmTile, b ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
         __syncthreads();
-        const int n = min(kTmTile, a.T - t0);
+        const int n = min(kTmTile, t_end - t0);
 #pragma unroll 2
         for (int t = 0; t < n; ++t) {
             const float* row = tm_smem + (b * kTmTile + t) * ROW;
-            f32x2 r[2 * NV], k[2 * NV], w[2 * NV];
-            lane_units<LPC, NV>(row, l, r); lane_units<LPC, NV>(row + D, l, k); lane_units<LPC, NV>(row + 2 * D, l, w);
-            const float bonus = row[3 * D + CB];
-            float o[NC];
+            f32x2 k[2 * NV], w[2 * NV];
+            float v[NC], o[NC];
+            lane_units<LPC, NV>(row, l, k); lane_units<LPC, NV>(row + D, l, w);
+#pragma unroll
+            for (int j = 0; j < NC; ++j) v[j] = row[3 * D + cg * NC + j];
+            if (!STATE_ONLY) {
+                f32x2 r[2 * NV];
+                lane_units<LPC, NV>(row + 2 * D, l, r);
+                const float bonus = row[3 * D + CB];
+#pragma unroll
+                for (int j = 0; j < NC; ++j) {
+                    f32x2 acc = 0ull, acc1 = 0ull;
+#pragma unroll
+                    for (int i = 0; i < 2 * NV; i += 2) { acc = fma2(s[j].s[i], r[i], acc); acc1 = fma2(s[j].s[i + 1], r[i + 1], acc1); }
+                    o[j] = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v[j];
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 2 * NV; ++i) prod[i] = mul2(prod[i], w[i]);
+            }
 #pragma unroll
             for (int j = 0; j < NC; ++j) {
-                const float v = row[3 * D + cg * NC + j];
-                const f32x2 v2 = pack2(v, v);
-                f32x2 acc = 0ull, acc1 = 0ull;
+                const f32x2 v2 = pack2(v[j], v[j]);
 #pragma unroll
-                for (int i = 0; i < 2 * NV; i += 2) {
-                    acc = fma2(s[j].s[i], r[i], acc); acc1 = fma2(s[j].s[i + 1], r[i + 1], acc1);
-                    s[j].s[i] = fma2(s[j].s[i], w[i], mul2(k[i], v2)); s[j].s[i + 1] = fma2(s[j].s[i + 1], w[i + 1], mul2(k[i + 1], v2));
-                }
-                o[j] = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v;
+                for (int i = 0; i < 2 * NV; ++i) s[j].s[i] = fma2(s[j].s[i], w[i], mul2(k[i], v2));
             }
-            if (l == 0) {
+            if (!STATE_ONLY && l == 0) {
 #pragma unroll
                 for (int j = 0; j < NC; ++j) { const int c = c0 + cg * NC + j; if (c < a.dimp) a.o[(size_t)(t0 + t) * a.ldo + ho + c] = o[j]; }
             }
         }
         __syncthreads();
     }
+    if (!STATE_ONLY && t_end < a.T) return;
+    float* to = STATE_ONLY ? a.seg_state + (size_t)(seg + 1) * states : a.state;
 #pragma unroll
-    for (int j = 0; j < NC; ++j) if (c0 + cg * NC + j < a.dimp) s[j].store(st[j], l, a.dimp);
+    for (int j = 0; j < NC; ++j) if (c0 + cg * NC + j < a.dimp) s[j].store(to + (ho + c0 + cg * NC + j) * a.dimp, l, a.dimp);
+    if (STATE_ONLY && c0 == 0 && cg == 0) {
+        StateCol<LPC, NV> p;
+#pragma unroll
+        for (int i = 0; i < 2 * NV; ++i) p.s[i] = prod[i];
+        p.store(a.seg_decay + ((size_t)seg * a.heads + h) * a.dimp, l, a.dimp);
+    }
+}
+// Slot g of seg_state: what segment g - 1 makes of a zero state becomes the state that segment g begins with, S <- decay product * (state
+// before) + S; slot 0 the portion's.
+__global__ void __launch_bounds__(256) time_mix_join_kernel(const TimeMixArgs a, int nseg) {
+    pdl_launch_dependents(); pdl_wait();
+    const size_t states = (size_t)a.heads * a.dimp * a.dimp, i = ((size_t)blockIdx.x * 256 + threadIdx.x) * 4;
+    if (i >= states) return;
+    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0;
+    const size_t key = i % a.dimp, h = i / ((size_t)a.dimp * a.dimp);
+    float4 s = first > 0 ? *reinterpret_cast<const float4*>(a.state + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    *reinterpret_cast<float4*>(a.seg_state + i) = s;
+#pragma unroll 4
+    for (int g = 1; g < nseg; ++g) {
+        float4* p = reinterpret_cast<float4*>(a.seg_state + (size_t)g * states + i);
+        const float4 x = *p, w = *reinterpret_cast<const float4*>(a.seg_decay + ((size_t)(g - 1) * a.heads + h) * a.dimp + key);
+        s = make_float4(fmaf(w.x, s.x, x.x), fmaf(w.y, s.y, x.y), fmaf(w.z, s.z, x.z), fmaf(w.w, s.w, x.w));
+        *p = s;
+    }
 }
 template <int LPC, int NV>
-static int tm_go(const TimeMixArgs& a, const LaunchCfg& cfg) {
-    constexpr int NC = 2, CB = 32, D = LPC * NV * 4;
+static int tm_go(TimeMixArgs a, const LaunchCfg& cfg) {
+    constexpr int NC = 4, CB = 32, D = LPC * NV * 4, NT = CB / NC * LPC;
     const size_t smem = (size_t)2 * kTmTile * (3 * D + CB + 4) * 4;
     static bool once = false;
     if (!once) {
-        const cudaError_t e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return (int)e;
         once = true;
     }
-    return st_launch(time_mix_scan_kernel<LPC, NV, NC, CB>, dim3(a.heads, (a.dimp + CB - 1) / CB), dim3(CB / NC * LPC), smem, cfg, a);
+    const int nseg = (a.T + a.seg_len - 1) / a.seg_len, cy = (a.dimp + CB - 1) / CB;
+    if (nseg > 1) {
+        if (int r = st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, true>, dim3(a.heads, cy, nseg - 1), dim3(NT), smem, cfg, a)) return r;
+        if (int r = st_launch(time_mix_join_kernel, dim3((unsigned)(((size_t)a.heads * a.dimp * a.dimp / 4 + 255) / 256)), dim3(256), 0, cfg, a, nseg)) return r;
+    }
+    return st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, false>, dim3(a.heads, cy, nseg), dim3(NT), smem, cfg, a);
+}
+// Segments of a portion: as many as fill the SMs with a few CTAs each, none shorter than 128 tokens.
+int time_mix_segment(int heads, int dimp, int T, int sm_count) {
+    const int ctas = heads * ((dimp + 31) / 32);
+    int n = (8 * sm_count + ctas - 1) / ctas;
+    if (n > T / 128) n = T / 128;
+    if (n > kTmMaxSeg) n = kTmMaxSeg;
+    return n < 2 ? T : (T + n - 1) / n;
 }
 int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg) {
-    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.ld % 4 || a.ldz % 4) return (int)cudaErrorInvalidValue;
+    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.ld % 4 || a.ldz % 4 || a.seg_len < 1 || (a.seg_len < a.T && (!a.seg_state || !a.seg_decay))) return (int)cudaErrorInvalidValue;
 #define GO(L, N) tm_go<L, N>(a, cfg)
     return RECUR_DISPATCH(a.dimp, GO);
 #undef GO

@@ -147,12 +147,13 @@ def test_time_mixing(built, heads, dim, n):
     (w0, w064), (u, u64) = f32_pair(rng, W), f32_pair(rng, W)
     w0, w064 = w0 - 3, w064 - 3
     hd = lambda a: a.reshape(-1, heads, dim)
+    seg_state, seg_decay = E.DevBuf(16 * W * dim * 4), E.DevBuf(16 * W * 4)
     want = M.bonus_recurrence(hd(r64), hd(k64), hd(v64), np.exp(-np.exp(hd(z64 + w064))), u64.reshape(heads, dim)).reshape(n, W)
-    for sizes in ([n], [1], [2, 15, 16, 17, 1, 33]):
+    for sizes, seg in (([n], 0), ([1], 0), ([2, 15, 16, 17, 1, 33], 0), ([n], -(-n // 9)), ([3, n], -(-n // 2)), ([n], 16 if n > 16 else n - 1)):
         pool, state, got = Pool(), dev(np.full(W * dim, 3.0, np.float32)), []          # what an earlier sequence left does not matter
         for i, m in pieces(n, sizes):
             o = E.DevBuf(m * W * 4)
-            K.time_mix(*[pool.p(a[i:i + m]) for a in (r, k, v)], pool.p(z[i:i + m].copy()), pool.p(w0), pool.p(u), E.DevBuf(m * heads * 4), state, o, heads, dim, m, i)
+            K.time_mix(*[pool.p(a[i:i + m]) for a in (r, k, v)], pool.p(z[i:i + m].copy()), pool.p(w0), pool.p(u), E.DevBuf(m * heads * 4), state, o, heads, dim, m, i, seg, seg_state, seg_decay)
             E.sync()
             got.append(o.numpy(np.float32).reshape(m, W))
         near(np.concatenate(got).astype(np.float64), want, "float32", 3.0)
@@ -228,7 +229,7 @@ def test_bad_arguments_are_refused(built):
                  lambda: K.linear_epi(0, K.LIN_CAP, b, 8, b, 128, 8, 1, 16, b, 16, 0, 0), lambda: K.shift_mix(0, b, 12, b, 10, 1e-6, b, 1, b, b, b, 0, 1),
                  lambda: K.grouped_attention(1, 0, b, b, b, 8, None, 0, b, None, 1, 0, None, 2, 1, 8, 8, 1.0, 1.0), lambda: K.grouped_attention(0, 2, b, b, b, 8, None, 0, b, b, 2, 0, b, 2, 1, 8, 8, 1.0, 1.0),
                  lambda: K.grouped_attention(0, 0, b, b, b, 8, None, 0, b, None, 1, 0, None, 3, 2, 8, 8, 1.0, 1.0), lambda: K.grouped_attention(0, 0, b, b, b, 8, None, 0, b, None, 4, 5, None, 2, 1, 8, 8, 1.0, 1.0),
-                 lambda: K.time_mix(b, b, b, b, b, b, b, b, b, 1, 520, 1, 0), lambda: K.time_mix_step(b, b, 128, 1, b, b, b, b, b, 1, 12, 1e-6, 1.0, b),
+                 lambda: K.time_mix(b, b, b, b, b, b, b, b, b, 1, 520, 1, 0, 0, None, None), lambda: K.time_mix(b, b, b, b, b, b, b, b, b, 1, 8, 4, 0, 2, None, None), lambda: K.time_mix_step(b, b, 128, 1, b, b, b, b, b, 1, 12, 1e-6, 1.0, b),
                  lambda: K.delta(b, b, 0, b, b, b, b, b, b, b, b, 2, 1, 8, 8, 1, 0), lambda: K.delta_step(b, b, 4, b, b, b, b, b, b, 3, 2, 8, 8, 1e-6, b)):
         with pytest.raises(CuQwenError) as e:
             call()
