@@ -86,10 +86,10 @@ SIGNATURES = {
     "cuqwen_k_latent_rows": (_i, [_i, _i, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _f, _i, _i]),
     "cuqwen_k_rot_table": (_i, [_i, _vp, _i, _i, C.c_double]),
     "cuqwen_k_latent_attention": (_i, [_i, _i, _i] + [_vp] * 7 + [_i] * 8 + [_f]),
-    "cuqwen_k_linear_epi": (_i, [_i, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _f, _f]),
+    "cuqwen_k_linear_epi": (_i, [_i, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _f, _f, _vp]),
     "cuqwen_k_shift_mix": (_i, [_i, _i, _vp, _i, _vp, _i, _f, _vp, _i, _vp, _vp, _vp, _i, _i]),
     "cuqwen_k_grouped_attention": (_i, [_i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _f]),
-    "cuqwen_k_time_mix": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp]),
+    "cuqwen_k_time_mix": (_i, [_i] + [_vp] * 7 + [_i] * 5 + [_vp, _vp]),
     "cuqwen_k_time_mix_step": (_i, [_i, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _f, _vp]),
     "cuqwen_k_delta": (_i, [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i]),
     "cuqwen_k_delta_step": (_i, [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _vp]),

@@ -1401,16 +1401,17 @@ extern "C" int cuqwen_k_latent_attention(int device, int act, int impl, const vo
     return CUQWEN_OK;
 }
 
-extern "C" int cuqwen_k_linear_epi(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, int n_tokens, int rows, void* out, int ldo, float c0, float c1) {
+extern "C" int cuqwen_k_linear_epi(int device, int act, int epi, const void* x, int ldx, const void* w, int pitch, int cols, int n_tokens, int rows, void* out, int ldo, float c0, float c1, const float* bias) {
     DEV(device);
     NOT_NULL(x, w, out);
-    if (bad_act(act) || (epi != LIN_ADD && epi != LIN_CAP && epi != LIN_GLU) || n_tokens < 1 || rows < 8 || rows % 8 || (epi == LIN_GLU && (rows % 16 || act == CUQWEN_ACT_F32)) || cols < 8 || cols % 8 || pitch % 128 ||
-        pitch < cols || ldx % 8 || ldx < cols || ldo % 8 || ldo < (epi == LIN_GLU ? rows / 2 : rows) || (epi == LIN_CAP && !(c0 > 0.f)))
-        return fail(CUQWEN_ERR_ARG, "linear_epi: rows, cols and row strides are multiples of 8, the weight pitch of 128; the gated unit has rows in sixteens and bfloat16");
+    if (bad_act(act) || (epi != LIN_ADD && epi != LIN_CAP && epi != LIN_GLU && epi != LIN_DECAY) || n_tokens < 1 || rows < 8 || rows % 8 || (epi == LIN_GLU && (rows % 16 || act == CUQWEN_ACT_F32)) || cols < 8 || cols % 8 || pitch % 128 ||
+        pitch < cols || ldx % 8 || ldx < cols || ldo % 8 || ldo < (epi == LIN_GLU ? rows / 2 : rows) || (epi == LIN_CAP && !(c0 > 0.f)) ||
+        (epi == LIN_DECAY && (!bias || (act == CUQWEN_ACT_BF16 && n_tokens == 1))))
+        return fail(CUQWEN_ERR_ARG, "linear_epi: rows, cols and row strides are multiples of 8, the weight pitch of 128; the gated unit has rows in sixteens and bfloat16, the decay of one bfloat16 row is time_mix_step's");
     if (act == CUQWEN_ACT_BF16 && n_tokens > 1) {
         PfGemmArgs g; memset(&g, 0, sizeof g);
         const PfBf16Mat m{w, rows, pitch};
-        g.T = n_tokens; g.K = cols; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = t_err; g.mode = epi == LIN_ADD ? PF_ADD_F32 : epi == LIN_CAP ? PF_CAP_F32 : PF_BF16_GLU; g.c0 = c0; g.c1 = c1;
+        g.T = n_tokens; g.K = cols; g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = t_err; g.mode = epi == LIN_ADD ? PF_ADD_F32 : epi == LIN_CAP ? PF_CAP_F32 : epi == LIN_DECAY ? PF_DECAY_F32 : PF_BF16_GLU; g.c0 = c0; g.c1 = c1; g.bias_f = bias;
         KK(launch_prefill_gemm_bf16(g, x, ldx, &m, 1, nullptr, 0, nullptr, dc->stream));
         return CUQWEN_OK;
     }
@@ -1422,7 +1423,7 @@ extern "C" int cuqwen_k_linear_epi(int device, int act, int epi, const void* x, 
         return CUQWEN_OK;
     }
     LinArgs a{};
-    a.x = x; a.ldx = ldx; a.w = (const bf16*)w; a.pitch = pitch; a.K = cols; a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.c0 = c0; a.c1 = c1;
+    a.x = x; a.ldx = ldx; a.w = (const bf16*)w; a.pitch = pitch; a.K = cols; a.T = n_tokens; a.R = rows; a.epi = epi; a.out = out; a.ldo = ldo; a.c0 = c0; a.c1 = c1; a.bias = bias;
     KK(launch_st_linear(act, a, cfg));
     return CUQWEN_OK;
 }
@@ -1466,16 +1467,16 @@ extern "C" int cuqwen_k_grouped_attention(int device, int act, int impl, const f
     else KK(launch_latent_attn(act, t, cfg));
     return CUQWEN_OK;
 }
-extern "C" int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, float* z, const float* w0, const float* u, float* bonus, float* state, float* o, int heads, int dim, int n_tokens, int pos0,
-                                 int segment, float* seg_state, float* seg_decay) {
+extern "C" int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v, const float* w, const float* u, float* state, float* o, int heads, int dim, int n_tokens, int pos0, int segment, float* seg_state,
+                                 float* seg_decay) {
     DEV(device);
-    NOT_NULL(r, k, v, z, w0, u, bonus, state, o);
-    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || n_tokens < 1 || pos0 < 0 || segment < 0 || (segment > 0 && (n_tokens + segment - 1) / segment > kTmMaxSeg)) return fail(CUQWEN_ERR_ARG, "time_mix: dim is a multiple of 8, at most %d", kRecurMaxDim);
+    NOT_NULL(r, k, v, w, u, state, o);
+    if (heads < 1 || dim < 8 || dim % 8 || dim > kRecurMaxDim || n_tokens < 1 || pos0 < 0 || segment < 0 || (segment > 0 && (n_tokens + segment - 1) / segment > kTmMaxSeg))
+        return fail(CUQWEN_ERR_ARG, "time_mix: dim is a multiple of 8, at most %d; at most %d segments", kRecurMaxDim, kTmMaxSeg);
     TimeMixArgs a{};
-    a.r = r; a.k = k; a.v = v; a.ld = a.ldz = a.ldo = heads * dim; a.z = z; a.w0 = w0; a.u = u; a.bonus = bonus; a.heads = heads; a.dim = a.dimp = dim; a.T = n_tokens; a.state = state; a.o = o; a.pos0 = pos0;
+    a.r = r; a.k = k; a.v = v; a.ld = a.ldw = a.ldo = heads * dim; a.w = w; a.u = u; a.heads = heads; a.dimp = dim; a.T = n_tokens; a.state = state; a.o = o; a.pos0 = pos0; a.err = t_err;
     a.seg_len = segment > 0 && segment < n_tokens ? segment : n_tokens; a.seg_state = seg_state; a.seg_decay = seg_decay;
     if (a.seg_len < n_tokens) NOT_NULL(seg_state, seg_decay);
-    KK(launch_time_mix_rows(a, cfg));
     KK(launch_time_mix_scan(a, cfg));
     return CUQWEN_OK;
 }

@@ -87,6 +87,16 @@ __device__ __forceinline__ void pf_store_bf16(const PfGemmArgs& a, const float (
                 *reinterpret_cast<float4*>(dst + i) = make_float4(a.c0 * tanhf(v[i] / a.c0), a.c0 * tanhf(v[i + 1] / a.c0), a.c0 * tanhf(v[i + 2] / a.c0), a.c0 * tanhf(v[i + 3] / a.c0));
         return;
     }
+    if (a.mode == PF_DECAY_F32) {
+        float* dst = a.out_f + (size_t)token * a.ldo + coff + r;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4)
+            if (r + i < R) {
+                const float4 z = *reinterpret_cast<const float4*>(a.bias_f + coff + r + i);
+                *reinterpret_cast<float4*>(dst + i) = make_float4(expf(-expf(v[i] + z.x)), expf(-expf(v[i + 1] + z.y)), expf(-expf(v[i + 2] + z.z)), expf(-expf(v[i + 3] + z.w)));
+            }
+        return;
+    }
     if (a.mode == PF_BF16_GLU) {
         __nv_bfloat16* dst = a.out_b + (size_t)token * a.ldo + r / 2;
 #pragma unroll

@@ -51,7 +51,8 @@ enum PfMode : int {
     PF_ADD_F32 = 6,         // out_f[t][r] += c0 * acc
     PF_BF16_GELU_SIDE = 7,  // out_b[t][r] = gelu_tanh(acc) * side[tokens[t]][r], r < side_dim, else 0
     PF_CAP_F32 = 8,         // out_f[t][r] = c0 * tanh(acc / c0)
-    PF_BF16_GLU = 9         // out_b[t][i] = clamped_glu(gate row i, up row i; limit c0, slope c1), rows as eight of each in turn
+    PF_BF16_GLU = 9,        // out_b[t][i] = clamped_glu(gate row i, up row i; limit c0, slope c1), rows as eight of each in turn
+    PF_DECAY_F32 = 10       // out_f[t][r] = exp(-exp(acc + bias_f[r]))
 };
 constexpr int kPfMaxMat = 6;
 
@@ -78,6 +79,7 @@ struct PfGemmArgs {
     int K2;
     const __nv_bfloat16* side; int side_pitch, side_dim; const int* tokens;
     float c0, c1;              // constants of the epilogue
+    const float* bias_f;
 };
 
 // Fills the tensor maps and launches.  PF_SWIGLU: w = {gate, up}, nmat = 2, rows[0] = rows of each.  Other modes: nmat

@@ -61,6 +61,7 @@ enum LinEpi : int {
     LIN_ADD = 3,          // out (float) += c0 * acc
     LIN_GELU_SIDE = 4,    // out (activation type) = gelu_tanh(acc) * side[tokens[t]][r]
     LIN_CAP = 5,          // out (float) = c0 * tanh(acc / c0)
+    LIN_DECAY = 7,        // out (float) = exp(-exp(acc + bias[r]))
     LIN_GLU = 6           // out (activation type) = clamped_glu(gate, up, limit c0, slope c1); rows come as eight of the gate, eight of the up matrix in turn
 };
 struct LinArgs {
@@ -70,6 +71,7 @@ struct LinArgs {
     void* out; int ldo;
     const bf16* side; int side_pitch, side_dim; const int* tokens; // LIN_GELU_SIDE
     float c0, c1;                                                  // constants of the epilogue
+    const float* bias;                                             // LIN_DECAY
 };
 // LIN_GLU is not among its epilogues: LIN_F32, then launch_st_glu_rows.
 int launch_st_linear(int act, const LinArgs& a, const LaunchCfg& cfg);
@@ -168,18 +170,18 @@ int launch_head_norm_gate(int act, const HeadNormArgs& a, int T, const LaunchCfg
 constexpr int kRecurMaxDim = 512;                                   // key channels of a head
 
 // Time mixing (time_mix.cu).  State [heads][dimp (value channel)][dimp (key channel)].
-// time_mix_rows: z -> exp(-exp(z + w0)) in place; bonus[t][h] = sum_i r_i u_i k_i.
 struct TimeMixArgs {
     const float *r, *k, *v; int ld;                                 // heads dimp apart
-    float* z; int ldz; const float *w0, *u; float* bonus;
-    int heads, dim, dimp, T;
+    const float* w; int ldw;                                        // decays
+    const float* u;
+    int heads, dimp, T;
     float* state; float* o; int ldo;
     const int* pos_ptr; int pos0;
     int seg_len; float *seg_state, *seg_decay;                      // tokens of a segment (T: one segment, no scratch); scratch [kTmMaxSeg][state], [kTmMaxSeg][heads][dimp]
+    unsigned* err;
 };
 constexpr int kTmMaxSeg = 16;
 int time_mix_segment(int heads, int dimp, int T, int sm_count);    // a good seg_len
-int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg);
 int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg);
 // One token in bfloat16: low-rank decay, recurrence, head norm, gate - and, in the same launch, the token's qkv rows (qkv.raw null: none).
 struct TimeMixStepArgs {

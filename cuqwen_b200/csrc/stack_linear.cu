@@ -12,6 +12,7 @@ __device__ __forceinline__ void lin_store(const LinArgs& a, int t, int r, float 
         case LIN_ACT: reinterpret_cast<A*>(a.out)[o] = to_act<A>(v); break;
         case LIN_RELU2: { const float p = fmaxf(v, 0.f); reinterpret_cast<A*>(a.out)[o] = to_act<A>(p * p); break; }
         case LIN_ADD: reinterpret_cast<float*>(a.out)[o] += a.c0 * v; break;
+        case LIN_DECAY: reinterpret_cast<float*>(a.out)[o] = expf(-expf(v + a.bias[r])); break;
         case LIN_CAP: reinterpret_cast<float*>(a.out)[o] = a.c0 * tanhf(v / a.c0); break;
         case LIN_GELU_SIDE: {
             const float e = r < a.side_dim ? __bfloat162float(a.side[(size_t)a.tokens[t] * a.side_pitch + r]) : 0.f;

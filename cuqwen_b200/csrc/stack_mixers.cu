@@ -20,8 +20,8 @@ TimeMixArgs Pass::time_mix(const StLayer& l) {
     const TimeMixSpec& t = l.spec.right;
     TimeMixArgs a{};
     a.r = w->raw + l.in_off[1]; a.k = w->raw + l.in_off[2]; a.v = w->raw + l.in_off[3]; a.ld = l.ldraw;
-    a.z = w->z; a.ldz = t.heads * l.rdimp; a.w0 = l.w0; a.u = l.u; a.bonus = (float*)w->sc;
-    a.heads = t.heads; a.dim = t.dim; a.dimp = l.rdimp; a.T = T;
+    a.w = w->z; a.ldw = t.heads * l.rdimp; a.u = l.u; a.err = err_word();
+    a.heads = t.heads; a.dimp = l.rdimp; a.T = T;
     a.state = (float*)at(l.state_off); a.o = w->ro; a.ldo = t.heads * l.rdimp; a.pos_ptr = pos_ptr; a.pos0 = pos0;
     a.seg_len = T > 1 ? time_mix_segment(t.heads, l.rdimp, T, cfg.sm_count) : 1; a.seg_state = w->seg_state; a.seg_decay = w->seg_decay;
     return a;
@@ -81,10 +81,10 @@ int Pass::parallel_mixer(const StLayer& l, bool stop) {
     GO(launch_tanh_rows(s->act, w->raw + l.in_off[5], l.ldraw, w->zin, l.rankp, part, t.rank, T, cfg));
     const StMat* w2[1] = {&l.w2};
     With low;
+    low.bias = l.w0;
     if (s->act == ACT_BF16) { low.x2 = (const uint8_t*)w->zin + part * s->esz; low.ldx2 = l.rankp; low.m2 = &l.w2; }
-    if (int r = product(LIN_F32, w->zin, l.rankp, w2, 1, w->z, t.heads * l.rdimp, T, low)) return r;
+    if (int r = product(LIN_DECAY, w->zin, l.rankp, w2, 1, w->z, t.heads * l.rdimp, T, low)) return r;
     const TimeMixArgs tm = time_mix(l);
-    GO(launch_time_mix_rows(tm, cfg));
     GO(launch_time_mix_scan(tm, cfg));
     if (stop) return CUQWEN_OK;
     HeadNormArgs n{w->ro, tm.ldo, t.heads, t.dim, l.rdimp, l.head_norm, l.rdimp, w->raw + l.in_off[4], l.ldraw, (float)sp.norm_eps, (float)l.spec.right_scale, w->att2, tm.ldo};

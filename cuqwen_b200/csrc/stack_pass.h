@@ -110,6 +110,7 @@ struct Pass {
         const void* x2 = nullptr; int ldx2 = 0; const StMat* m2 = nullptr;
         const LinArgs* side = nullptr;
         float c0 = 1.f, c1 = 0.f;
+        const float* bias = nullptr;
         int var_rows = 0;
     };
     // out[t] = epilogue(W x[t]) for n rows of x; several matrices (one epilogue) write their rows side by side.  The tensor-core GEMM in
@@ -117,11 +118,11 @@ struct Pass {
     int product(int epi, const void* x, int ldx, const StMat* const* m, int nm, void* out, int ldo, int n) { return product(epi, x, ldx, m, nm, out, ldo, n, With{}); }
     int product(int epi, const void* x, int ldx, const StMat* const* m, int nm, void* out, int ldo, int n, const With& o) {
         if (s->act == ACT_BF16 && (n > 1 || epi == LIN_GLU)) {
-            static const int modes[] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE, PF_CAP_F32, PF_BF16_GLU};
+            static const int modes[] = {PF_OUT_F32, PF_BF16, PF_BF16_RELU2, PF_ADD_F32, PF_BF16_GELU_SIDE, PF_CAP_F32, PF_BF16_GLU, PF_DECAY_F32};
             PfGemmArgs g; memset(&g, 0, sizeof g);
             PfBf16Mat pm[kPfMaxMat], pm2{};
             for (int i = 0; i < nm; ++i) pm[i] = PfBf16Mat{m[i]->w, m[i]->rows, m[i]->pitch, i * o.var_rows};
-            g.T = n; g.K = pad8(m[0]->cols); g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = err_word(); g.mode = modes[epi]; g.c0 = o.c0; g.c1 = o.c1;
+            g.T = n; g.K = pad8(m[0]->cols); g.ldo = ldo; g.out_f = (float*)out; g.out_b = (bf16*)out; g.err = err_word(); g.mode = modes[epi]; g.c0 = o.c0; g.c1 = o.c1; g.bias_f = o.bias;
             if (o.m2) { pm2 = PfBf16Mat{o.m2->w, o.m2->rows, o.m2->pitch}; g.K2 = o.m2->cols; }
             if (o.side) { g.side = o.side->side; g.side_pitch = o.side->side_pitch; g.side_dim = o.side->side_dim; g.tokens = o.side->tokens; }
             GO(launch_prefill_gemm_bf16(g, x, ldx, pm, nm, o.m2 ? o.x2 : nullptr, o.ldx2, o.m2 ? &pm2 : nullptr, cfg.stream));
@@ -129,8 +130,8 @@ struct Pass {
         }
         size_t off = 0;
         for (int i = 0; i < nm; ++i) {
-            LinArgs a = lin((const uint8_t*)x + (size_t)i * o.var_rows * ldx * s->esz, ldx, *m[i], epi, (uint8_t*)out + off * (epi == LIN_F32 || epi == LIN_ADD || epi == LIN_CAP ? 4 : s->esz), ldo);
-            a.T = n; a.c0 = o.c0; a.c1 = o.c1;
+            LinArgs a = lin((const uint8_t*)x + (size_t)i * o.var_rows * ldx * s->esz, ldx, *m[i], epi, (uint8_t*)out + off * (epi == LIN_F32 || epi == LIN_ADD || epi == LIN_CAP || epi == LIN_DECAY ? 4 : s->esz), ldo);
+            a.T = n; a.c0 = o.c0; a.c1 = o.c1; a.bias = o.bias;
             if (o.m2) { a.x2 = o.x2; a.ldx2 = o.ldx2; a.w2 = o.m2->w; a.pitch2 = o.m2->pitch; a.K2 = o.m2->cols; }
             if (o.side) { a.side = o.side->side; a.side_pitch = o.side->side_pitch; a.side_dim = o.side->side_dim; a.tokens = o.side->tokens; }
             GO(launch_st_linear(s->act, a, cfg));

@@ -1,8 +1,8 @@
 // Time mixing: state S of a head with a decay per key channel, S <- diag(w) S + k v^T, read out before the update with a bonus
 // for the current token: o = S^T r + (sum_i r_i u_i k_i) v.  All of it in float32.
 //
-// Portions: the row kernel turns the low-rank products into decays and takes the bonus sums; the scan walks the tokens with the
-// state in registers (recur.cuh), r, k, decays and values brought a tile of tokens at a time by cp.async.  Value channels are
+// Portions: the scan walks the tokens with the state in registers (recur.cuh); r, k, the decays (made in the epilogue of the low-rank
+// product) and the values come a tile of tokens at a time by TMA, the bonus is summed beside the read-out.  Value channels are
 // independent of one another, so a head is cut into CTAs of a few of them; and since a segment of the portion acts on the state it
 // begins with by a factor per key channel and a sum, a long portion is also cut into segments.
 #include "qkv_rows.cuh"
@@ -10,117 +10,95 @@
 
 namespace cq {
 
-// A warp per (row, head).
-__global__ void __launch_bounds__(256) time_mix_rows_kernel(const TimeMixArgs a) {
-    pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = blockIdx.x;
-    if (h >= a.heads) return;
-    const size_t o = (size_t)h * a.dimp;
-    const float *r = a.r + (size_t)t * a.ld + o, *k = a.k + (size_t)t * a.ld + o, *u = a.u + o, *w0 = a.w0 + o;
-    float* z = a.z + (size_t)t * a.ldz + o;
-    float b = 0.f;
-    for (int i = lane; i < a.dimp; i += 32) {
-        z[i] = expf(-expf(z[i] + w0[i]));
-        b = fmaf(r[i] * u[i], k[i], b);                 // padded places hold zeros
-    }
-    b = warp_sum(b);
-    if (lane == 0) a.bonus[(size_t)t * a.heads + h] = b;
-}
-int launch_time_mix_rows(const TimeMixArgs& a, const LaunchCfg& cfg) {
-    return st_launch(time_mix_rows_kernel, dim3(a.T, (a.heads + 7) / 8), dim3(256), 0, cfg, a);
-}
-
-constexpr int kTmTile = 16;                             // tokens brought at a time
+struct TimeMixTmaps { CUtensorMap r, k, w, v; };
 // CTA: head x CB value channels x segment of the portion, NC channels to a thread.  A portion of several segments takes three passes:
 // every segment's state from zero and its decay product (STATE_ONLY), the states the segments begin with (time_mix_join_kernel), and the
 // segments' outputs.
 template <int LPC, int NV, int NC, int CB, bool STATE_ONLY>
-__global__ void __launch_bounds__(CB / NC * LPC) time_mix_scan_kernel(const TimeMixArgs a) {
-    constexpr int D = LPC * NV * 4, NT = CB / NC * LPC, ROW = 3 * D + CB + 4;            // k | w | r | v | bonus
-    extern __shared__ __align__(16) float tm_smem[];    // [2][kTmTile][ROW]
-    pdl_launch_dependents(); pdl_wait();
+__global__ void __launch_bounds__(CB / NC * LPC) time_mix_scan_kernel(const TimeMixArgs a, const __grid_constant__ TimeMixTmaps m) {
+    constexpr int D = LPC * NV * 4, NVEC = STATE_ONLY ? 2 : 3, STAGE = kRecurTile * (NVEC * D + CB);      // k | w | (r) | v
+    static_assert(NC == 4, "a thread's channels are one 16-byte unit of a value row");
+    extern __shared__ __align__(128) float tm_smem[];   // [2][STAGE]
+    __shared__ __align__(8) unsigned long long bars[2];
+    const uint32_t bar = smem_u32(bars), sm0 = smem_u32(tm_smem);
     const int h = blockIdx.x, c0 = blockIdx.y * CB, seg = blockIdx.z, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC;
-    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0, nc = min(CB, a.dimp - c0);
+    if (tid == 0) { mbar_init(bar, 1); mbar_init(bar + 8, 1); mbar_fence_init(); }
+    pdl_launch_dependents(); pdl_wait();
+    __syncthreads();
+    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0;
     const int t_begin = seg * a.seg_len, t_end = min(t_begin + a.seg_len, a.T);
     const size_t ho = (size_t)h * a.dimp, states = (size_t)a.heads * a.dimp * a.dimp;
-    for (int i = tid; i < 2 * kTmTile * ROW; i += NT) tm_smem[i] = 0.f;                 // what no copy reaches stays zero
-    __syncthreads();
-    // a warp brings whole tokens, a lane 16-byte units
-    auto bring = [&](int t0, int b) {
-        const int n = min(kTmTile, t_end - t0), du = a.dimp / 4, cu = nc / 4;
-        for (int t = tid >> 5; t < n; t += NT / 32) {
-            const size_t tt = (size_t)(t0 + t);
-            float* dst = tm_smem + (b * kTmTile + t) * ROW;
-            const float *k = a.k + tt * a.ld + ho, *w = a.z + tt * a.ldz + ho, *r = a.r + tt * a.ld + ho, *v = a.v + tt * a.ld + ho + c0;
-            for (int u = tid & 31; u < du; u += 32) {
-                cp_async16(dst + 4 * u, k + 4 * u); cp_async16(dst + D + 4 * u, w + 4 * u);
-                if (!STATE_ONLY) cp_async16(dst + 2 * D + 4 * u, r + 4 * u);
-            }
-            for (int u = tid & 31; u < cu; u += 32) cp_async16(dst + 3 * D + 4 * u, v + 4 * u);
-            if (!STATE_ONLY && (tid & 31) == 0) dst[3 * D + CB] = a.bonus[tt * a.heads + h];
-        }
-        cp_async_commit();
+    auto bring = [&](int t, int b) {
+        const uint32_t dst = sm0 + b * STAGE * 4, fb = bar + 8 * b;
+        mbar_expect_tx(fb, STAGE * 4);
+        recur_load<D>(dst, &m.k, 0, h, t, fb); recur_load<D>(dst + kRecurTile * D * 4, &m.w, 0, h, t, fb);
+        if (!STATE_ONLY) recur_load<D>(dst + 2 * kRecurTile * D * 4, &m.r, 0, h, t, fb);
+        tma_load_3d(dst + NVEC * kRecurTile * D * 4, &m.v, c0, h, t, fb);
     };
-    bring(t_begin, 0);
+    if (tid == 0) { bring(t_begin, 0); if (t_begin + kRecurTile < t_end) bring(t_begin + kRecurTile, 1); }
     StateCol<LPC, NV> s[NC];
-    f32x2 prod[2 * NV];
+    f32x2 aux[2 * NV];                                  // STATE_ONLY: decay product; else the bonus of this lane's key channels
 #pragma unroll
-    for (int i = 0; i < 2 * NV; ++i) prod[i] = pack2(1.f, 1.f);
+    for (int i = 0; i < NV; ++i) {
+        const int k = (i * LPC + l) * 4;
+        ulonglong2 u = make_ulonglong2(0ull, 0ull);
+        if (STATE_ONLY) u.x = u.y = pack2(1.f, 1.f);
+        else if (k < a.dimp) u = *reinterpret_cast<const ulonglong2*>(a.u + ho + k);
+        aux[2 * i] = u.x; aux[2 * i + 1] = u.y;
+    }
     const bool joined = gridDim.z > 1;                  // every segment begins with its slot of seg_state (a.state itself is the last segment's to write)
     const float* from = joined ? a.seg_state + (size_t)seg * states : a.state;
+    const int c = c0 + cg * NC;                         // this thread's channels; dimp is a multiple of eight: all of them exist or none
 #pragma unroll
-    for (int j = 0; j < NC; ++j) {
-        const int c = c0 + cg * NC + j;
-        if (!STATE_ONLY && c < a.dimp && (joined || first > 0)) s[j].load(from + (ho + c) * a.dimp, l, a.dimp); else s[j].zero();
-    }
-    for (int t0 = t_begin, b = 0; t0 < t_end; t0 += kTmTile, b ^= 1) {
-        if (t0 + kTmTile < t_end) { bring(t0 + kTmTile, b ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
-        __syncthreads();
-        const int n = min(kTmTile, t_end - t0);
+    for (int j = 0; j < NC; ++j) if (!STATE_ONLY && c < a.dimp && (joined || first > 0)) s[j].load(from + (ho + c + j) * a.dimp, l, a.dimp); else s[j].zero();
+    bool failed = false;
+    for (int t0 = t_begin, i = 0; t0 < t_end; t0 += kRecurTile, ++i) {
+        const int b = i & 1;
+        if (!failed && !mbar_wait(bar + 8 * b, (uint32_t)(i >> 1) & 1u)) { failed = true; if (a.err) atomicExch(a.err, 21u); }
+        const float *kb = tm_smem + b * STAGE, *wb = kb + kRecurTile * D, *rb = wb + kRecurTile * D, *vb = kb + NVEC * kRecurTile * D;
+        const int n = min(kRecurTile, t_end - t0);
 #pragma unroll 2
         for (int t = 0; t < n; ++t) {
-            const float* row = tm_smem + (b * kTmTile + t) * ROW;
             f32x2 k[2 * NV], w[2 * NV];
-            float v[NC], o[NC];
-            lane_units<LPC, NV>(row, l, k); lane_units<LPC, NV>(row + D, l, w);
-#pragma unroll
-            for (int j = 0; j < NC; ++j) v[j] = row[3 * D + cg * NC + j];
+            lane_row<LPC, NV>(kb, t, l, k); lane_row<LPC, NV>(wb, t, l, w);
+            const float4 v4 = *reinterpret_cast<const float4*>(vb + t * CB + cg * NC);
+            const float v[4] = {v4.x, v4.y, v4.z, v4.w};
             if (!STATE_ONLY) {
-                f32x2 r[2 * NV];
-                lane_units<LPC, NV>(row + 2 * D, l, r);
-                const float bonus = row[3 * D + CB];
+                f32x2 r[2 * NV], bon = 0ull;
+                float o[NC];
+                lane_row<LPC, NV>(rb, t, l, r);
+#pragma unroll
+                for (int q = 0; q < 2 * NV; ++q) bon = fma2(mul2(r[q], aux[q]), k[q], bon);
 #pragma unroll
                 for (int j = 0; j < NC; ++j) {
-                    f32x2 acc = 0ull, acc1 = 0ull;
+                    f32x2 acc = mul2(bon, pack2(v[j], v[j])), acc1 = 0ull;
 #pragma unroll
-                    for (int i = 0; i < 2 * NV; i += 2) { acc = fma2(s[j].s[i], r[i], acc); acc1 = fma2(s[j].s[i + 1], r[i + 1], acc1); }
-                    o[j] = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v[j];
+                    for (int q = 0; q < 2 * NV; q += 2) { acc = fma2(s[j].s[q], r[q], acc); acc1 = fma2(s[j].s[q + 1], r[q + 1], acc1); }
+                    o[j] = lanes_sum<LPC>(sum2(add2(acc, acc1)));
                 }
+                if (l == 0 && c < a.dimp) *reinterpret_cast<float4*>(a.o + (size_t)(t0 + t) * a.ldo + ho + c) = make_float4(o[0], o[1], o[2], o[3]);
             } else {
 #pragma unroll
-                for (int i = 0; i < 2 * NV; ++i) prod[i] = mul2(prod[i], w[i]);
+                for (int q = 0; q < 2 * NV; ++q) aux[q] = mul2(aux[q], w[q]);
             }
 #pragma unroll
             for (int j = 0; j < NC; ++j) {
                 const f32x2 v2 = pack2(v[j], v[j]);
 #pragma unroll
-                for (int i = 0; i < 2 * NV; ++i) s[j].s[i] = fma2(s[j].s[i], w[i], mul2(k[i], v2));
-            }
-            if (!STATE_ONLY && l == 0) {
-#pragma unroll
-                for (int j = 0; j < NC; ++j) { const int c = c0 + cg * NC + j; if (c < a.dimp) a.o[(size_t)(t0 + t) * a.ldo + ho + c] = o[j]; }
+                for (int q = 0; q < 2 * NV; ++q) s[j].s[q] = fma2(s[j].s[q], w[q], mul2(k[q], v2));
             }
         }
         __syncthreads();
+        if (tid == 0 && t0 + 2 * kRecurTile < t_end) bring(t0 + 2 * kRecurTile, b);
     }
     if (!STATE_ONLY && t_end < a.T) return;
     float* to = STATE_ONLY ? a.seg_state + (size_t)(seg + 1) * states : a.state;
 #pragma unroll
-    for (int j = 0; j < NC; ++j) if (c0 + cg * NC + j < a.dimp) s[j].store(to + (ho + c0 + cg * NC + j) * a.dimp, l, a.dimp);
+    for (int j = 0; j < NC; ++j) if (c < a.dimp) s[j].store(to + (ho + c + j) * a.dimp, l, a.dimp);
     if (STATE_ONLY && c0 == 0 && cg == 0) {
         StateCol<LPC, NV> p;
 #pragma unroll
-        for (int i = 0; i < 2 * NV; ++i) p.s[i] = prod[i];
+        for (int q = 0; q < 2 * NV; ++q) p.s[q] = aux[q];
         p.store(a.seg_decay + ((size_t)seg * a.heads + h) * a.dimp, l, a.dimp);
     }
 }
@@ -143,22 +121,28 @@ __global__ void __launch_bounds__(256) time_mix_join_kernel(const TimeMixArgs a,
     }
 }
 template <int LPC, int NV>
-static int tm_go(TimeMixArgs a, const LaunchCfg& cfg) {
+static int tm_go(const TimeMixArgs& a, const LaunchCfg& cfg) {
     constexpr int NC = 4, CB = 32, D = LPC * NV * 4, NT = CB / NC * LPC;
-    const size_t smem = (size_t)2 * kTmTile * (3 * D + CB + 4) * 4;
+    const size_t smem = (size_t)2 * kRecurTile * (3 * D + CB) * 4, smem2 = (size_t)2 * kRecurTile * (2 * D + CB) * 4;
     static bool once = false;
     if (!once) {
-        cudaError_t e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(time_mix_scan_kernel<LPC, NV, NC, CB, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
         if (e != cudaSuccess) return (int)e;
         once = true;
     }
+    TimeMixTmaps m;
+    auto map = [&](CUtensorMap* t, const float* p, int ld, int box) { return recur_map(t, p, a.dimp, a.heads, a.dimp, a.T, ld, box, kRecurTile); };
+    if (int r = map(&m.r, a.r, a.ld, recur_box(D))) return r;
+    if (int r = map(&m.k, a.k, a.ld, recur_box(D))) return r;
+    if (int r = map(&m.w, a.w, a.ldw, recur_box(D))) return r;
+    if (int r = map(&m.v, a.v, a.ld, CB)) return r;
     const int nseg = (a.T + a.seg_len - 1) / a.seg_len, cy = (a.dimp + CB - 1) / CB;
     if (nseg > 1) {
-        if (int r = st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, true>, dim3(a.heads, cy, nseg - 1), dim3(NT), smem, cfg, a)) return r;
+        if (int r = st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, true>, dim3(a.heads, cy, nseg - 1), dim3(NT), smem2, cfg, a, m)) return r;
         if (int r = st_launch(time_mix_join_kernel, dim3((unsigned)(((size_t)a.heads * a.dimp * a.dimp / 4 + 255) / 256)), dim3(256), 0, cfg, a, nseg)) return r;
     }
-    return st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, false>, dim3(a.heads, cy, nseg), dim3(NT), smem, cfg, a);
+    return st_launch(time_mix_scan_kernel<LPC, NV, NC, CB, false>, dim3(a.heads, cy, nseg), dim3(NT), smem, cfg, a, m);
 }
 // Segments of a portion: as many as fill the SMs with a few CTAs each, none shorter than 128 tokens.
 int time_mix_segment(int heads, int dimp, int T, int sm_count) {
@@ -169,7 +153,7 @@ int time_mix_segment(int heads, int dimp, int T, int sm_count) {
     return n < 2 ? T : (T + n - 1) / n;
 }
 int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg) {
-    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.ld % 4 || a.ldz % 4 || a.seg_len < 1 || (a.seg_len < a.T && (!a.seg_state || !a.seg_decay))) return (int)cudaErrorInvalidValue;
+    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.ld % 4 || a.ldw % 4 || a.ldo % 4 || a.seg_len < 1 || (a.seg_len < a.T && (!a.seg_state || !a.seg_decay))) return (int)cudaErrorInvalidValue;
 #define GO(L, N) tm_go<L, N>(a, cfg)
     return RECUR_DISPATCH(a.dimp, GO);
 #undef GO

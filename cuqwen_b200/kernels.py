@@ -134,7 +134,7 @@ def capture_replay(replays: int, device=0) -> float:
 
 
 # ---- kernels of the layer-list designs (act: 0 bfloat16, 1 float32 activations) ----
-LIN_F32, LIN_ACT, LIN_RELU2, LIN_ADD, LIN_GELU_SIDE, LIN_CAP, LIN_GLU = range(7)
+LIN_F32, LIN_ACT, LIN_RELU2, LIN_ADD, LIN_GELU_SIDE, LIN_CAP, LIN_GLU, LIN_DECAY = range(8)
 
 
 def linear(act, epi, x, ldx, w, pitch, cols, n_tokens, rows, out, ldo, second=None, side=None, device=0):
