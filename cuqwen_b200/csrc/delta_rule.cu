@@ -2,8 +2,8 @@
 // state before the token,   u = beta (v - g S^T k),   o = g S^T q + (k . q) u,   S <- g S + k u^T,   so that both products read
 // the same state and one round of sums serves them.
 //
-// Portions: the row kernel applies the convolutions, silu and unit norms and the heads' decays and step sizes; the scan walks
-// the tokens as time_mix.cu's does.
+// Portions: the row kernel applies the convolutions, silu and unit norms and prepares the heads' decays, step sizes and the products of
+// keys and queries among four tokens; the scan walks the tokens four at a time with the state in registers (recur.cuh).
 #include "recur.cuh"
 
 namespace cq {
@@ -21,121 +21,223 @@ __device__ __forceinline__ float delta_conv(const DeltaArgs& a, int t, int pos, 
 }
 __device__ __forceinline__ float delta_decay(const DeltaArgs& a, const float* raw, int h) { return expf(-a.a_exp[h] * softplus_f(__ldcg(raw + a.a_off + h) + a.dt[h])); }
 
-// CTA = row; a warp per key head, query and key together.
-__global__ void __launch_bounds__(256) delta_rows_kernel(const DeltaArgs a) {
-    extern __shared__ float kq_smem[];                  // [kv_heads] k . q
+// CTA = (four tokens, key head): the head's queries and keys and the values of the heads that share it, then everything that the scan wants to
+// know about the four tokens together.  Tokens past the portion's end are zeros that neither decay nor write.
+constexpr int kDrThreads = 128;
+__global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs a) {
+    extern __shared__ __align__(16) float dq_smem[];    // [4][q dimp | k dimp]
+    __shared__ float sums[24];                          // q . q [4], k . k [4], k_i . k_t (6), k_i . q_t (10)
     pdl_launch_dependents(); pdl_wait();
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t;
-    for (int g = warp; g < a.kv_heads; g += 8) {
-        float qq = 0.f, kk = 0.f, kq = 0.f;
-        float* out = a.qk + ((size_t)t * a.kv_heads + g) * 2 * a.dimp;
-        for (int i = lane; i < a.dimp; i += 32) {
-            const float q = delta_conv(a, t, pos, g * a.dimp + i), k = delta_conv(a, t, pos, a.k_off + g * a.dimp + i);
-            qq = fmaf(q, q, qq); kk = fmaf(k, k, kk); kq = fmaf(k, q, kq);
-            out[i] = q; out[a.dimp + i] = k;            // the same lane scales them below
+    const int blk = blockIdx.x, g = blockIdx.y, t0 = blk * 4, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, per = a.heads / a.kv_heads;
+    const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t0, n = min(4, a.T - t0), d2 = 2 * a.dimp;
+    const int uq = a.dimp / 4, units = 2 * uq + per * a.vdimp / 4;
+    for (int u = tid; u < units; u += kDrThreads) {
+        const int ch = u < uq ? g * a.dimp + 4 * u : u < 2 * uq ? a.k_off + g * a.dimp + 4 * (u - uq) : a.v_off + g * per * a.vdimp + 4 * (u - 2 * uq);
+        float4 y[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) y[t] = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int r = -(a.taps - 1); r < n; ++r) {       // r: row of the four that the input belongs to
+            if (pos + r < 0) continue;
+            const float4 x = t0 + r >= 0 ? __ldcg(reinterpret_cast<const float4*>(a.raw + (size_t)(t0 + r) * a.ld + ch)) : *reinterpret_cast<const float4*>(a.ring + (size_t)((pos + r) % a.taps) * a.g_off + ch);
+#pragma unroll
+            for (int t = 0; t < 4; ++t)
+                if (t >= r && t - r < a.taps) {
+                    const float4 w = __ldg(reinterpret_cast<const float4*>(a.conv + (size_t)(a.taps - 1 - (t - r)) * a.g_off + ch));
+                    y[t] = make_float4(fmaf(w.x, x.x, y[t].x), fmaf(w.y, x.y, y[t].y), fmaf(w.z, x.z, y[t].z), fmaf(w.w, x.w, y[t].w));
+                }
         }
-        const float fq = 1.0f / (sqrtf((float)a.dim) * sqrtf(warp_sum(qq) + kUnitEps)), fk = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
-        for (int i = lane; i < a.dimp; i += 32) { out[i] *= fq; out[a.dimp + i] *= fk; }
-        kq = warp_sum(kq);
-        if (lane == 0) kq_smem[g] = kq * fq * fk;
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float4 z = t < n ? make_float4(silu_f(y[t].x), silu_f(y[t].y), silu_f(y[t].z), silu_f(y[t].w)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (u < 2 * uq) reinterpret_cast<float4*>(dq_smem + t * d2)[u] = z;
+            else if (t < n) reinterpret_cast<float4*>(a.v + (size_t)(t0 + t) * a.heads * a.vdimp + (size_t)g * per * a.vdimp)[u - 2 * uq] = z;
+        }
     }
-    for (int c = threadIdx.x; c < a.heads * a.vdimp; c += 256) a.v[(size_t)t * a.heads * a.vdimp + c] = delta_conv(a, t, pos, a.v_off + c);
     __syncthreads();
-    const float* raw = a.raw + (size_t)t * a.ld;
-    for (int h = threadIdx.x; h < a.heads; h += 256)
-        a.sc[(size_t)t * a.heads + h] = make_float4(delta_decay(a, raw, h), sigmoid_f(raw[a.b_off + h]), kq_smem[h / (a.heads / a.kv_heads)], 0.f);
+    for (int i = warp; i < 24; i += kDrThreads / 32) {
+        int p, q;                                       // places in dq_smem of the two vectors
+        if (i < 4) p = q = i * d2;
+        else if (i < 8) p = q = (i - 4) * d2 + a.dimp;
+        else {
+            int j = i < 14 ? i - 8 : i - 14, t = i < 14 ? 1 : 0;
+            while (j >= t + (i < 14 ? 0 : 1)) { j -= t + (i < 14 ? 0 : 1); ++t; }
+            p = j * d2 + a.dimp; q = t * d2 + (i < 14 ? a.dimp : 0);
+        }
+        float s = 0.f;
+        for (int c = lane; c < a.dimp; c += 32) s = fmaf(dq_smem[p + c], dq_smem[q + c], s);
+        s = warp_sum(s);
+        if (lane == 0) sums[i] = s;
+    }
+    __syncthreads();
+    float fq[4], fk[4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t) { fq[t] = 1.0f / (sqrtf((float)a.dim) * sqrtf(sums[t] + kUnitEps)); fk[t] = 1.0f / sqrtf(sums[4 + t] + kUnitEps); }
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+        for (int c = tid; c < d2 / 4; c += kDrThreads) {
+            if (t >= n) break;
+            float4 z = reinterpret_cast<const float4*>(dq_smem + t * d2)[c];
+            const float f = c < uq ? fq[t] : fk[t];
+            z = make_float4(z.x * f, z.y * f, z.z * f, z.w * f);
+            reinterpret_cast<float4*>(a.qk + ((size_t)(t0 + t) * a.kv_heads + g) * d2)[c] = z;
+        }
+    for (int j = tid; j < per; j += kDrThreads) {
+        const int h = g * per + j;
+        float dec[4], out[kDeltaBlock];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float* raw = a.raw + (size_t)(t0 + t) * a.ld;
+            dec[t] = t < n ? delta_decay(a, raw, h) : 1.f;
+            out[4 + t] = t < n ? sigmoid_f(__ldcg(raw + a.b_off + h)) : 0.f;
+            out[t] = t ? out[t - 1] * dec[t] : dec[t];
+        }
+        int ia = 8, ib = 14;
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+            for (int i = 0; i <= t; ++i) {
+                float f = 1.f;                          // decay from behind token i to token t
+#pragma unroll
+                for (int q = i + 1; q <= t; ++q) f *= dec[q];
+                if (i < t) { out[ia] = f * sums[ia] * fk[i] * fk[t]; ++ia; }
+                out[ib] = f * sums[ib] * fk[i] * fq[t]; ++ib;
+                if (t == 3) out[24 + i] = f;
+            }
+        float* dst = a.sc + ((size_t)blk * a.heads + h) * kDeltaBlock;
+#pragma unroll
+        for (int i = 0; i < 28; ++i) dst[i] = out[i];
+    }
 }
 int launch_delta_rows(const DeltaArgs& a, const LaunchCfg& cfg) {
-    if (a.T < 1 || a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.taps < 1 || a.kv_heads > 8192) return (int)cudaErrorInvalidValue;
-    return st_launch(delta_rows_kernel, dim3(a.T), dim3(256), (size_t)a.kv_heads * 4, cfg, a);
+    if (a.T < 1 || a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.taps < 1 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.vdimp % 8 || a.ld % 4) return (int)cudaErrorInvalidValue;
+    return st_launch(delta_rows_kernel, dim3((a.T + 3) / 4, a.kv_heads), dim3(kDrThreads), (size_t)8 * a.dimp * 4, cfg, a);
 }
 
-constexpr int kDrTile = 16;                             // tokens brought at a time
-// CTA: head x CB value channels, NC of them to a thread.
+struct DeltaTmaps { CUtensorMap qk, v, sc; };
+// CTA: head x CB value channels, NC of them to a thread; four tokens at a time: their products with the state before them are summed over the
+// lanes together, the four corrections follow from the pair products of delta_rows, and the state takes one decay and four updates.
 template <int LPC, int NV, int NC, int CB>
-__global__ void __launch_bounds__(CB / NC * LPC) delta_scan_kernel(const DeltaArgs a) {
-    constexpr int D = LPC * NV * 4, NT = CB / NC * LPC, ROW = 2 * D + CB + 4;            // q | k | v | scalars
-    extern __shared__ __align__(16) float dr_smem[];    // [2][kDrTile][ROW]
+__global__ void __launch_bounds__(CB / NC * LPC) delta_scan_kernel(const DeltaArgs a, const __grid_constant__ DeltaTmaps m) {
+    constexpr int D = LPC * NV * 4, SC = kRecurTile / 4 * kDeltaBlock, STAGE = kRecurTile * (2 * D + CB) + SC;       // q | k | v | block scalars
+    static_assert(NC == 2, "a thread's channels are one 8-byte unit of a value row");
+    extern __shared__ __align__(128) float dr_smem[];   // [2][STAGE]
+    __shared__ __align__(8) unsigned long long bars[2];
+    const uint32_t bar = smem_u32(bars), sm0 = smem_u32(dr_smem);
+    const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), c0 = blockIdx.y * CB, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC, c = c0 + cg * NC;
+    if (tid == 0) { mbar_init(bar, 1); mbar_init(bar + 8, 1); mbar_fence_init(); }
     pdl_launch_dependents(); pdl_wait();
-    const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), c0 = blockIdx.y * CB, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC;
-    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0, nc = min(CB, a.vdimp - c0);
-    for (int i = tid; i < 2 * kDrTile * ROW; i += NT) dr_smem[i] = 0.f;
     __syncthreads();
-    auto bring = [&](int t0, int b) {
-        const int n = min(kDrTile, a.T - t0), du = a.dimp / 4, cu = nc / 4, per = 2 * du + cu + 1;
-        for (int i = tid; i < n * per; i += NT) {
-            const int t = i / per, u = i - t * per, tt = t0 + t;
-            float* dst = dr_smem + (b * kDrTile + t) * ROW;
-            if (u < 2 * du) cp_async16(dst + (u < du ? 4 * u : D + 4 * (u - du)), a.qk + ((size_t)tt * a.kv_heads + g) * 2 * a.dimp + 4 * u);
-            else if (u < 2 * du + cu) cp_async16(dst + 2 * D + 4 * (u - 2 * du), a.v + ((size_t)tt * a.heads + h) * a.vdimp + c0 + 4 * (u - 2 * du));
-            else cp_async16(dst + 2 * D + CB, a.sc + (size_t)tt * a.heads + h);
-        }
-        cp_async_commit();
+    const int first = a.pos_ptr ? *a.pos_ptr : a.pos0;
+    auto bring = [&](int t, int b) {
+        const uint32_t dst = sm0 + b * STAGE * 4, fb = bar + 8 * b;
+        mbar_expect_tx(fb, STAGE * 4);
+        recur_load<D>(dst, &m.qk, 0, 2 * g, t, fb); recur_load<D>(dst + kRecurTile * D * 4, &m.qk, 0, 2 * g + 1, t, fb);
+        tma_load_3d(dst + 2 * kRecurTile * D * 4, &m.v, c0, h, t, fb);
+        tma_load_3d(dst + kRecurTile * (2 * D + CB) * 4, &m.sc, 0, h, t / 4, fb);
     };
-    bring(0, 0);
+    if (tid == 0) { bring(0, 0); if (kRecurTile < a.T) bring(kRecurTile, 1); }
     StateCol<LPC, NV> s[NC];
-    float* st[NC];
+    float* st = a.state + ((size_t)h * a.vdimp + c) * a.dimp;         // vdimp is a multiple of eight: both channels exist or none
 #pragma unroll
-    for (int j = 0; j < NC; ++j) {
-        const int c = c0 + cg * NC + j;
-        st[j] = a.state + ((size_t)h * a.vdimp + c) * a.dimp;
-        if (c < a.vdimp && first > 0) s[j].load(st[j], l, a.dimp); else s[j].zero();
-    }
-    for (int t0 = 0, b = 0; t0 < a.T; t0 += kDrTile, b ^= 1) {
-        if (t0 + kDrTile < a.T) { bring(t0 + kDrTile, b ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
-        __syncthreads();
-        const int n = min(kDrTile, a.T - t0);
+    for (int j = 0; j < NC; ++j) if (c < a.vdimp && first > 0) s[j].load(st + j * a.dimp, l, a.dimp); else s[j].zero();
+    bool failed = false;
+    for (int t0 = 0, i = 0; t0 < a.T; t0 += kRecurTile, ++i) {
+        const int b = i & 1;
+        if (!failed && !mbar_wait(bar + 8 * b, (uint32_t)(i >> 1) & 1u)) { failed = true; if (a.err) atomicExch(a.err, 22u); }
+        const float *qb = dr_smem + b * STAGE, *kb = qb + kRecurTile * D, *vb = kb + kRecurTile * D, *cb = vb + kRecurTile * CB;
+        const int n = min(kRecurTile, a.T - t0);
 #pragma unroll 1
-        for (int t = 0; t < n; ++t) {
-            const float* row = dr_smem + (b * kDrTile + t) * ROW;
-            f32x2 q[2 * NV], k[2 * NV];
-            lane_units<LPC, NV>(row, l, q); lane_units<LPC, NV>(row + D, l, k);
-            const float4 sc = *reinterpret_cast<const float4*>(row + 2 * D + CB);
-            const f32x2 g2 = pack2(sc.x, sc.x);
-            float sk[NC], sq[NC];
+        for (int tb = 0; tb < n; tb += 4) {
+            f32x2 k[4][2 * NV];
+            float sk[4][NC], sq[4][NC];
 #pragma unroll
-            for (int j = 0; j < NC; ++j) {
-                f32x2 k0 = 0ull, k1 = 0ull, q0 = 0ull, q1 = 0ull;
+            for (int t = 0; t < 4; ++t) {
+                f32x2 q[2 * NV];
+                lane_row<LPC, NV>(kb, tb + t, l, k[t]); lane_row<LPC, NV>(qb, tb + t, l, q);
 #pragma unroll
-                for (int i = 0; i < 2 * NV; i += 2) {
-                    k0 = fma2(s[j].s[i], k[i], k0); k1 = fma2(s[j].s[i + 1], k[i + 1], k1);
-                    q0 = fma2(s[j].s[i], q[i], q0); q1 = fma2(s[j].s[i + 1], q[i + 1], q1);
+                for (int j = 0; j < NC; ++j) {
+                    f32x2 ka = mul2(s[j].s[0], k[t][0]), qa = mul2(s[j].s[0], q[0]);
+#pragma unroll
+                    for (int x = 1; x < 2 * NV; ++x) { ka = fma2(s[j].s[x], k[t][x], ka); qa = fma2(s[j].s[x], q[x], qa); }
+                    sk[t][j] = sum2(ka); sq[t][j] = sum2(qa);
                 }
-                sk[j] = sum2(add2(k0, k1)); sq[j] = sum2(add2(q0, q1));
             }
 #pragma unroll
             for (int o = LPC / 2; o > 0; o >>= 1)
 #pragma unroll
-                for (int j = 0; j < NC; ++j) { sk[j] += __shfl_xor_sync(0xffffffffu, sk[j], o); sq[j] += __shfl_xor_sync(0xffffffffu, sq[j], o); }
+                for (int t = 0; t < 4; ++t)
+#pragma unroll
+                    for (int j = 0; j < NC; ++j) { sk[t][j] += __shfl_xor_sync(0xffffffffu, sk[t][j], o); sq[t][j] += __shfl_xor_sync(0xffffffffu, sq[t][j], o); }
+            float x[kDeltaBlock];
+#pragma unroll
+            for (int q = 0; q < 7; ++q) {
+                const float4 v = reinterpret_cast<const float4*>(cb + (tb >> 2) * kDeltaBlock)[q];
+                x[4 * q] = v.x; x[4 * q + 1] = v.y; x[4 * q + 2] = v.z; x[4 * q + 3] = v.w;
+            }
+            float u[4][NC], o[4][NC];
+            {
+                int ia = 8, ib = 14;
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    const float2 v = *reinterpret_cast<const float2*>(vb + (tb + t) * CB + cg * NC);
+#pragma unroll
+                    for (int j = 0; j < NC; ++j) {
+                        float e = (j ? v.y : v.x) - x[t] * sk[t][j];
+#pragma unroll
+                        for (int p = 0; p < t; ++p) e -= x[ia + p] * u[p][j];
+                        u[t][j] = x[4 + t] * e;
+                        float r = x[t] * sq[t][j];
+#pragma unroll
+                        for (int p = 0; p <= t; ++p) r = fmaf(x[ib + p], u[p][j], r);
+                        o[t][j] = r;
+                    }
+                    ia += t; ib += t + 1;
+                }
+            }
+            const f32x2 g2 = pack2(x[3], x[3]);
 #pragma unroll
             for (int j = 0; j < NC; ++j) {
-                const float u = sc.y * (row[2 * D + cg * NC + j] - sc.x * sk[j]), o = fmaf(sc.z, u, sc.x * sq[j]);
-                const f32x2 u2 = pack2(u, u);
+                f32x2 e[4];
 #pragma unroll
-                for (int i = 0; i < 2 * NV; ++i) s[j].s[i] = fma2(s[j].s[i], g2, mul2(k[i], u2));
-                const int c = c0 + cg * NC + j;
-                if (l == 0 && c < a.vdimp) a.o[(size_t)(t0 + t) * a.ldo + (size_t)h * a.vdimp + c] = o;
+                for (int t = 0; t < 4; ++t) { const float f = x[24 + t] * u[t][j]; e[t] = pack2(f, f); }
+#pragma unroll
+                for (int y = 0; y < 2 * NV; ++y) {
+                    f32x2 z = mul2(s[j].s[y], g2);
+#pragma unroll
+                    for (int t = 0; t < 4; ++t) z = fma2(k[t][y], e[t], z);
+                    s[j].s[y] = z;
+                }
+            }
+            // lane t of a channel's first four stores token t
+            if (l < 4 && tb + l < n && c < a.vdimp) {
+                const float2 r = l == 0 ? make_float2(o[0][0], o[0][1]) : l == 1 ? make_float2(o[1][0], o[1][1]) : l == 2 ? make_float2(o[2][0], o[2][1]) : make_float2(o[3][0], o[3][1]);
+                *reinterpret_cast<float2*>(a.o + (size_t)(t0 + tb + l) * a.ldo + (size_t)h * a.vdimp + c) = r;
             }
         }
         __syncthreads();
+        if (tid == 0 && t0 + 2 * kRecurTile < a.T) bring(t0 + 2 * kRecurTile, b);
     }
 #pragma unroll
-    for (int j = 0; j < NC; ++j) if (c0 + cg * NC + j < a.vdimp) s[j].store(st[j], l, a.dimp);
+    for (int j = 0; j < NC; ++j) if (c < a.vdimp) s[j].store(st + j * a.dimp, l, a.dimp);
 }
 template <int LPC, int NV>
 static int dr_go(const DeltaArgs& a, const LaunchCfg& cfg) {
     constexpr int NC = 2, CB = 32, D = LPC * NV * 4;
-    const size_t smem = (size_t)2 * kDrTile * (2 * D + CB + 4) * 4;
+    const size_t smem = (size_t)2 * (kRecurTile * (2 * D + CB) + kRecurTile / 4 * kDeltaBlock) * 4;
     static bool once = false;
     if (!once) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<LPC, NV, NC, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<LPC, NV, NC, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
         if (e != cudaSuccess) return (int)e;
         once = true;
     }
-    return st_launch(delta_scan_kernel<LPC, NV, NC, CB>, dim3(a.heads, (a.vdimp + CB - 1) / CB), dim3(CB / NC * LPC), smem, cfg, a);
+    DeltaTmaps m;
+    if (int r = recur_map(&m.qk, a.qk, a.dimp, 2 * a.kv_heads, a.dimp, a.T, 2 * a.kv_heads * a.dimp, recur_box(D), kRecurTile)) return r;
+    if (int r = recur_map(&m.v, a.v, a.vdimp, a.heads, a.vdimp, a.T, a.heads * a.vdimp, CB, kRecurTile)) return r;
+    if (int r = recur_map(&m.sc, a.sc, kDeltaBlock, a.heads, kDeltaBlock, (a.T + 3) / 4, a.heads * kDeltaBlock, kDeltaBlock, kRecurTile / 4)) return r;
+    return st_launch(delta_scan_kernel<LPC, NV, NC, CB>, dim3(a.heads, (a.vdimp + CB - 1) / CB), dim3(CB / NC * LPC), smem, cfg, a, m);
 }
 int launch_delta_scan(const DeltaArgs& a, const LaunchCfg& cfg) {
-    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.vdimp % 8) return (int)cudaErrorInvalidValue;
+    if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.vdimp % 8 || a.ldo % 4) return (int)cudaErrorInvalidValue;
 #define GO(L, N) dr_go<L, N>(a, cfg)
     return RECUR_DISPATCH(a.dimp, GO);
 #undef GO

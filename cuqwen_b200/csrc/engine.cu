@@ -1507,7 +1507,7 @@ extern "C" int cuqwen_k_delta(int device, const float* raw, const float* conv, i
     NOT_NULL(raw, conv, ring, a_exp, dt, qk, v, sc, state, o);
     if (!delta_ok(heads, kv_heads, dim, vdim, taps) || n_tokens < 1 || pos0 < 0) return fail(CUQWEN_ERR_ARG, "delta: lengths are multiples of 8, dim at most %d", kRecurMaxDim);
     DeltaArgs a = delta_args(raw, conv, taps, ring, a_exp, dt, state, heads, kv_heads, dim, vdim);
-    a.qk = qk; a.v = v; a.sc = (float4*)sc; a.o = o; a.T = n_tokens; a.pos0 = pos0;
+    a.qk = qk; a.v = v; a.sc = sc; a.o = o; a.err = t_err; a.T = n_tokens; a.pos0 = pos0;
     KK(launch_delta_rows(a, cfg));
     const TailRowsArgs t{raw, a.ld, n_tokens, ring, a.g_off, a.g_off, taps, taps - 1, nullptr, pos0};
     if (taps > 1) KK(launch_tail_rows(t, cfg));

@@ -45,7 +45,7 @@ static int alloc_ws(Stack* s, Stack::Ws* w, int rows, bool decode) {
         w->sg = a.get(R * (s->sidep ? s->sidep : 8) * E);
         if (s->spec.recurrent()) {
             w->z = (float*)a.get(R * s->max_z * 4); w->zin = a.get(2 * R * s->max_rank * E); w->qk = (float*)a.get(R * s->max_qk * 4); w->vv = (float*)a.get(R * s->max_vv * 4);
-            w->ro = (float*)a.get(R * s->max_ro * 4); w->att2 = a.get(R * s->max_ro * E); w->sc = (float4*)a.get(R * s->max_sc * 16); w->tail = (float*)a.get((size_t)s->wp * 4);
+            w->ro = (float*)a.get(R * s->max_ro * 4); w->att2 = a.get(R * s->max_ro * E); w->sc = (float*)a.get((R + 3) / 4 * s->max_sc * kDeltaBlock * 4); w->tail = (float*)a.get((size_t)s->wp * 4);
             if (!decode) { w->seg_state = (float*)a.get((size_t)kTmMaxSeg * s->max_tm_state * 4); w->seg_decay = (float*)a.get((size_t)kTmMaxSeg * s->max_z * 4); }
         }
         if (decode) {
@@ -113,7 +113,7 @@ int stack_create(cuqwen_engine* e, const StackSpec& spec, int act, int max_seq_l
             for (int i = 2; i < 6; ++i) l.in_off[i] = l.in_off[i - 1] + rw;
             l.ldraw = l.in_off[5] + l.rankp;
             l.kv_off = room((size_t)g.kv_heads * max_seq_len * l.crow * s->esz); l.state_off = room((size_t)rw * l.rdimp * 4); l.ring_off = room((size_t)2 * s->wp * 4);
-            up(s->max_q, g.heads * l.dimp); up(s->max_att, g.heads * l.vdimp); up(s->max_var, 6); up(s->max_z, rw); up(s->max_rank, l.rankp); up(s->max_ro, rw); up(s->max_sc, t.heads); up(s->max_tm_state, rw * l.rdimp);
+            up(s->max_q, g.heads * l.dimp); up(s->max_att, g.heads * l.vdimp); up(s->max_var, 6); up(s->max_z, rw); up(s->max_rank, l.rankp); up(s->max_ro, rw); up(s->max_tm_state, rw * l.rdimp);
             up(s->max_kvr, g.heads * l.vdimp); up(s->max_heads, g.heads);
             if (act == ACT_BF16) l.nsplit = grouped_decode_splits(g.heads, g.kv_heads, l.dimp, l.vdimp, max_seq_len, e->sms);
         } else {

@@ -194,15 +194,18 @@ struct TimeMixStepArgs {
 int launch_time_mix_step(const TimeMixStepArgs& a, const LaunchCfg& cfg);
 
 // Gated delta rule (delta_rule.cu).  State [heads][vdimp][dimp]; ring [taps][channels]: raw projections by position.
-// delta_rows: convolution, silu, unit vectors; per value head decay and step size.
+// delta_rows: convolution, silu, unit vectors; per value head and block of four tokens (kDeltaBlock floats) decays up to each token [4], step
+// sizes [4], decayed k_i . k_t of i < t [6] and k_i . q_t of i <= t [10], decays from each token to the last [4].
+constexpr int kDeltaBlock = 32;
 struct DeltaArgs {
     const float* raw; int ld, k_off, v_off, g_off, a_off, b_off;    // raw rows [q | k | v | g | a | b]
     const float* conv; int taps; float* ring;                       // conv [taps][channels], channels = g_off
     const float *a_exp, *dt;                                        // exp(A_log), dt_bias [heads]
     int heads, kv_heads, dim, dimp, vdim, vdimp, T;
-    float* qk; float* v; float4* sc;                                // [T][kv_heads][q dimp | k dimp], [T][heads * vdimp], [T][heads] (decay, step, k . q, -)
+    float *qk, *v, *sc;                                             // [T][kv_heads][q dimp | k dimp], [T][heads * vdimp], [blocks][heads][kDeltaBlock]
     float* state; float* o; int ldo;
     const int* pos_ptr; int pos0;
+    unsigned* err;
 };
 int launch_delta_rows(const DeltaArgs& a, const LaunchCfg& cfg);
 int launch_delta_scan(const DeltaArgs& a, const LaunchCfg& cfg);

@@ -32,7 +32,7 @@ DeltaArgs Pass::delta(const StLayer& l) {
     a.raw = w->raw; a.ld = l.ldraw; a.k_off = l.k_off; a.v_off = l.v_off; a.g_off = l.g_off; a.a_off = l.a_off; a.b_off = l.b_off;
     a.conv = l.conv; a.taps = d.conv; a.ring = (float*)at(l.ring_off); a.a_exp = l.a_exp; a.dt = l.dt;
     a.heads = d.heads; a.kv_heads = d.kv_heads; a.dim = d.dim; a.dimp = l.dimp; a.vdim = d.vdim; a.vdimp = l.vdimp; a.T = T;
-    a.qk = w->qk; a.v = w->vv; a.sc = w->sc; a.state = (float*)at(l.state_off); a.o = w->ro; a.ldo = d.heads * l.vdimp; a.pos_ptr = pos_ptr; a.pos0 = pos0;
+    a.qk = w->qk; a.v = w->vv; a.sc = w->sc; a.state = (float*)at(l.state_off); a.o = w->ro; a.ldo = d.heads * l.vdimp; a.err = err_word(); a.pos_ptr = pos_ptr; a.pos0 = pos0;
     return a;
 }
 

@@ -59,7 +59,7 @@ struct Stack {
     struct Ws {
         int rows = 0, kv_rows = 0;
         float *x = nullptr, *x2 = nullptr, *raw = nullptr, *qf = nullptr, *y = nullptr, *o_lat = nullptr, *part_o = nullptr, *part_ml = nullptr;
-        float *z = nullptr, *qk = nullptr, *vv = nullptr, *ro = nullptr, *tail = nullptr; float *seg_state = nullptr, *seg_decay = nullptr; float4* sc = nullptr;      // recurrences: segments of a portion, decays, convolution outputs, read-outs, head scalars
+        float *z = nullptr, *qk = nullptr, *vv = nullptr, *ro = nullptr, *tail = nullptr; float *seg_state = nullptr, *seg_decay = nullptr, *sc = nullptr;      // recurrences: segments of a portion, decays, convolution outputs, read-outs, head scalars
         void *zin = nullptr, *att2 = nullptr;
         void *xn1 = nullptr, *xn2 = nullptr, *cq = nullptr, *q = nullptr, *att = nullptr, *h = nullptr, *sg = nullptr, *kv = nullptr;
         uint8_t* arena = nullptr;

@@ -325,7 +325,7 @@ int cuqwen_k_time_mix(int device, const float* r, const float* k, const float* v
 /* One token: raw [r | k | v | g, heads x dim each | w1 product, rank]; decay through w2 [heads * dim][w2_pitch]; out = o / rms(o) * norm * silu(g) * scale (bfloat16). */
 int cuqwen_k_time_mix_step(int device, const float* raw, const void* w2, int w2_pitch, int rank, const float* w0, const float* u, const float* norm, float* state, void* out, int heads, int dim, float eps, float scale, const int* d_pos);
 /* Gated delta rule of a portion in float32: raw rows [q, k: kv_heads x dim | v, g: heads x vdim | a, b: heads rounded up to eight]; conv [taps][q | k | v channels], last tap
- * = current token; ring [taps][channels] raw rows by position; a_exp = exp(A_log); qk [t][kv_heads][2 dim], v [t][heads * vdim], sc [t][heads][4] scratch; state
+ * = current token; ring [taps][channels] raw rows by position; a_exp = exp(A_log); qk [t][kv_heads][2 dim], v [t][heads * vdim], sc [t / 4][heads][32] scratch; state
  * [heads][value][key]; o [t][heads][vdim] before norm and gate. */
 int cuqwen_k_delta(int device, const float* raw, const float* conv, int taps, float* ring, const float* a_exp, const float* dt, float* qk, float* v, float* sc, float* state, float* o, int heads, int kv_heads, int dim, int vdim, int n_tokens, int pos0);
 /* One token of the same, with o / rms(o) * norm * silu(g) (bfloat16). */

@@ -209,7 +209,7 @@ def test_gated_delta_rule(built, heads, kv, dim, vd, taps, n):
         pool, state, ring, got = Pool(), dev(np.full(heads * vd * dim, 3.0, np.float32)), dev(np.full((taps, ch), 5.0, np.float32)), []
         for i, m in pieces(n, sizes):
             o = E.DevBuf(m * heads * vd * 4)
-            K.delta(pool.p(raw[i:i + m].copy()), pool.p(conv), taps, ring, pool.p(a_exp), pool.p(dt), E.DevBuf(m * kv * 2 * dim * 4), E.DevBuf(m * heads * vd * 4), E.DevBuf(m * heads * 16), state, o, heads, kv, dim, vd, m, i)
+            K.delta(pool.p(raw[i:i + m].copy()), pool.p(conv), taps, ring, pool.p(a_exp), pool.p(dt), E.DevBuf(m * kv * 2 * dim * 4), E.DevBuf(m * heads * vd * 4), E.DevBuf((m + 3) // 4 * heads * 128), state, o, heads, kv, dim, vd, m, i)
             E.sync()
             got.append(o.numpy(np.float32).reshape(m, heads, vd))
         near(np.concatenate(got).astype(np.float64), want, "float32", 4.0)
