@@ -24,6 +24,7 @@ __device__ __forceinline__ float delta_decay(const DeltaArgs& a, const float* ra
 // CTA = (four tokens, key head): the head's queries and keys and the values of the heads that share it, then everything that the scan wants to
 // know about the four tokens together.  Tokens past the portion's end are zeros that neither decay nor write.
 constexpr int kDrThreads = 128;
+template <int TAPS>                                     // 0: any number
 __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs a) {
     extern __shared__ __align__(16) float dq_smem[];    // [4][q dimp | k dimp]
     __shared__ float sums[24];                          // q . q [4], k . k [4], k_i . k_t (6), k_i . q_t (10)
@@ -31,21 +32,46 @@ __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs 
     const int blk = blockIdx.x, g = blockIdx.y, t0 = blk * 4, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, per = a.heads / a.kv_heads;
     const int pos = (a.pos_ptr ? *a.pos_ptr : a.pos0) + t0, n = min(4, a.T - t0), d2 = 2 * a.dimp;
     const int uq = a.dimp / 4, units = 2 * uq + per * a.vdimp / 4;
+    // the decays and step sizes of the group's heads, by the last warp while the others begin with the convolutions
+    __shared__ float dec_s[4][32], step_s[4][32];
+    auto scalars = [&](int j0) {
+        for (int i = 127 - tid; i < 4 * 32; i += kDrThreads) {
+            const int t = i >> 5, j = j0 + (i & 31);
+            if (j < per) {
+                const float* raw = a.raw + (size_t)(t0 + t) * a.ld;
+                dec_s[t][i & 31] = t < n ? delta_decay(a, raw, g * per + j) : 1.f;
+                step_s[t][i & 31] = t < n ? sigmoid_f(__ldcg(raw + a.b_off + g * per + j)) : 0.f;
+            }
+        }
+    };
+    scalars(0);
     for (int u = tid; u < units; u += kDrThreads) {
         const int ch = u < uq ? g * a.dimp + 4 * u : u < 2 * uq ? a.k_off + g * a.dimp + 4 * (u - uq) : a.v_off + g * per * a.vdimp + 4 * (u - 2 * uq);
         float4 y[4];
 #pragma unroll
         for (int t = 0; t < 4; ++t) y[t] = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int r = -(a.taps - 1); r < n; ++r) {       // r: row of the four that the input belongs to
-            if (pos + r < 0) continue;
-            const float4 x = t0 + r >= 0 ? __ldcg(reinterpret_cast<const float4*>(a.raw + (size_t)(t0 + r) * a.ld + ch)) : *reinterpret_cast<const float4*>(a.ring + (size_t)((pos + r) % a.taps) * a.g_off + ch);
+        auto input = [&](int r) {                       // r: row of the four that the input belongs to
+            if (r >= n || pos + r < 0) return make_float4(0.f, 0.f, 0.f, 0.f);
+            return t0 + r >= 0 ? __ldcg(reinterpret_cast<const float4*>(a.raw + (size_t)(t0 + r) * a.ld + ch)) : *reinterpret_cast<const float4*>(a.ring + (size_t)((pos + r) % a.taps) * a.g_off + ch);
+        };
+        auto tap = [&](int t, int j, float4 x) {        // input j rows before token t
+            const float4 w = __ldg(reinterpret_cast<const float4*>(a.conv + (size_t)(a.taps - 1 - j) * a.g_off + ch));
+            y[t] = make_float4(fmaf(w.x, x.x, y[t].x), fmaf(w.y, x.y, y[t].y), fmaf(w.z, x.z, y[t].z), fmaf(w.w, x.w, y[t].w));
+        };
+        if (TAPS > 0) {
+            float4 x[TAPS + 3];
+#pragma unroll
+            for (int r = 0; r < TAPS + 3; ++r) x[r] = input(r - (TAPS - 1));
 #pragma unroll
             for (int t = 0; t < 4; ++t)
-                if (t >= r && t - r < a.taps) {
-                    const float4 w = __ldg(reinterpret_cast<const float4*>(a.conv + (size_t)(a.taps - 1 - (t - r)) * a.g_off + ch));
-                    y[t] = make_float4(fmaf(w.x, x.x, y[t].x), fmaf(w.y, x.y, y[t].y), fmaf(w.z, x.z, y[t].z), fmaf(w.w, x.w, y[t].w));
-                }
-        }
+#pragma unroll
+                for (int j = TAPS - 1; j >= 0; --j) tap(t, j, x[t + TAPS - 1 - j]);
+        } else
+            for (int r = -(a.taps - 1); r < n; ++r) {
+                const float4 x = input(r);
+#pragma unroll
+                for (int t = 0; t < 4; ++t) if (t >= r && t - r < a.taps) tap(t, t - r, x);
+            }
 #pragma unroll
         for (int t = 0; t < 4; ++t) {
             const float4 z = t < n ? make_float4(silu_f(y[t].x), silu_f(y[t].y), silu_f(y[t].z), silu_f(y[t].w)) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -81,14 +107,15 @@ __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs 
             z = make_float4(z.x * f, z.y * f, z.z * f, z.w * f);
             reinterpret_cast<float4*>(a.qk + ((size_t)(t0 + t) * a.kv_heads + g) * d2)[c] = z;
         }
-    for (int j = tid; j < per; j += kDrThreads) {
-        const int h = g * per + j;
+    for (int j0 = 0; j0 < per; j0 += 32) {
+        if (j0) { __syncthreads(); scalars(j0); __syncthreads(); }
+        if (tid >= 32 || j0 + tid >= per) continue;
+        const int h = g * per + j0 + tid;
         float dec[4], out[kDeltaBlock];
 #pragma unroll
         for (int t = 0; t < 4; ++t) {
-            const float* raw = a.raw + (size_t)(t0 + t) * a.ld;
-            dec[t] = t < n ? delta_decay(a, raw, h) : 1.f;
-            out[4 + t] = t < n ? sigmoid_f(__ldcg(raw + a.b_off + h)) : 0.f;
+            dec[t] = dec_s[t][tid];
+            out[4 + t] = step_s[t][tid];
             out[t] = t ? out[t - 1] * dec[t] : dec[t];
         }
         int ia = 8, ib = 14;
@@ -103,14 +130,16 @@ __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs 
                 out[ib] = f * sums[ib] * fk[i] * fq[t]; ++ib;
                 if (t == 3) out[24 + i] = f;
             }
-        float* dst = a.sc + ((size_t)blk * a.heads + h) * kDeltaBlock;
+        float4* dst = reinterpret_cast<float4*>(a.sc + ((size_t)blk * a.heads + h) * kDeltaBlock);
 #pragma unroll
-        for (int i = 0; i < 28; ++i) dst[i] = out[i];
+        for (int i = 0; i < 7; ++i) dst[i] = make_float4(out[4 * i], out[4 * i + 1], out[4 * i + 2], out[4 * i + 3]);
     }
 }
 int launch_delta_rows(const DeltaArgs& a, const LaunchCfg& cfg) {
     if (a.T < 1 || a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.taps < 1 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.vdimp % 8 || a.ld % 4) return (int)cudaErrorInvalidValue;
-    return st_launch(delta_rows_kernel, dim3((a.T + 3) / 4, a.kv_heads), dim3(kDrThreads), (size_t)8 * a.dimp * 4, cfg, a);
+    const dim3 grid((a.T + 3) / 4, a.kv_heads);
+    const size_t smem = (size_t)8 * a.dimp * 4;
+    return a.taps == 4 ? st_launch(delta_rows_kernel<4>, grid, dim3(kDrThreads), smem, cfg, a) : st_launch(delta_rows_kernel<0>, grid, dim3(kDrThreads), smem, cfg, a);
 }
 
 struct DeltaTmaps { CUtensorMap qk, v, sc; };

@@ -89,9 +89,26 @@ int launch_st_glu_rows(int act, const float* raw, int ld, void* out, int ldo, in
                           : st_launch(st_glu_rows_kernel<bf16>, dim3(T), dim3(256), 0, cfg, raw, ld, (bf16*)out, ldo, ff, limit, slope);
 }
 
-// A warp per head, eight heads a CTA.
-template <typename A>
+// Heads of 4 * LP places, LP a power of two: a thread per four places, the LP threads of a head side by side.
+template <typename A, int LP>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs a) {
+    pdl_launch_dependents(); pdl_wait();
+    const int t = blockIdx.x, u = blockIdx.y * 256 + threadIdx.x, h = u / LP, i = u % LP * 4;
+    const bool in = h < a.heads;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f), g = o, w = o;
+    if (in) {
+        o = *reinterpret_cast<const float4*>(a.o + (size_t)t * a.ldo + (size_t)u * 4); g = *reinterpret_cast<const float4*>(a.gate + (size_t)t * a.ldg + (size_t)u * 4);
+        w = *reinterpret_cast<const float4*>(a.w + (size_t)h * a.w_hs + i);
+    }
+    float ss = dot4(o, o);                              // places past a head's length hold zeros
+#pragma unroll
+    for (int d = LP / 2; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+    const float f = inv_rms(ss, a.n, a.eps) * a.scale;
+    if (in) store4(reinterpret_cast<A*>(a.out) + (size_t)t * a.ldout + (size_t)u * 4, make_float4(o.x * f * w.x * silu_f(g.x), o.y * f * w.y * silu_f(g.y), o.z * f * w.z * silu_f(g.z), o.w * f * w.w * silu_f(g.w)));
+}
+// Any length: a warp per head, eight heads a CTA.
+template <typename A>
+__global__ void __launch_bounds__(256) head_norm_gate_any_kernel(const HeadNormArgs a) {
     pdl_launch_dependents(); pdl_wait();
     const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = blockIdx.x;
     if (h >= a.heads) return;
@@ -102,9 +119,19 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
     const float inv = inv_rms(warp_sum(ss), a.n, a.eps) * a.scale;
     for (int i = lane; i < a.np; i += 32) out[i] = to_act<A>(i < a.n ? o[i] * inv * w[i] * silu_f(g[i]) : 0.f);
 }
+template <typename A>
+static int go_head_norm(const HeadNormArgs& a, int T, const LaunchCfg& cfg) {
+    const dim3 grid(T, (a.heads * (a.np / 4) + 255) / 256);
+    switch (a.np) {
+        case 32: return st_launch(head_norm_gate_kernel<A, 8>, grid, dim3(256), 0, cfg, a);
+        case 64: return st_launch(head_norm_gate_kernel<A, 16>, grid, dim3(256), 0, cfg, a);
+        case 128: return st_launch(head_norm_gate_kernel<A, 32>, grid, dim3(256), 0, cfg, a);
+    }
+    return st_launch(head_norm_gate_any_kernel<A>, dim3(T, (a.heads + 7) / 8), dim3(256), 0, cfg, a);
+}
 int launch_head_norm_gate(int act, const HeadNormArgs& a, int T, const LaunchCfg& cfg) {
-    const dim3 grid(T, (a.heads + 7) / 8);
-    return act == ACT_F32 ? st_launch(head_norm_gate_kernel<float>, grid, dim3(256), 0, cfg, a) : st_launch(head_norm_gate_kernel<bf16>, grid, dim3(256), 0, cfg, a);
+    if (T < 1 || a.heads < 1 || a.np % 8 || a.ldo % 4 || a.ldg % 4 || a.ldout % 4) return (int)cudaErrorInvalidValue;
+    return act == ACT_F32 ? go_head_norm<float>(a, T, cfg) : go_head_norm<bf16>(a, T, cfg);
 }
 
 }  // namespace cq
