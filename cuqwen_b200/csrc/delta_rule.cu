@@ -24,6 +24,8 @@ __device__ __forceinline__ float delta_decay(const DeltaArgs& a, const float* ra
 // CTA = (four tokens, key head): the head's queries and keys and the values of the heads that share it, then everything that the scan wants to
 // know about the four tokens together.  Tokens past the portion's end are zeros that neither decay nor write.
 constexpr int kDrThreads = 128;
+// The 24 products: q_t = vector 2 t, k_t = vector 2 t + 1; (first vector) * 8 + second.
+__constant__ unsigned char kDrPairs[24] = {0 * 9, 2 * 9, 4 * 9, 6 * 9, 1 * 9, 3 * 9, 5 * 9, 7 * 9, 8 + 3, 8 + 5, 24 + 5, 8 + 7, 24 + 7, 40 + 7, 8 + 0, 8 + 2, 24 + 2, 8 + 4, 24 + 4, 40 + 4, 8 + 6, 24 + 6, 40 + 6, 56 + 6};
 template <int TAPS>                                     // 0: any number
 __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs a) {
     extern __shared__ __align__(16) float dq_smem[];    // [4][q dimp | k dimp]
@@ -80,19 +82,24 @@ __global__ void __launch_bounds__(kDrThreads) delta_rows_kernel(const DeltaArgs 
         }
     }
     __syncthreads();
-    for (int i = warp; i < 24; i += kDrThreads / 32) {
-        int p, q;                                       // places in dq_smem of the two vectors
-        if (i < 4) p = q = i * d2;
-        else if (i < 8) p = q = (i - 4) * d2 + a.dimp;
-        else {
-            int j = i < 14 ? i - 8 : i - 14, t = i < 14 ? 1 : 0;
-            while (j >= t + (i < 14 ? 0 : 1)) { j -= t + (i < 14 ? 0 : 1); ++t; }
-            p = j * d2 + a.dimp; q = t * d2 + (i < 14 ? a.dimp : 0);
+    {
+        float s[6];
+        int p[6], q[6];                                 // this warp's six products of two of the eight vectors
+#pragma unroll
+        for (int j = 0; j < 6; ++j) {
+            const int e = kDrPairs[warp + 4 * j], x = e >> 3, y = e & 7;
+            p[j] = (x >> 1) * d2 + (x & 1) * a.dimp; q[j] = (y >> 1) * d2 + (y & 1) * a.dimp; s[j] = 0.f;
         }
-        float s = 0.f;
-        for (int c = lane; c < a.dimp; c += 32) s = fmaf(dq_smem[p + c], dq_smem[q + c], s);
-        s = warp_sum(s);
-        if (lane == 0) sums[i] = s;
+        for (int c = lane; c < a.dimp; c += 32)
+#pragma unroll
+            for (int j = 0; j < 6; ++j) s[j] = fmaf(dq_smem[p[j] + c], dq_smem[q[j] + c], s[j]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int j = 0; j < 6; ++j) s[j] += __shfl_xor_sync(0xffffffffu, s[j], o);
+        if (lane == 0)
+#pragma unroll
+            for (int j = 0; j < 6; ++j) sums[warp + 4 * j] = s[j];
     }
     __syncthreads();
     float fq[4], fk[4];

@@ -48,11 +48,11 @@ __device__ __forceinline__ float inv_rms(float sum_sq, int n, float eps) { retur
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
-__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope) {
     g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit);
-    return g * sigmoid_f(slope * g) * (u + 1.0f);
+    return __fdividef(g, 1.0f + expf(-slope * g)) * (u + 1.0f);
 }
 
 // Two float32 lanes in one 64-bit register.
