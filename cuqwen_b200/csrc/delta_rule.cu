@@ -256,9 +256,9 @@ __global__ void __launch_bounds__(CB / NC * LPC) delta_scan_kernel(const DeltaAr
 #pragma unroll
     for (int j = 0; j < NC; ++j) if (c < a.vdimp) s[j].store(st + j * a.dimp, l, a.dimp);
 }
-template <int LPC, int NV>
-static int dr_go(const DeltaArgs& a, const LaunchCfg& cfg) {
-    constexpr int NC = 2, CB = 32, D = LPC * NV * 4;
+template <int LPC, int NV, int CB>
+static int dr_launch(const DeltaArgs& a, const LaunchCfg& cfg) {
+    constexpr int NC = 2, D = LPC * NV * 4;
     const size_t smem = (size_t)2 * (kRecurTile * (2 * D + CB) + kRecurTile / 4 * kDeltaBlock) * 4;
     static bool once = false;
     if (!once) {
@@ -271,6 +271,12 @@ static int dr_go(const DeltaArgs& a, const LaunchCfg& cfg) {
     if (int r = recur_map(&m.v, a.v, a.vdimp, a.heads, a.vdimp, a.T, a.heads * a.vdimp, CB, kRecurTile)) return r;
     if (int r = recur_map(&m.sc, a.sc, kDeltaBlock, a.heads, kDeltaBlock, (a.T + 3) / 4, a.heads * kDeltaBlock, kDeltaBlock, kRecurTile / 4)) return r;
     return st_launch(delta_scan_kernel<LPC, NV, NC, CB>, dim3(a.heads, (a.vdimp + CB - 1) / CB), dim3(CB / NC * LPC), smem, cfg, a, m);
+}
+// The tokens' operands pass through an SM's shared memory once for every CTA there: few heads are cut finer, so that a CTA has an SM to itself.
+template <int LPC, int NV>
+static int dr_go(const DeltaArgs& a, const LaunchCfg& cfg) {
+    if (a.heads * ((a.vdimp + 15) / 16) <= cfg.sm_count) return dr_launch<LPC, NV, 16>(a, cfg);
+    return dr_launch<LPC, NV, 32>(a, cfg);
 }
 int launch_delta_scan(const DeltaArgs& a, const LaunchCfg& cfg) {
     if (a.T < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.vdimp % 8 || a.ldo % 4) return (int)cudaErrorInvalidValue;
