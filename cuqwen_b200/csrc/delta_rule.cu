@@ -10,15 +10,6 @@ namespace cq {
 
 constexpr float kUnitEps = 1e-6f;                       // added to the sum of squares of a unit vector
 
-// One channel's convolution and silu at row t (position pos): earlier rows of the portion, before them the ring.
-__device__ __forceinline__ float delta_conv(const DeltaArgs& a, int t, int pos, int ch) {
-    float s = 0.f;
-    for (int j = 0; j < a.taps && j <= pos; ++j) {      // j rows back
-        const float x = t - j >= 0 ? __ldcg(a.raw + (size_t)(t - j) * a.ld + ch) : a.ring[(size_t)((pos - j) % a.taps) * a.g_off + ch];
-        s = fmaf(a.conv[(size_t)(a.taps - 1 - j) * a.g_off + ch], x, s);
-    }
-    return silu_f(s);
-}
 __device__ __forceinline__ float delta_decay(const DeltaArgs& a, const float* raw, int h) { return expf(-a.a_exp[h] * softplus_f(__ldcg(raw + a.a_off + h) + a.dt[h])); }
 
 // CTA = (four tokens, key head): the head's queries and keys and the values of the heads that share it, then everything that the scan wants to
@@ -286,87 +277,98 @@ int launch_delta_scan(const DeltaArgs& a, const LaunchCfg& cfg) {
 }
 
 // ---- one token --------------------------------------------------------------------------------------------------------
-// CTA = value head.  The state of the first value channels is on its way before the dependency wait (it was written by an earlier
-// step), and so are the ring's rows.  A key head's ring row is written by the first of the value heads that share it.
-constexpr int kDsThreads = 512, kDsHold = 2;            // channels of a thread held at a time
+// A cluster per value head.  On their way before the dependency wait, as earlier steps wrote them: the state of a CTA's first value channels,
+// and the part of the convolutions that earlier tokens make.  A key head's ring row is written by the first of the value heads that share it.
+constexpr int kDsHold = 2;                              // convolution channels of a thread that are begun before the wait
 template <int LPC, int NV>
-__global__ void __launch_bounds__(kDsThreads) delta_step_kernel(const DeltaStepArgs sa) {
-    constexpr int D = LPC * NV * 4, CH = kDsThreads / LPC;                               // value channels at a time
-    extern __shared__ __align__(16) float ds_smem[];    // q [D], k [D], v [vdimp], o [vdimp]
-    __shared__ float red[40];
+__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaStepArgs sa, const StepSplit sp) {
+    constexpr int D = LPC * NV * 4, CH = kStepThreads / LPC;
+    extern __shared__ __align__(16) float ds_smem[];    // q [D], k [D], v [cw], o [cw]
+    __shared__ float red[8], slots[8], sc[8];
     const DeltaArgs& a = sa.d;
     pdl_launch_dependents();
-    const int h = blockIdx.x, per = a.heads / a.kv_heads, g = h / per, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC, pos = *a.pos_ptr;
-    float *q = ds_smem, *k = q + D, *v = k + D, *o = v + a.vdimp;
-    StateCol<LPC, NV> s[kDsHold];
-    auto fetch = [&](int c0) {
-#pragma unroll
-        for (int j = 0; j < kDsHold; ++j) {
-            const int c = c0 + j * CH + cg;
-            if (c < a.vdimp && pos > 0) s[j].load(a.state + ((size_t)h * a.vdimp + c) * a.dimp, l, a.dimp); else s[j].zero();
-        }
+    const int h = blockIdx.x, rank = blockIdx.y, per = a.heads / a.kv_heads, g = h / per, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = tid % LPC, cg = tid / LPC, pos = *a.pos_ptr;
+    const int c0 = rank * sp.cw, cw = min(sp.cw, a.vdimp - c0);
+    float *q = ds_smem, *k = q + D, *v = k + D, *o = v + sp.cw;
+    if (sp.ncl > 1) cluster_arrive();
+    StateCol<LPC, NV> s;
+    auto fetch = [&](int c) { if (c < cw && pos > 0) s.load(a.state + ((size_t)h * a.vdimp + c0 + c) * a.dimp, l, a.dimp); else s.zero(); };
+    fetch(cg);
+    const int items = 2 * a.dimp + cw;                  // channels of the head's query, its key, and this CTA's values
+    auto channel = [&](int i) { return i < a.dimp ? g * a.dimp + i : i < 2 * a.dimp ? a.k_off + g * a.dimp + i - a.dimp : a.v_off + h * a.vdimp + c0 + i - 2 * a.dimp; };
+    auto before = [&](int ch) {
+        float y = 0.f;
+        for (int j = 1; j < a.taps && j <= pos; ++j) y = fmaf(a.conv[(size_t)(a.taps - 1 - j) * a.g_off + ch], a.ring[(size_t)((pos - j) % a.taps) * a.g_off + ch], y);
+        return y;
     };
-    fetch(0);
+    float early[kDsHold], tap[kDsHold];
+#pragma unroll
+    for (int x = 0; x < kDsHold; ++x) {
+        const int i = tid + x * kStepThreads;
+        early[x] = tap[x] = 0.f;
+        if (i < items) { const int ch = channel(i); early[x] = before(ch); tap[x] = a.conv[(size_t)(a.taps - 1) * a.g_off + ch]; }
+    }
+    for (int i = a.dimp + tid; i < D; i += kStepThreads) q[i] = k[i] = 0.f;
     pdl_wait();
-    float* ring = a.ring + (size_t)(pos % a.taps) * a.g_off;
-    float qq = 0.f, kk = 0.f, kq = 0.f;
-    for (int i = tid; i < D; i += kDsThreads) {
-        float qv = 0.f, kv = 0.f;
-        if (i < a.dimp) {
-            const int cq = g * a.dimp + i, ck = a.k_off + cq;
-            qv = delta_conv(a, 0, pos, cq); kv = delta_conv(a, 0, pos, ck);
-        }
-        q[i] = qv; k[i] = kv;
-        qq = fmaf(qv, qv, qq); kk = fmaf(kv, kv, kk); kq = fmaf(kv, qv, kq);
+    float* ring = a.ring + (size_t)(pos % a.taps) * a.g_off;        // no convolution of this step reads this row
+    auto take = [&](int i, float y, float w) {
+        const int ch = channel(i);
+        const float x = __ldcg(a.raw + ch);
+        (i < a.dimp ? q + i : i < 2 * a.dimp ? k + i - a.dimp : v + i - 2 * a.dimp)[0] = silu_f(fmaf(w, x, y));
+        if (i >= 2 * a.dimp || (h % per == 0 && rank == 0)) ring[ch] = x;
+    };
+#pragma unroll
+    for (int x = 0; x < kDsHold; ++x) if (tid + x * kStepThreads < items) take(tid + x * kStepThreads, early[x], tap[x]);
+    for (int i = tid + kDsHold * kStepThreads; i < items; i += kStepThreads) { const int ch = channel(i); take(i, before(ch), a.conv[(size_t)(a.taps - 1) * a.g_off + ch]); }
+    if (tid == kStepThreads - 1) { sc[3] = delta_decay(a, a.raw, h); sc[4] = sigmoid_f(__ldcg(a.raw + a.b_off + h)); }
+    __syncthreads();
+    if (warp < 3) {                                     // q . q, k . k, k . q
+        const float *x = warp == 1 ? k : q, *y = warp == 0 ? q : k;
+        float t = 0.f;
+        for (int i = lane; i < a.dimp; i += 32) t = fmaf(x[i], y[i], t);
+        t = warp_sum(t);
+        if (lane == 0) sc[warp] = t;
     }
-    for (int c = tid; c < a.vdimp; c += kDsThreads) {
-        const int ch = a.v_off + h * a.vdimp + c;
-        v[c] = delta_conv(a, 0, pos, ch);
-        ring[ch] = __ldcg(a.raw + ch);                  // the ring's row of this position is read by no convolution of this step
-    }
-    if (h % per == 0)
-        for (int i = tid; i < a.dimp; i += kDsThreads) { const int cq = g * a.dimp + i; ring[cq] = __ldcg(a.raw + cq); ring[a.k_off + cq] = __ldcg(a.raw + a.k_off + cq); }
-    qq = cta_sum(qq, red); kk = cta_sum(kk, red); kq = cta_sum(kq, red);
-    const float fq = 1.0f / (sqrtf((float)a.dim) * sqrtf(qq + kUnitEps)), fk = 1.0f / sqrtf(kk + kUnitEps);
-    const float dec = delta_decay(a, a.raw, h), beta = sigmoid_f(__ldcg(a.raw + a.b_off + h));
-    kq *= fq * fk;
+    __syncthreads();
+    const float fq = 1.0f / (sqrtf((float)a.dim) * sqrtf(sc[0] + kUnitEps)), fk = 1.0f / sqrtf(sc[1] + kUnitEps), dec = sc[3], beta = sc[4], kq = sc[2] * fq * fk;
     const f32x2 g2 = pack2(dec, dec), fq2 = pack2(fq, fq), fk2 = pack2(fk, fk);
     f32x2 qu[2 * NV], ku[2 * NV];
     lane_units<LPC, NV>(q, l, qu); lane_units<LPC, NV>(k, l, ku);
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) { qu[i] = mul2(qu[i], fq2); ku[i] = mul2(ku[i], fk2); }
     float ss = 0.f;
-    for (int c0 = 0; c0 < a.vdimp; c0 += kDsHold * CH) {
-        if (c0) fetch(c0);
+    for (int cb = 0; cb < cw; cb += CH) {
+        const int c = cb + cg;
+        if (cb) fetch(c);
+        f32x2 k0 = 0ull, k1 = 0ull, q0 = 0ull, q1 = 0ull;
 #pragma unroll
-        for (int j = 0; j < kDsHold; ++j) {
-            const int c = c0 + j * CH + cg;
-            f32x2 k0 = 0ull, k1 = 0ull, q0 = 0ull, q1 = 0ull;
+        for (int i = 0; i < 2 * NV; i += 2) {
+            k0 = fma2(s.s[i], ku[i], k0); k1 = fma2(s.s[i + 1], ku[i + 1], k1);
+            q0 = fma2(s.s[i], qu[i], q0); q1 = fma2(s.s[i + 1], qu[i + 1], q1);
+        }
+        const float sk = lanes_sum<LPC>(sum2(add2(k0, k1))), sq = lanes_sum<LPC>(sum2(add2(q0, q1)));
+        if (c < cw) {
+            const float u = beta * (v[c] - dec * sk), x = fmaf(kq, u, dec * sq);
+            const f32x2 u2 = pack2(u, u);
 #pragma unroll
-            for (int i = 0; i < 2 * NV; i += 2) {
-                k0 = fma2(s[j].s[i], ku[i], k0); k1 = fma2(s[j].s[i + 1], ku[i + 1], k1);
-                q0 = fma2(s[j].s[i], qu[i], q0); q1 = fma2(s[j].s[i + 1], qu[i + 1], q1);
-            }
-            const float sk = lanes_sum<LPC>(sum2(add2(k0, k1))), sq = lanes_sum<LPC>(sum2(add2(q0, q1)));
-            if (c < a.vdimp) {
-                const float u = beta * (v[c] - dec * sk), x = fmaf(kq, u, dec * sq);
-                const f32x2 u2 = pack2(u, u);
-#pragma unroll
-                for (int i = 0; i < 2 * NV; ++i) s[j].s[i] = fma2(s[j].s[i], g2, mul2(ku[i], u2));
-                s[j].store(a.state + ((size_t)h * a.vdimp + c) * a.dimp, l, a.dimp);
-                if (l == 0) { o[c] = x; ss = fmaf(x, x, ss); }
-            }
+            for (int i = 0; i < 2 * NV; ++i) s.s[i] = fma2(s.s[i], g2, mul2(ku[i], u2));
+            s.store(a.state + ((size_t)h * a.vdimp + c0 + c) * a.dimp, l, a.dimp);
+            if (l == 0) { o[c] = x; ss = fmaf(x, x, ss); }
         }
     }
-    const float inv = inv_rms(cta_sum(ss, red), a.vdim, sa.eps) * sa.scale;
-    const size_t ho = (size_t)h * a.vdimp;
-    for (int c = tid; c < a.vdimp; c += kDsThreads) sa.out[ho + c] = __float2bfloat16_rn(c < a.vdim ? o[c] * inv * sa.norm[c] * silu_f(__ldcg(a.raw + a.g_off + ho + c)) : 0.f);
+    const float inv = inv_rms(cluster_sum(ss, sp.ncl, rank, red, slots), a.vdim, sa.eps) * sa.scale;
+    for (int i = tid; i < cw; i += kStepThreads) {
+        const int c = c0 + i;
+        const size_t at = (size_t)h * a.vdimp + c;
+        sa.out[at] = __float2bfloat16_rn(c < a.vdim ? o[i] * inv * sa.norm[c] * silu_f(__ldcg(a.raw + a.g_off + at)) : 0.f);
+    }
 }
 template <int LPC, int NV>
 static int ds_go(const DeltaStepArgs& a, const LaunchCfg& cfg) {
-    const size_t smem = (size_t)(2 * LPC * NV * 4 + 2 * a.d.vdimp) * 4;
+    const StepSplit sp = step_split(a.d.vdimp, LPC);
+    const size_t smem = (size_t)(2 * LPC * NV * 4 + 2 * sp.cw) * 4;
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-    return st_launch(delta_step_kernel<LPC, NV>, dim3(a.d.heads), dim3(kDsThreads), smem, cfg, a);
+    return st_launch_cluster(delta_step_kernel<LPC, NV>, dim3(a.d.heads, sp.ncl), sp.ncl, dim3(kStepThreads), smem, cfg, a, sp);
 }
 int launch_delta_step(const DeltaStepArgs& a, const LaunchCfg& cfg) {
     const DeltaArgs& d = a.d;

@@ -66,6 +66,56 @@ inline int recur_map(CUtensorMap* m, const float* p, int len, int heads, int hs,
                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
 }
+// One token, one head to a cluster: CTA `rank` of the cluster has value channels [rank * cw, ...).  The cluster's CTAs exchange the sums of
+// squares of their read-outs, so that each norms its own channels.
+constexpr int kStepThreads = 256;
+struct StepSplit { int ncl, cw; };
+inline StepSplit step_split(int channels, int lpc) {
+    const int ch = kStepThreads / lpc;                  // channels at a time
+    int n = (channels + ch - 1) / ch;
+    if (n > 8) n = 8;
+    const int cw = ((channels + n - 1) / n + 7) / 8 * 8;
+    return {(channels + cw - 1) / cw, cw};
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+// Sum over the cluster of every CTA's `v` (summed over its threads).  red: 8 warps' sums, slots: one word per CTA.  Every CTA has arrived at the
+// cluster barrier once before.
+__device__ __forceinline__ float cluster_sum(float v, int ncl, int rank, float* red, float* slots) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) s += red[i];
+    if (ncl == 1) return s;
+    cluster_wait();                                     // all CTAs of the cluster run
+    if ((int)threadIdx.x < ncl) {
+        uint32_t dst;
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(smem_u32(slots + rank)), "r"((int)threadIdx.x));
+        asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(s) : "memory");
+    }
+    __syncwarp();
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    cluster_wait();
+    s = 0.f;
+    for (int i = 0; i < ncl; ++i) s += slots[i];        // the same order in every CTA
+    return s;
+}
+// Launch with clusters of ncl CTAs along y.
+template <typename... KArgs, typename... Args>
+static int st_launch_cluster(void (*kern)(KArgs...), dim3 grid, int ncl, dim3 block, size_t smem, const LaunchCfg& cfg, Args... args) {
+    cudaLaunchConfig_t lc = {};
+    lc.gridDim = grid; lc.blockDim = block; lc.dynamicSmemBytes = smem; lc.stream = cfg.stream;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = 1; at[0].val.clusterDim.y = ncl; at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    lc.attrs = at; lc.numAttrs = cfg.pdl ? 2 : 1;
+    return (int)cudaLaunchKernelEx(&lc, kern, KArgs(args)...);
+}
+
 constexpr int kRecurTile = 16;                          // tokens brought at a time
 constexpr int recur_box(int d) { return d < 256 ? d : 256; }
 // One head's `D` places of kRecurTile rows from row t on, [row][place] in pieces of 256 places.

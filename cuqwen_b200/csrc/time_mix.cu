@@ -160,85 +160,95 @@ int launch_time_mix_scan(const TimeMixArgs& a, const LaunchCfg& cfg) {
 }
 
 // ---- one token --------------------------------------------------------------------------------------------------------
-// CTA = head; the three CTAs behind the heads put the token's q, k and v rows in place.  The state of the first value channels is
-// on its way before the dependency wait (it was written by an earlier step).
-constexpr int kTsThreads = 512, kTsHold = 2;            // channels of a thread held at a time
+// A cluster per head; a CTA each for the token's q, k and v rows behind the heads (the first of their clusters).  On their way before the
+// dependency wait: the state of a CTA's first value channels (an earlier step wrote it) and the first rows of w2.
+constexpr int kTsRowLanes = 8;                          // lanes to a key channel's row of w2, eight values each at a time
 template <int LPC, int NV>
-__global__ void __launch_bounds__(kTsThreads) time_mix_step_kernel(const TimeMixStepArgs a) {
-    constexpr int D = LPC * NV * 4, CH = kTsThreads / LPC;                               // value channels at a time
-    extern __shared__ __align__(16) float ts_smem[];    // r [D], k [D], w [D], tanh [rank], o [dimp]
-    __shared__ float red[40];
+__global__ void __launch_bounds__(kStepThreads) time_mix_step_kernel(const TimeMixStepArgs a, const StepSplit sp) {
+    constexpr int D = LPC * NV * 4, CH = kStepThreads / LPC, ROWS = kStepThreads / kTsRowLanes, PRE = 2;
+    extern __shared__ __align__(16) float ts_smem[];    // r [D], k [D], w [D], tanh [rank rounded up to eight], o [cw]
+    __shared__ float red[8], slots[8], bonus_s;
     pdl_launch_dependents();
-    const int h = blockIdx.x, tid = threadIdx.x, l = tid % LPC, cg = tid / LPC, pos = *a.pos_ptr;      // written before the step's first kernel released its dependents
+    const int h = blockIdx.x, rank = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = tid % LPC, cg = tid / LPC, pos = *a.pos_ptr;      // written before the step's first kernel released its dependents
     if (h >= a.heads) {
         pdl_wait();
-        qkv_section<bf16>(a.qkv, 0, pos, h - a.heads, tid, kTsThreads);
+        if (rank == 0) qkv_section<bf16>(a.qkv, 0, pos, h - a.heads, tid, kStepThreads);
         return;
     }
-    float *r = ts_smem, *k = r + D, *w = k + D, *o = w + D, *th = o + a.dimp;
+    const int c0 = rank * sp.cw, cw = min(sp.cw, a.dimp - c0), rankp = (a.rank + 7) / 8 * 8;
+    float *r = ts_smem, *k = r + D, *w = k + D, *th = w + D, *o = th + rankp;
     const size_t ho = (size_t)h * a.dimp;
-    StateCol<LPC, NV> s[kTsHold];
-    auto fetch = [&](int c0) {
+    if (sp.ncl > 1) cluster_arrive();
+    StateCol<LPC, NV> s;
+    auto fetch = [&](int c) { if (c < cw && pos > 0) s.load(a.state + (ho + c0 + c) * a.dimp, l, a.dimp); else s.zero(); };
+    fetch(cg);
+    const int row = tid / kTsRowLanes, part = tid % kTsRowLanes * 8;
+    uint4 pre[PRE];                                     // the pitch covers whole units of eight, zeros behind the rank
 #pragma unroll
-        for (int j = 0; j < kTsHold; ++j) {
-            const int c = c0 + j * CH + cg;
-            if (c < a.dimp && pos > 0) s[j].load(a.state + (ho + c) * a.dimp, l, a.dimp); else s[j].zero();
-        }
-    };
-    fetch(0);
+    for (int j = 0; j < PRE; ++j) pre[j] = row + j * ROWS < a.dimp && part < rankp ? ldg_stream(a.w2 + (ho + row + j * ROWS) * a.w2_pitch + part) : make_uint4(0u, 0u, 0u, 0u);
+    for (int i = a.dimp + tid; i < D; i += kStepThreads) r[i] = k[i] = w[i] = 0.f;
     pdl_wait();
-    float b = 0.f;
-    for (int i = tid; i < D; i += kTsThreads) {
-        const bool in = i < a.dimp;
-        const float rv = in ? __ldcg(a.r + ho + i) : 0.f, kv = in ? __ldcg(a.k + ho + i) : 0.f;
-        r[i] = rv; k[i] = kv; w[i] = 0.f;
-        if (in) b = fmaf(rv * a.u[ho + i], kv, b);
-    }
-    for (int i = tid; i < a.rank; i += kTsThreads) th[i] = tanhf(__ldcg(a.w1 + i));
-    const float bonus = cta_sum(b, red);                // barriers inside
-    // decays: a warp per key channel
-    for (int i = tid >> 5; i < a.dimp; i += kTsThreads / 32) {
-        const bf16* row = a.w2 + (ho + i) * a.w2_pitch;
+    for (int i = tid; i < 2 * a.dimp; i += kStepThreads) { if (i < a.dimp) r[i] = __ldcg(a.r + ho + i); else k[i - a.dimp] = __ldcg(a.k + ho + i - a.dimp); }
+    for (int i = tid; i < rankp; i += kStepThreads) th[i] = i < a.rank ? tanhf(__ldcg(a.w1 + i)) : 0.f;
+    __syncthreads();
+    for (int j = 0; row + j * ROWS < a.dimp; ++j) {     // the lanes of a row leave together; rows of a warp may differ by one round
+        const int key = row + j * ROWS;
         float z = 0.f;
-        for (int q = tid & 31; q < a.rank; q += 32) z = fmaf(th[q], __bfloat162float(row[q]), z);
-        z = warp_sum(z);
-        if ((tid & 31) == 0) w[i] = expf(-expf(z + a.w0[ho + i]));
+        for (int p = part; p < rankp; p += kTsRowLanes * 8) {
+            float x[8];
+            if (j < PRE && p == part) unpack8(j == 0 ? pre[0] : pre[1], x); else load8(a.w2 + (ho + key) * a.w2_pitch + p, x);
+#pragma unroll
+            for (int q = 0; q < 8; ++q) z = fmaf(th[p + q], x[q], z);
+        }
+        const unsigned mask = 0xffu << (lane & 24);
+#pragma unroll
+        for (int d = kTsRowLanes / 2; d > 0; d >>= 1) z += __shfl_xor_sync(mask, z, d);
+        if (part == 0) w[key] = expf(-expf(z + a.w0[ho + key]));
+    }
+    if (warp == kStepThreads / 32 - 1) {
+        __syncwarp();
+        float b = 0.f;
+        for (int i = lane; i < a.dimp; i += 32) b = fmaf(r[i] * a.u[ho + i], k[i], b);
+        b = warp_sum(b);
+        if (lane == 0) bonus_s = b;
     }
     __syncthreads();
+    const float bonus = bonus_s;
     f32x2 rr[2 * NV], kk[2 * NV], ww[2 * NV];
     lane_units<LPC, NV>(r, l, rr); lane_units<LPC, NV>(k, l, kk); lane_units<LPC, NV>(w, l, ww);
     float ss = 0.f;
-    for (int c0 = 0; c0 < a.dimp; c0 += kTsHold * CH) {
-        if (c0) fetch(c0);
+    for (int cb = 0; cb < cw; cb += CH) {
+        const int c = cb + cg;
+        if (cb) fetch(c);
+        const float v = c < cw ? __ldcg(a.v + ho + c0 + c) : 0.f;
+        const f32x2 v2 = pack2(v, v);
+        f32x2 acc = 0ull, acc1 = 0ull;
 #pragma unroll
-        for (int j = 0; j < kTsHold; ++j) {
-            const int c = c0 + j * CH + cg;
-            const float v = c < a.dimp ? __ldcg(a.v + ho + c) : 0.f;
-            const f32x2 v2 = pack2(v, v);
-            f32x2 acc = 0ull, acc1 = 0ull;
-#pragma unroll
-            for (int i = 0; i < 2 * NV; i += 2) {
-                acc = fma2(s[j].s[i], rr[i], acc); acc1 = fma2(s[j].s[i + 1], rr[i + 1], acc1);
-                s[j].s[i] = fma2(s[j].s[i], ww[i], mul2(kk[i], v2)); s[j].s[i + 1] = fma2(s[j].s[i + 1], ww[i + 1], mul2(kk[i + 1], v2));
-            }
-            const float x = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v;
-            if (c < a.dimp) {
-                s[j].store(a.state + (ho + c) * a.dimp, l, a.dimp);
-                if (l == 0) { o[c] = x; ss = fmaf(x, x, ss); }
-            }
+        for (int i = 0; i < 2 * NV; i += 2) {
+            acc = fma2(s.s[i], rr[i], acc); acc1 = fma2(s.s[i + 1], rr[i + 1], acc1);
+            s.s[i] = fma2(s.s[i], ww[i], mul2(kk[i], v2)); s.s[i + 1] = fma2(s.s[i + 1], ww[i + 1], mul2(kk[i + 1], v2));
+        }
+        const float x = lanes_sum<LPC>(sum2(add2(acc, acc1))) + bonus * v;
+        if (c < cw) {
+            s.store(a.state + (ho + c0 + c) * a.dimp, l, a.dimp);
+            if (l == 0) { o[c] = x; ss = fmaf(x, x, ss); }
         }
     }
-    const float inv = inv_rms(cta_sum(ss, red), a.dim, a.eps) * a.scale;
-    for (int c = tid; c < a.dimp; c += kTsThreads) a.out[ho + c] = __float2bfloat16_rn(c < a.dim ? o[c] * inv * a.norm[ho + c] * silu_f(__ldcg(a.g + ho + c)) : 0.f);
+    const float inv = inv_rms(cluster_sum(ss, sp.ncl, rank, red, slots), a.dim, a.eps) * a.scale;
+    for (int i = tid; i < cw; i += kStepThreads) {
+        const int c = c0 + i;
+        a.out[ho + c] = __float2bfloat16_rn(c < a.dim ? o[i] * inv * a.norm[ho + c] * silu_f(__ldcg(a.g + ho + c)) : 0.f);
+    }
 }
 template <int LPC, int NV>
 static int ts_go(const TimeMixStepArgs& a, const LaunchCfg& cfg) {
-    const size_t smem = (size_t)(3 * LPC * NV * 4 + a.dimp + a.rank) * 4;
+    const StepSplit sp = step_split(a.dimp, LPC);
+    const size_t smem = (size_t)(3 * LPC * NV * 4 + sp.cw + (a.rank + 7) / 8 * 8) * 4;
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-    return st_launch(time_mix_step_kernel<LPC, NV>, dim3(a.heads + (a.qkv.raw ? 3 : 0)), dim3(kTsThreads), smem, cfg, a);
+    return st_launch_cluster(time_mix_step_kernel<LPC, NV>, dim3(a.heads + (a.qkv.raw ? 3 : 0), sp.ncl), sp.ncl, dim3(kStepThreads), smem, cfg, a, sp);
 }
 int launch_time_mix_step(const TimeMixStepArgs& a, const LaunchCfg& cfg) {
-    if (a.heads < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.rank < 1 || (a.qkv.raw && !qkv_rows_ok(a.qkv))) return (int)cudaErrorInvalidValue;
+    if (a.heads < 1 || a.dimp < 8 || a.dimp % 8 || a.dimp > kRecurMaxDim || a.rank < 1 || a.w2_pitch % 8 || a.w2_pitch < a.rank || (a.qkv.raw && !qkv_rows_ok(a.qkv))) return (int)cudaErrorInvalidValue;
 #define GO(L, N) ts_go<L, N>(a, cfg)
     return RECUR_DISPATCH(a.dimp, GO);
 #undef GO
