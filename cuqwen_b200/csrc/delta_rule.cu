@@ -167,6 +167,7 @@ __global__ void __launch_bounds__(CB / NC * LPC) delta_scan_kernel(const DeltaAr
     float* st = a.state + ((size_t)h * a.vdimp + c) * a.dimp;         // vdimp is a multiple of eight: both channels exist or none
 #pragma unroll
     for (int j = 0; j < NC; ++j) if (c < a.vdimp && first > 0) s[j].load(st + j * a.dimp, l, a.dimp); else s[j].zero();
+    float* out = a.o + (size_t)l * a.ldo + (size_t)h * a.vdimp + c;
     bool failed = false;
     for (int t0 = 0, i = 0; t0 < a.T; t0 += kRecurTile, ++i) {
         const int b = i & 1;
@@ -236,10 +237,10 @@ __global__ void __launch_bounds__(CB / NC * LPC) delta_scan_kernel(const DeltaAr
                 }
             }
             // lane t of a channel's first four stores token t
-            if (l < 4 && tb + l < n && c < a.vdimp) {
-                const float2 r = l == 0 ? make_float2(o[0][0], o[0][1]) : l == 1 ? make_float2(o[1][0], o[1][1]) : l == 2 ? make_float2(o[2][0], o[2][1]) : make_float2(o[3][0], o[3][1]);
-                *reinterpret_cast<float2*>(a.o + (size_t)(t0 + tb + l) * a.ldo + (size_t)h * a.vdimp + c) = r;
-            }
+            float2 r = make_float2(o[0][0], o[0][1]);
+#pragma unroll
+            for (int t = 1; t < 4; ++t) { r.x = l == t ? o[t][0] : r.x; r.y = l == t ? o[t][1] : r.y; }
+            if (tb + l < min(n, tb + 4) && c < a.vdimp) *reinterpret_cast<float2*>(out + (size_t)(t0 + tb) * a.ldo) = r;
         }
         __syncthreads();
         if (tid == 0 && t0 + 2 * kRecurTile < a.T) bring(t0 + 2 * kRecurTile, b);

@@ -1006,7 +1006,7 @@ extern "C" int cuqwen_get_ptr(cuqwen_engine* e, int which, int layer, void** ptr
         switch (which) {
             case CUQWEN_PTR_X: stack_residual(e->stack, &r, &b); break;                       // float32
             case CUQWEN_PTR_LOGITS: r = stack_logits(e->stack); b = (size_t)p.vocab_size * 4; break;      // float32
-            case CUQWEN_PTR_KEY_CACHE: b = stack_cache_bytes(e->stack, &r); break;             // every layer's latent rows
+            case CUQWEN_PTR_KEY_CACHE: b = stack_cache_bytes(e->stack, &r); break;             // every layer's cache rows and states
             case CUQWEN_PTR_HISTORY: r = e->d_hist; b = (size_t)p.max_seq_len * 4; break;
             case CUQWEN_PTR_TOKEN: r = &e->ctl->token; b = 4; break;
             case CUQWEN_PTR_POS: r = &e->ctl->pos; b = 4; break;

@@ -1,18 +1,19 @@
-// Host side of the layer-list designs: weights from a model directory, the latent cache, and the launch sequences of a
-// decode step and of a prompt portion.  Kernels: stack.h.
+// Host side of the layer-list designs: weights from a model directory, caches and states, and the launch sequences of a decode
+// step and of a prompt portion (latent attention layers; stack_mixers.cu has those of sequential layers).  Kernels: stack.h.
 //
 // Layout.  Every per-head or per-part length is padded to a multiple of eight with zero weight rows / columns when the
 // weights are loaded, so that rows start on 16-byte boundaries and padded places hold zeros; weight rows are padded to a
 // multiple of 128 columns.  For the usual sizes nothing is added.
 //   q            [heads][dim | rot_dim]
 //   cache row    [latent kv_rank | rotated key part rot_dim], one array [max_seq_len][row] per layer with a projection of its own
+// Sequential layers: keys and values [kv_heads][max_seq_len][key dim | value vdim]; recurrent states float32 [heads][value channel]
+// [key channel]; the inputs that a later token still needs in rings by position.
 //   raw          [query latent q_rank | cache row | gate heads * vdim], float32 sums of the first launch of a layer
 #include "stack_pass.h"
 
 #include <cmath>
 
 namespace cq {
-
 
 const StackSpec& stack_spec(const Stack* s) { return s->spec; }
 int stack_act(const Stack* s) { return s->act; }

@@ -61,8 +61,8 @@ enum LinEpi : int {
     LIN_ADD = 3,          // out (float) += c0 * acc
     LIN_GELU_SIDE = 4,    // out (activation type) = gelu_tanh(acc) * side[tokens[t]][r]
     LIN_CAP = 5,          // out (float) = c0 * tanh(acc / c0)
-    LIN_DECAY = 7,        // out (float) = exp(-exp(acc + bias[r]))
-    LIN_GLU = 6           // out (activation type) = clamped_glu(gate, up, limit c0, slope c1); rows come as eight of the gate, eight of the up matrix in turn
+    LIN_GLU = 6,          // out (activation type) = clamped_glu(gate, up, limit c0, slope c1); rows come as eight of the gate, eight of the up matrix in turn
+    LIN_DECAY = 7         // out (float) = exp(-exp(acc + bias[r]))
 };
 struct LinArgs {
     const void* x; int ldx; const bf16* w; int pitch, K;

@@ -8,7 +8,7 @@
 
 namespace cq {
 
-// Sizes, workspace-independent state and the latent cache.  Fills e->p's model fields.
+// Sizes, caches and recurrent states.  Fills e->p's model fields.
 int stack_create(cuqwen_engine* e, const StackSpec& spec, int act, int max_seq_len);
 int stack_load(cuqwen_engine* e, const char* dir);
 void stack_destroy(cuqwen_engine* e);
