@@ -71,7 +71,8 @@ typedef struct cuqwen_params {
  * DIR/config.json names a design of the library's registry and describes it layer by layer; DIR/model.safetensors holds
  * its bfloat16 weights.  An engine opened from a directory takes the same calls as one made by cuqwen_create: cuqwen_step,
  * cuqwen_step_loop, cuqwen_decode_n, cuqwen_prefill, cuqwen_extend, cuqwen_step_profile, cuqwen_destroy.  Its logits and
- * residual stream (cuqwen_get_ptr) are float32.  One GPU. */
+ * residual stream (cuqwen_get_ptr) are float32.  One GPU.  A design with a recurrence takes positions in order: a call goes on
+ * where the last one ended or starts a sequence at position 0, anything else is CUQWEN_ERR_STATE and changes nothing. */
 enum { CUQWEN_ACT_BF16 = 0,      /* bfloat16 matrix products and activations, 32-bit accumulation, residual stream, norms, softmax */
        CUQWEN_ACT_F32 = 1 };     /* everything in 32-bit (plain CUDA-core kernels: a check, not a serving mode) */
 typedef struct cuqwen_open_params {
@@ -81,7 +82,7 @@ typedef struct cuqwen_open_params {
     uint32_t flags;              /* CUQWEN_FLAG_NO_PDL, CUQWEN_FLAG_NO_GRAPH */
     float repetition_penalty;    /* 0 = 1.1 */
 } cuqwen_open_params;
-/* Reads, creates and loads in one call.  Designs: Falivik. */
+/* Reads, creates and loads in one call.  Designs: Falivik, Gipotar. */
 int cuqwen_open(const char* dir, const cuqwen_open_params* p, cuqwen_engine** out);
 /* The configuration as the library understood it, one line of text per layer.  Host only. */
 int cuqwen_describe(const char* dir, char* out, size_t cap);
